@@ -2,7 +2,7 @@
 grouped by what layers need, and slots of fixed-size per-request state.
 
 * A *group* is a set of scheduled layer runs with the same paged-cache needs
-  (kv heads, head size, window).  Each group has its own page pool, its own
+  (kv heads, head sizes, window, run of positions).  Each group has its own page pool, its own
   device pools (one K and one V tensor ``[pages, kv_heads, page_size, hd]``
   per member) and its own block table per request; one page id covers all
   members of its group.  The reference has a single implicit group: one table
@@ -10,8 +10,9 @@ grouped by what layers need, and slots of fixed-size per-request state.
   719-721).
 * Pages are taken per step for exactly the tokens of that step (``extend``),
   counted as cached after the step ran (``commit``), and given back when the
-  request ends (``release``) or - in a group with a window - once every token
-  on them is out of reach of all later queries (pages that hold one of the
+  request ends (``release``) or - in a group with a window, or whose queries see
+  their own run of positions only (``chunk``) - once every token on them is out of
+  reach of all later queries (pages that hold one of the
   group's ``keep_first`` first tokens stay).  A returned page is handed out
   again first.  (The reference allocates a whole prompt at admission and
   frees only at the end: infernum-runtime/src/scheduler.rs:289-337.)
@@ -219,11 +220,13 @@ class CacheManager:
     def peak_pages(self, total_tokens: int, step_tokens: int) -> List[int]:
         """Per group, the most pages a request of ``total_tokens`` cached tokens
         holds at any time when it is fed at most ``step_tokens`` a step: all of
-        its pages, or, in a group with a window, those the window and one step
-        reach (older ones are given back at every commit)."""
+        its pages, or, in a group with a window or runs of positions, those the window
+        (the run) and one step reach (older ones are given back at every commit)."""
         out = []
         for g in self.groups:
             need = self.pages_for(total_tokens)
+            if g.spec.chunk > 0:
+                need = min(need, self.pages_for(g.spec.chunk + step_tokens) + 1)
             if g.spec.window > 0:
                 need = min(need, self.pages_for(g.spec.window + step_tokens) + 1 + self.pages_for(g.spec.keep_first))
             out.append(need)
@@ -311,12 +314,14 @@ class CacheManager:
             raise CacheError("commit: more tokens than pages were held for")
         rc.num_tokens += new_tokens
         for g, table in zip(self.groups, rc.tables):
-            w = g.spec.window
-            if w <= 0:
+            w, chunk = g.spec.window, g.spec.chunk
+            if w <= 0 and chunk <= 0:
                 continue
-            # the next query sits at position >= num_tokens and reads keys
-            # >= num_tokens - w + 1; page i holds [i*ps, (i+1)*ps)
-            first_needed = rc.num_tokens - w + 1
+            # the next query sits at position >= num_tokens and reads keys >= num_tokens - w + 1 and none
+            # before its own run of ``chunk`` positions; page i holds [i*ps, (i+1)*ps)
+            first_needed = rc.num_tokens - w + 1 if w > 0 else 0
+            if chunk > 0:
+                first_needed = max(first_needed, rc.num_tokens // chunk * chunk)
             i = self.pages_for(g.spec.keep_first)  # the pages of the tokens that stay visible are kept
             while i < len(table) and (i + 1) * self.page_size <= first_needed:
                 if table[i] >= 0:

@@ -194,6 +194,19 @@ __device__ __forceinline__ float block_max(float v, float* scratch) {
     return scratch[32];
 }
 
+// The activated gate times its up, in 32-bit: act 1 = SiLU, g / (1 + exp(-g)); 2 = GELU in its tanh form,
+// 0.5 g (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3))); 3 = clamped swish, g' / (1 + exp(-alpha g')) * (u' + 1) with
+// g' = min(g, limit) and u' = u held to [-limit, limit] (limit and alpha matter to it alone).
+__device__ __forceinline__ float gate_times(float g, float u, int act, float limit, float alpha) {
+    if (act == 2) return 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
+    if (act == 3) {
+        g = fminf(g, limit);
+        u = fminf(fmaxf(u, -limit), limit);
+        return g / (1.f + expf(-alpha * g)) * (u + 1.f);
+    }
+    return g / (1.f + expf(-g)) * u;
+}
+
 }  // namespace ib
 
 // Turns programmatic dependent launch on or off for this library (default on).

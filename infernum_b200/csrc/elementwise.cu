@@ -18,11 +18,12 @@
 using namespace ib;
 
 // ---------------------------------------------------------------------------
-// Embedding: residual[t, :] = table[ids[t], :] widened to 32-bit.
+// Embedding: residual[t, :] = table[ids[t], :] * scale, in 32-bit.
 // ---------------------------------------------------------------------------
 template <typename TW>
 __global__ void embed_kernel(const int* __restrict__ ids, const TW* __restrict__ table,
-                             float* __restrict__ out, int H, int V, unsigned* __restrict__ err) {
+                             float* __restrict__ out, int H, int V, float scale,
+                             unsigned* __restrict__ err) {
     pdl_trigger();
     pdl_wait();
     const int row = blockIdx.x;
@@ -34,23 +35,28 @@ __global__ void embed_kernel(const int* __restrict__ ids, const TW* __restrict__
         return;
     }
     const TW* src = table + (size_t)id * H;
-    for (int i = threadIdx.x; i < H; i += blockDim.x) o[i] = to_f32(src[i]);
+    for (int i = threadIdx.x; i < H; i += blockDim.x) o[i] = to_f32(src[i]) * scale;
 }
 
-IB_EXPORT int ib_embed(const int* ids, const void* table, int table_dtype, float* out, int n_rows,
-                       int H, int V, unsigned* err, void* stream) {
+IB_EXPORT int ib_embed_scaled(const int* ids, const void* table, int table_dtype, float* out, int n_rows,
+                       int H, int V, float scale, unsigned* err, void* stream) {
     if (n_rows <= 0) return IB_OK;
     if (H <= 0 || V <= 0 || !ids || !table || !out || !err) return IB_ERR_BAD_ARG;
     cudaStream_t s = (cudaStream_t)stream;
     const int threads = H >= 1024 ? 256 : 128;
     if (table_dtype == 0)
-        { cudaError_t le__ = launch_kernel(embed_kernel<float>, dim3(n_rows), dim3(threads), 0, s, ids, (const float*)table, out, H, V, err); if (le__ != cudaSuccess) return (int)le__; }
+        { cudaError_t le__ = launch_kernel(embed_kernel<float>, dim3(n_rows), dim3(threads), 0, s, ids, (const float*)table, out, H, V, scale, err); if (le__ != cudaSuccess) return (int)le__; }
     else if (table_dtype == 1)
-        { cudaError_t le__ = launch_kernel(embed_kernel<bf16>, dim3(n_rows), dim3(threads), 0, s, ids, (const bf16*)table, out, H, V, err); if (le__ != cudaSuccess) return (int)le__; }
+        { cudaError_t le__ = launch_kernel(embed_kernel<bf16>, dim3(n_rows), dim3(threads), 0, s, ids, (const bf16*)table, out, H, V, scale, err); if (le__ != cudaSuccess) return (int)le__; }
     else
         return IB_ERR_UNSUPPORTED;
     IB_LAUNCH_CHECK();
     return IB_OK;
+}
+
+IB_EXPORT int ib_embed(const int* ids, const void* table, int table_dtype, float* out, int n_rows, int H, int V,
+                       unsigned* err, void* stream) {
+    return ib_embed_scaled(ids, table, table_dtype, out, n_rows, H, V, 1.f, err, stream);
 }
 
 // ---------------------------------------------------------------------------
@@ -233,6 +239,125 @@ IB_EXPORT int ib_add_rmsnorm(float* residual, const void* delta, const void* wei
     if (act_dtype == 1)
         return launch_add_rmsnorm<bf16, bf16>(residual, delta, weight, weight_dtype, out, row_idx,
                                               n_rows, H, eps, write_residual, s);
+    return IB_ERR_UNSUPPORTED;
+}
+
+// ---------------------------------------------------------------------------
+// Two RMS norms of one row, for layers whose mixer and feed-forward read the
+// same sum: s = x[row] (+ delta[row]); x_out[row] = s (x_out may be x, and is
+// not written when there is no delta and it is x); with the one root r of
+// (mean(s^2) + eps), out1 = s / r * w1 and out2 = s / r * w2.  One block per row;
+// a row stays in shared memory between the two passes.
+// ---------------------------------------------------------------------------
+template <typename TD, typename TW>
+__global__ void add_rmsnorm_pair_kernel(const float* x, const TD* __restrict__ delta, float* x_out,
+                                        const TW* __restrict__ w1, const TW* __restrict__ w2, TD* __restrict__ out1,
+                                        TD* __restrict__ out2, int H, float eps) {
+    pdl_trigger();
+    pdl_wait();
+    __shared__ float scratch[33];
+    extern __shared__ __align__(16) float held[];
+    const size_t at = (size_t)blockIdx.x * H;
+    const bool store = delta != nullptr || x_out != x;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+        float v = x[at + i];
+        if (delta) v += to_f32(delta[at + i]);
+        if (store) x_out[at + i] = v;
+        held[i] = v;
+        ss = fmaf(v, v, ss);
+    }
+    ss = block_sum(ss, scratch);
+    const float inv = rsqrtf(ss / (float)H + eps);
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+        const float n = held[i] * inv;
+        out1[at + i] = from_f32<TD>(n * to_f32(w1[i]));
+        out2[at + i] = from_f32<TD>(n * to_f32(w2[i]));
+    }
+}
+
+// Four elements a load, NV groups of four a thread in registers (H a multiple of 4, 16-byte aligned rows).
+template <typename TD, typename TW, int NV>
+__global__ void add_rmsnorm_pair_vec_kernel(const float* x, const TD* __restrict__ delta, float* x_out,
+                                            const TW* __restrict__ w1, const TW* __restrict__ w2, TD* __restrict__ out1,
+                                            TD* __restrict__ out2, int H, float eps) {
+    pdl_trigger();
+    pdl_wait();
+    __shared__ float scratch[33];
+    const size_t at = (size_t)blockIdx.x * H;
+    const bool store = delta != nullptr || x_out != x;
+    const int groups = H >> 2;
+    float4 v[NV];
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+        const int g = threadIdx.x + k * blockDim.x;
+        if (g < groups) {
+            v[k] = Vec4<float>::load(x + at + 4 * g);
+            if (delta) {
+                const float4 dv = Vec4<TD>::load(delta + at + 4 * g);
+                v[k].x += dv.x; v[k].y += dv.y; v[k].z += dv.z; v[k].w += dv.w;
+            }
+            if (store) Vec4<float>::store(x_out + at + 4 * g, v[k]);
+            ss += v[k].x * v[k].x + v[k].y * v[k].y + v[k].z * v[k].z + v[k].w * v[k].w;
+        }
+    }
+    ss = block_sum(ss, scratch);
+    const float inv = rsqrtf(ss / (float)H + eps);
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+        const int g = threadIdx.x + k * blockDim.x;
+        if (g < groups) {
+            const float4 n = make_float4(v[k].x * inv, v[k].y * inv, v[k].z * inv, v[k].w * inv);
+            const float4 a = Vec4<TW>::load(w1 + 4 * g), b = Vec4<TW>::load(w2 + 4 * g);
+            Vec4<TD>::store(out1 + at + 4 * g, make_float4(n.x * a.x, n.y * a.y, n.z * a.z, n.w * a.w));
+            Vec4<TD>::store(out2 + at + 4 * g, make_float4(n.x * b.x, n.y * b.y, n.z * b.z, n.w * b.w));
+        }
+    }
+}
+
+template <typename TD, typename TW>
+static int launch_rmsnorm_pair(const float* x, const void* delta, float* x_out, const void* w1, const void* w2, void* out1,
+                               void* out2, int n_rows, int H, float eps, cudaStream_t s) {
+    cudaError_t le;
+    const uintptr_t bases = (uintptr_t)x | (uintptr_t)delta | (uintptr_t)x_out | (uintptr_t)w1 | (uintptr_t)w2 |
+                            (uintptr_t)out1 | (uintptr_t)out2;
+    const int groups = H / 4;
+    if (H % 4 == 0 && !(bases & 15) && groups <= 4096) {
+        const int nv = groups <= 512 ? 1 : (groups <= 1024 ? 2 : (groups <= 2048 ? 4 : 8));
+        const int threads = ((groups + nv - 1) / nv + 31) / 32 * 32;
+#define IB_PAIR(NV)                                                                                                    \
+    le = launch_kernel(add_rmsnorm_pair_vec_kernel<TD, TW, NV>, dim3(n_rows), dim3(threads), 0, s, x, (const TD*)delta, \
+                       x_out, (const TW*)w1, (const TW*)w2, (TD*)out1, (TD*)out2, H, eps)
+        if (nv == 1) IB_PAIR(1);
+        else if (nv == 2) IB_PAIR(2);
+        else if (nv == 4) IB_PAIR(4);
+        else IB_PAIR(8);
+#undef IB_PAIR
+    } else {
+        const size_t smem = (size_t)H * sizeof(float);
+        if (smem > 48 * 1024 - 256) return IB_ERR_TOO_LARGE;
+        le = launch_kernel(add_rmsnorm_pair_kernel<TD, TW>, dim3(n_rows), dim3(256), smem, s, x, (const TD*)delta, x_out,
+                           (const TW*)w1, (const TW*)w2, (TD*)out1, (TD*)out2, H, eps);
+    }
+    if (le != cudaSuccess) return (int)le;
+    IB_LAUNCH_CHECK();
+    return IB_OK;
+}
+
+// act_dtype is the type of `delta`, `out1` and `out2`; weight_dtype that of both weights.
+IB_EXPORT int ib_add_rmsnorm_pair(const float* x, const void* delta, float* x_out, const void* w1, const void* w2,
+                                  int weight_dtype, void* out1, void* out2, int act_dtype, int n_rows, int H, float eps,
+                                  void* stream) {
+    if (n_rows <= 0) return IB_OK;
+    if (H <= 0 || !x || !x_out || !w1 || !w2 || !out1 || !out2 || !(eps > 0.f)) return IB_ERR_BAD_ARG;
+    cudaStream_t s = (cudaStream_t)stream;
+    if (act_dtype == 0 && weight_dtype == 0)
+        return launch_rmsnorm_pair<float, float>(x, delta, x_out, w1, w2, out1, out2, n_rows, H, eps, s);
+    if (act_dtype == 1 && weight_dtype == 1)
+        return launch_rmsnorm_pair<bf16, bf16>(x, delta, x_out, w1, w2, out1, out2, n_rows, H, eps, s);
+    if (act_dtype == 1 && weight_dtype == 0)
+        return launch_rmsnorm_pair<bf16, float>(x, delta, x_out, w1, w2, out1, out2, n_rows, H, eps, s);
     return IB_ERR_UNSUPPORTED;
 }
 
@@ -494,23 +619,16 @@ IB_EXPORT int ib_rope_append(void* qkv, int act_dtype, int qkv_stride, const int
 // tcgen05 product holds gates and their ups).
 // ---------------------------------------------------------------------------
 // `act` chooses the activation of the gate: 0 = SiLU, g / (1 + exp(-g));
-// 1 = GELU in its tanh form, 0.5 g (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3))).
+// 1 = GELU in its tanh form, 0.5 g (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3))); 2 = clamped swish
+// (the codes of gate_times less one).  Rows of the output may lie `out_stride` apart.
 // With `scale` [N, n_scales] every output is also multiplied by
 // scale[row, i / cols_per_scale]: the outputs are those of n_scales experts
 // side by side and the scale is the weight the row's router gave each (0 for
 // an expert it did not choose).
-__device__ __forceinline__ float gate_act(float g, int act) {
-    if (act == 1) {
-        const float inner = 0.7978845608028654f * (g + 0.044715f * g * g * g);
-        return 0.5f * g * (1.f + tanhf(inner));
-    }
-    return g / (1.f + expf(-g));
-}
-
 template <typename T>
 __global__ void gated_act_kernel(const T* __restrict__ x, T* __restrict__ out, int I, int blk,
                                  size_t total, int act, const float* __restrict__ scale,
-                                 int cols_per_scale, int n_scales) {
+                                 int cols_per_scale, int n_scales, float limit, float alpha, int out_stride) {
     pdl_trigger();
     pdl_wait();
     size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -520,15 +638,16 @@ __global__ void gated_act_kernel(const T* __restrict__ x, T* __restrict__ out, i
     const size_t gi = row * 2 * I + (size_t)(i / blk) * 2 * blk + (i % blk);
     const float g = to_f32(x[gi]);
     const float u = to_f32(x[gi + blk]);
-    float y = gate_act(g, act) * u;
+    float y = gate_times(g, u, act + 1, limit, alpha);
     if (scale) y *= scale[row * n_scales + i / cols_per_scale];
-    out[idx] = from_f32<T>(y);
+    out[row * out_stride + i] = from_f32<T>(y);
 }
 
 // Eight outputs per thread with 16-byte loads and stores (I and blk multiples of 8).
 __global__ void gated_act_vec8_kernel(const bf16* __restrict__ x, bf16* __restrict__ out, int I,
                                       int blk, size_t total_vec, int act, const float* __restrict__ scale,
-                                      int cols_per_scale, int n_scales) {
+                                      int cols_per_scale, int n_scales, float limit, float alpha,
+                                      int out_stride) {
     pdl_trigger();
     pdl_wait();
     const size_t v = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -548,27 +667,28 @@ __global__ void gated_act_vec8_kernel(const bf16* __restrict__ x, bf16* __restri
 #pragma unroll
     for (int k = 0; k < 4; ++k) {
         const float2 g = __bfloat1622float2(g2[k]), u = __bfloat1622float2(u2[k]);
-        float a = gate_act(g.x, act) * u.x, b = gate_act(g.y, act) * u.y;
+        float a = gate_times(g.x, u.x, act + 1, limit, alpha), b = gate_times(g.y, u.y, act + 1, limit, alpha);
         if (scale) { a *= sc; b *= sc; }
         o2[k] = __floats2bfloat162_rn(a, b);
     }
-    *reinterpret_cast<uint4*>(out + row * I + i) = o4;
+    *reinterpret_cast<uint4*>(out + row * out_stride + i) = o4;
 }
 
-IB_EXPORT int ib_gated_act(const void* x, void* out, int act_dtype, int n_rows, int I, int blk, int act,
-                           const float* scale, int cols_per_scale, void* stream) {
+IB_EXPORT int ib_gated_act_strided(const void* x, void* out, int out_stride, int act_dtype, int n_rows, int I, int blk,
+                                   int act, float limit, float alpha, const float* scale, int cols_per_scale,
+                                   void* stream) {
     if (n_rows <= 0) return IB_OK;
-    if (!x || !out || I <= 0 || blk <= 0 || I % blk || act < 0 || act > 1) return IB_ERR_BAD_ARG;
+    if (!x || !out || I <= 0 || blk <= 0 || I % blk || act < 0 || act > 2 || out_stride < I) return IB_ERR_BAD_ARG;
     if (scale && (cols_per_scale <= 0 || I % cols_per_scale)) return IB_ERR_BAD_ARG;
     const int n_scales = scale ? I / cols_per_scale : 0;
     cudaStream_t s = (cudaStream_t)stream;
     const size_t total = (size_t)n_rows * I;
-    if (act_dtype == 1 && I % 8 == 0 && blk % 8 == 0 && (!scale || cols_per_scale % 8 == 0) &&
+    if (act_dtype == 1 && I % 8 == 0 && blk % 8 == 0 && out_stride % 8 == 0 && (!scale || cols_per_scale % 8 == 0) &&
         !(((uintptr_t)x | (uintptr_t)out) & 15)) {
         const size_t total_vec = total / 8;
         cudaError_t le = launch_kernel(gated_act_vec8_kernel, dim3((unsigned)((total_vec + 255) / 256)),
                                        dim3(256), 0, s, (const bf16*)x, (bf16*)out, I, blk, total_vec, act, scale,
-                                       cols_per_scale, n_scales);
+                                       cols_per_scale, n_scales, limit, alpha, out_stride);
         if (le != cudaSuccess) return (int)le;
         IB_LAUNCH_CHECK();
         return IB_OK;
@@ -577,18 +697,24 @@ IB_EXPORT int ib_gated_act(const void* x, void* out, int act_dtype, int n_rows, 
     if (act_dtype == 0) {
         cudaError_t le = launch_kernel(gated_act_kernel<float>, dim3(blocks), dim3(256), 0, s,
                                        (const float*)x, (float*)out, I, blk, total, act, scale, cols_per_scale,
-                                       n_scales);
+                                       n_scales, limit, alpha, out_stride);
         if (le != cudaSuccess) return (int)le;
     } else if (act_dtype == 1) {
         cudaError_t le = launch_kernel(gated_act_kernel<bf16>, dim3(blocks), dim3(256), 0, s,
                                        (const bf16*)x, (bf16*)out, I, blk, total, act, scale, cols_per_scale,
-                                       n_scales);
+                                       n_scales, limit, alpha, out_stride);
         if (le != cudaSuccess) return (int)le;
     } else {
         return IB_ERR_UNSUPPORTED;
     }
     IB_LAUNCH_CHECK();
     return IB_OK;
+}
+
+IB_EXPORT int ib_gated_act(const void* x, void* out, int act_dtype, int n_rows, int I, int blk, int act,
+                           const float* scale, int cols_per_scale, void* stream) {
+    if (act > 1) return IB_ERR_BAD_ARG;  // (the clamped activation comes with its limit)
+    return ib_gated_act_strided(x, out, I, act_dtype, n_rows, I, blk, act, 0.f, 0.f, scale, cols_per_scale, stream);
 }
 
 IB_EXPORT int ib_silu_mul(const void* x, void* out, int act_dtype, int n_rows, int I, int blk,

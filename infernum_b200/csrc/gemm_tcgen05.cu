@@ -186,7 +186,8 @@ struct GemmParams {
     int splits;           // slices of K = CTAs per cluster (1, 2, 4 or 8)
     int kblocks_per_split;
     int out_f32;
-    int swiglu;           // 1: W rows are 64 gates then their 64 ups per tile; out is [T, N/2]
+    float act_limit, act_alpha;  // of the clamped activation
+    int swiglu;           // gate_times' code: W rows are 64 gates then their 64 ups per tile; out is [T, N/2]
 };
 
 template <int BN>
@@ -345,11 +346,8 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w,
                         if (t < p.T) {
                             const float g = __uint_as_float(v[j]);
                             const float u = xch[(c + j) * 64 + row];
-                            // (swiglu 1: SiLU; 2: GELU in its tanh form)
-                            const float a = p.swiglu == 2
-                                ? 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)))
-                                : g / (1.f + expf(-g));
-                            ((bf16*)p.out)[(size_t)t * p.ldo + col] = __float2bfloat16_rn(a * u);
+                            ((bf16*)p.out)[(size_t)t * p.ldo + col] =
+                                __float2bfloat16_rn(gate_times(g, u, p.swiglu, p.act_limit, p.act_alpha));
                         }
                     }
                 }
@@ -558,12 +556,12 @@ IB_EXPORT int ib_gemm_tc_token_tile(int T) {
 
 // out[T, N] = X[T, K] . W[N, K]^T, bf16 operands, out bf16 (out_f32 = 0) or float32.
 // ldx, ldw, ldo: row strides in elements.  `splits` (1..8) cuts K over the
-// CTAs of a cluster.  swiglu = 1: W holds, per
+// CTAs of a cluster.  swiglu > 0 (gate_times' code; act_limit and act_alpha are those of code 3): W holds, per
 // 128 rows, 64 gate rows followed by their 64 up rows; out is [T, N / 2] bf16 with
-// out[t, 64 b + r] = silu(x . W[128 b + r]) * (x . W[128 b + 64 + r]); K is not split.
+// out[t, 64 b + r] = gate_times(x . W[128 b + r], x . W[128 b + 64 + r]); K is not split.
 IB_EXPORT int ib_gemm_tc(const void* x, int ldx, const void* w, int ldw, void* out, int ldo,
                          int out_f32, int T, int N, int K, int splits, int swiglu, unsigned* err,
-                         void* stream) {
+                         void* stream, float act_limit, float act_alpha) {
     if (T <= 0 || N <= 0) return IB_OK;
     if (!x || !w || !out || !err || K <= 0) return IB_ERR_BAD_ARG;
     // TMA: 16-byte aligned bases and row strides
@@ -589,6 +587,8 @@ IB_EXPORT int ib_gemm_tc(const void* x, int ldx, const void* w, int ldw, void* o
     p.splits = (kblocks + p.kblocks_per_split - 1) / p.kblocks_per_split;  // no empty slice
     p.out_f32 = out_f32;
     p.swiglu = swiglu;
+    p.act_limit = act_limit;
+    p.act_alpha = act_alpha;
     CUtensorMap mw, mx;
     int rc = make_map(&mw, w, N, K, ldw, BM);
     if (rc != IB_OK) return rc;

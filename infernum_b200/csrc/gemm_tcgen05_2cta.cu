@@ -141,15 +141,6 @@ __device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
     __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
     return *reinterpret_cast<unsigned*>(&v);
 }
-// The formula of the other SwiGLU kernels of this package, in float32.
-__device__ __forceinline__ float silu_times(float g, float u) { return g / (1.f + expf(-g)) * u; }
-// The gate's activation times up: act 1 = SiLU, 2 = GELU in its tanh form (the formulas of
-// the stand-alone activation kernel).
-__device__ __forceinline__ float gate_times(float g, float u, int act) {
-    if (act == 2) return 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
-    return silu_times(g, u);
-}
-
 // Sixteen values of a token's row, bf16, at out[col .. col+16); `limit` ends the row.
 __device__ __forceinline__ void store16(bf16* row, int col, int limit, const float (&v)[16]) {
     if (col + 16 <= limit) {
@@ -172,7 +163,8 @@ struct Params {
     bf16* out;
     unsigned* err;
     int T, N, K, ldo;
-    int act;  // with the gated epilogue: 1 = SiLU, 2 = GELU (tanh form)
+    int act;  // with the gated epilogue: gate_times' code
+    float act_limit, act_alpha;
     const float* scale;   // with the gated epilogue, optional [T, n_scales]: out[t, c] *= scale[t, c / cols_per_scale]
     int n_scales, cols_per_scale;   // (experts side by side and the weight a token's router gave each; 16 | cols_per_scale)
     int t_tiles;   // token tiles of 256
@@ -347,7 +339,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constan
                                              ? p.scale[(size_t)gt * p.n_scales + col / p.cols_per_scale] : 1.f;
 #pragma unroll
                         for (int q = 0; q < 16; ++q)
-                            v[q] = gate_times(__uint_as_float(g[q]), __uint_as_float(u[q]), p.act) * sc;
+                            v[q] = gate_times(__uint_as_float(g[q]), __uint_as_float(u[q]), p.act, p.act_limit, p.act_alpha) * sc;
                         if (live) store16(row, col, limit, v);
                     }
                 }
@@ -455,11 +447,13 @@ int launch_pair(const CUtensorMap& mx, const CUtensorMap& mw, const CUtensorMap&
 // that walk over them.  The weight rows are cut into `cols_a` columns of `bn_a`
 // rows and the rest into columns of `bn_b` rows (multiples of 16 from 32 to 256; of
 // 128 with `swiglu`).
+// `swiglu` names the activation (gate_times' codes; act_limit and act_alpha are those of code 3).
 // `scale` (with `swiglu` only; float32 [T, (N/2) / cols_per_scale], or null): every output is also
 // multiplied by scale[t, column / cols_per_scale] (cols_per_scale a multiple of 16 that divides N/2).
 IB_EXPORT int ib_gemm_pair_scaled(const void* x, int ldx, const void* w, int ldw, void* out, int ldo, int T, int N,
                                   int K, int swiglu, int bn_a, int cols_a, int bn_b, int t_group, int sm_count,
-                                  const float* scale, int cols_per_scale, unsigned* err, void* stream) {
+                                  const float* scale, int cols_per_scale, unsigned* err, void* stream, float act_limit,
+                                  float act_alpha) {
     if (T <= 0 || N <= 0) return IB_OK;
     if (scale && (!swiglu || cols_per_scale <= 0 || cols_per_scale % 16 || (N / 2) % cols_per_scale))
         return IB_ERR_BAD_ARG;
@@ -478,6 +472,8 @@ IB_EXPORT int ib_gemm_pair_scaled(const void* x, int ldx, const void* w, int ldw
     p.K = K;
     p.ldo = ldo;
     p.act = swiglu;
+    p.act_limit = act_limit;
+    p.act_alpha = act_alpha;
     p.scale = scale;
     p.cols_per_scale = scale ? cols_per_scale : 1;
     p.n_scales = scale ? (N / 2) / cols_per_scale : 0;
@@ -509,5 +505,5 @@ IB_EXPORT int ib_gemm_pair(const void* x, int ldx, const void* w, int ldw, void*
                            int K, int swiglu, int bn_a, int cols_a, int bn_b, int t_group, int sm_count,
                            unsigned* err, void* stream) {
     return ib_gemm_pair_scaled(x, ldx, w, ldw, out, ldo, T, N, K, swiglu, bn_a, cols_a, bn_b, t_group, sm_count,
-                               nullptr, 0, err, stream);
+                               nullptr, 0, err, stream, 0.f, 0.f);
 }

@@ -370,3 +370,37 @@ IB_EXPORT int ib_add_row(float* x, const float* v, int n_rows, int W, void* stre
     IB_LAUNCH_CHECK();
     return IB_OK;
 }
+
+// The stream where a pass over a run of layers begins: out[n] = x[n] (+ delta[n]) (+ origin[n]) + v, all sums in
+// 32-bit in that order; `out` may be `x`.
+template <typename TD>
+__global__ void reenter_add_kernel(const float* x, const TD* __restrict__ delta, const float* origin,
+                                   const float* __restrict__ v, float* out, int W) {
+    pdl_trigger();
+    pdl_wait();
+    const size_t at = (size_t)blockIdx.x * W;
+    for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < W; i += gridDim.y * blockDim.x) {
+        float a = x[at + i];
+        if (delta) a += to_f32(delta[at + i]);
+        if (origin) a += origin[at + i];
+        out[at + i] = a + v[i];
+    }
+}
+
+IB_EXPORT int ib_reenter_add(const float* x, const void* delta, int act_dtype, const float* origin, const float* v,
+                             float* out, int n_rows, int W, void* stream) {
+    if (n_rows <= 0) return IB_OK;
+    if (!x || !v || !out || W <= 0) return IB_ERR_BAD_ARG;
+    cudaStream_t s = (cudaStream_t)stream;
+    const dim3 grid(n_rows, (W + 1023) / 1024), block(256);
+    cudaError_t le;
+    if (act_dtype == 0)
+        le = launch_kernel(reenter_add_kernel<float>, grid, block, 0, s, x, (const float*)delta, origin, v, out, W);
+    else if (act_dtype == 1)
+        le = launch_kernel(reenter_add_kernel<bf16>, grid, block, 0, s, x, (const bf16*)delta, origin, v, out, W);
+    else
+        return IB_ERR_UNSUPPORTED;
+    if (le != cudaSuccess) return (int)le;
+    IB_LAUNCH_CHECK();
+    return IB_OK;
+}

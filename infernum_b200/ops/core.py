@@ -18,7 +18,7 @@ from ..errors import KernelError
 
 CORE_SOURCES = ["elementwise.cu", "attention_plain.cu", "gemm_plain.cu", "sampling.cu", "layernorm.cu",
                 "embed_hashed.cu", "latent.cu", "moe.cu", "hyper.cu", "recurrent.cu", "subnorm.cu", "shortconv.cu",
-                "attention_diff.cu"]
+                "attention_diff.cu", "attention_talk.cu"]
 
 _c_int = ctypes.c_int
 _c_float = ctypes.c_float
@@ -178,6 +178,24 @@ def core_lib() -> ctypes.CDLL:
         for fn in ("ib_latent_prepare_ex", "ib_latent_q_rotate_ex", "ib_moe_route_softmax_all", "ib_moe_combine",
                    "ib_gated_norm_add", "ib_concat_round", "ib_add_row", "ib_causal_conv", "ib_conv_state_update",
                    "ib_conv_rope_append", "ib_attention_diff"):
+            getattr(lib, fn).restype = _c_int
+        lib.ib_embed_scaled.argtypes = [_c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_float,
+                                        _c_void_p, _c_void_p]
+        lib.ib_gated_act_strided.argtypes = [_c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
+                                             _c_float, _c_float, _c_void_p, _c_int, _c_void_p]
+        lib.ib_add_rmsnorm_pair.argtypes = [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p,
+                                            _c_void_p, _c_int, _c_int, _c_int, _c_float, _c_void_p]
+        lib.ib_reenter_add.argtypes = [_c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int,
+                                       _c_void_p]
+        lib.ib_qk_row_norm_append.argtypes = [_c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_float, _c_void_p, _c_int,
+                                              _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_int,
+                                              _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p]
+        lib.ib_attention_talk.argtypes = [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_void_p,
+                                          _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int,
+                                          _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int,
+                                          _c_void_p, _c_void_p]
+        for fn in ("ib_embed_scaled", "ib_gated_act_strided", "ib_add_rmsnorm_pair", "ib_reenter_add",
+                   "ib_qk_row_norm_append", "ib_attention_talk"):
             getattr(lib, fn).restype = _c_int
         for fn in ("ib_decode_advance", "ib_feed_tokens", "ib_embed", "ib_add_rmsnorm", "ib_residual_add", "ib_rope_append",
                    "ib_silu_mul", "ib_attention_plain", "ib_gemm_plain", "ib_argmax", "ib_sample"):
@@ -361,8 +379,8 @@ def step_fence(device) -> None:
     check(core_lib().ib_step_fence(torch.cuda.current_stream(device).cuda_stream), "step_fence")
 
 
-def embed(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor, err: torch.Tensor) -> None:
-    """out[t, :] = table[ids[t], :] into a float32 residual stream."""
+def embed(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor, err: torch.Tensor, scale: float = 1.0) -> None:
+    """out[t, :] = table[ids[t], :] * scale into a float32 residual stream."""
     require_cuda(ids, table, out, err)
     _int32(ids, "ids")
     n = ids.numel()
@@ -371,8 +389,8 @@ def embed(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor, err: torch.
         raise KernelError(f"embed: out must be contiguous float32 [{n}, {H}]")
     if not table.is_contiguous():
         raise KernelError("embed: table must be contiguous")
-    check(core_lib().ib_embed(ids.data_ptr(), table.data_ptr(), dtype_code(table.dtype),
-                              out.data_ptr(), n, H, V, err.data_ptr(), stream_ptr(out)), "embed")
+    check(core_lib().ib_embed_scaled(ids.data_ptr(), table.data_ptr(), dtype_code(table.dtype), out.data_ptr(), n, H, V,
+                                     float(scale), err.data_ptr(), stream_ptr(out)), "embed")
 
 
 def add_rmsnorm(residual: torch.Tensor, delta: Optional[torch.Tensor], weight: torch.Tensor,
@@ -616,7 +634,7 @@ def decode_advance(tokens: torch.Tensor, selected: Optional[torch.Tensor], posit
 # SiLU, a soft cap on logits, a hashed bigram embedding, attention over a latent
 # cache, batched per-head products, and the routing of a mixture of experts.
 # ---------------------------------------------------------------------------
-ACTIVATIONS = {"silu": 0, "gelu_tanh": 1}
+ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "clamped_swish": 2}
 
 
 def scale_add_norm(residual: torch.Tensor, delta: Optional[torch.Tensor], weight: torch.Tensor,
@@ -657,15 +675,18 @@ def softcap(logits: torch.Tensor, cap: float) -> None:
 
 
 def gated_act(gate_up: torch.Tensor, out: torch.Tensor, activation: str = "silu", block: Optional[int] = None,
-              scale: Optional[torch.Tensor] = None, cols_per_scale: int = 0) -> None:
+              scale: Optional[torch.Tensor] = None, cols_per_scale: int = 0, limit: float = float("inf"),
+              alpha: float = 1.0) -> None:
     """out = act(gate) * up for rows [N, 2I] (``block`` as in ``silu_mul``); with
     ``scale`` [N, I / cols_per_scale] (float32) each run of ``cols_per_scale``
-    outputs is multiplied by its scale."""
+    outputs is multiplied by its scale.  ``clamped_swish`` is ``g' sigmoid(alpha g') (u' + 1)``
+    with ``g' = min(g, limit)`` and ``u'`` the up held to [-limit, limit].  The rows of
+    ``out`` may lie in wider ones."""
     require_cuda(gate_up, out, scale)
     N, two_i = gate_up.shape
     if two_i % 2 or out.shape != (N, two_i // 2) or out.dtype != gate_up.dtype \
-            or not gate_up.is_contiguous() or not out.is_contiguous():
-        raise KernelError("gated_act: gate_up [N, 2I] and out [N, I] must be contiguous, same dtype")
+            or not gate_up.is_contiguous() or out.stride(1) != 1:
+        raise KernelError("gated_act: gate_up [N, 2I] contiguous, out [N, I] with unit inner stride, same dtype")
     I = two_i // 2
     blk = I if block is None else int(block)
     if blk <= 0 or I % blk:
@@ -675,9 +696,9 @@ def gated_act(gate_up: torch.Tensor, out: torch.Tensor, activation: str = "silu"
     if scale is not None and (scale.dtype != torch.float32 or not scale.is_contiguous() or cols_per_scale <= 0
                               or I % cols_per_scale or scale.shape != (N, I // cols_per_scale)):
         raise KernelError("gated_act: scale must be contiguous float32 [N, I / cols_per_scale]")
-    check(core_lib().ib_gated_act(gate_up.data_ptr(), out.data_ptr(), dtype_code(out.dtype), N, I, blk,
-                                  ACTIVATIONS[activation], _ptr(scale), int(cols_per_scale), stream_ptr(out)),
-          "gated_act")
+    check(core_lib().ib_gated_act_strided(gate_up.data_ptr(), out.data_ptr(), out.stride(0), dtype_code(out.dtype), N, I,
+                                          blk, ACTIVATIONS[activation], float(limit), float(alpha), _ptr(scale),
+                                          int(cols_per_scale), stream_ptr(out)), "gated_act")
 
 
 def embed_hashed(ctx, prev_state: torch.Tensor, table: torch.Tensor, bigram: torch.Tensor, buckets: int,
@@ -1337,3 +1358,113 @@ def moe_combine(routed: Optional[torch.Tensor], h: torch.Tensor, shared: Optiona
         raise KernelError("moe_combine: extra must be contiguous float32 [N, 2]")
     check(core_lib().ib_moe_combine(_ptr(routed), h.data_ptr(), h.stride(0), _ptr(shared), extra.data_ptr(), out.data_ptr(),
                                     dtype_code(out.dtype), N, W, stream_ptr(out)), "moe_combine")
+
+
+# ---------------------------------------------------------------------------
+# Layers whose two sub-layers read one sum, passes that begin with sums, attention
+# whose heads exchange their scores.
+# ---------------------------------------------------------------------------
+def add_rmsnorm_pair(x: torch.Tensor, delta: Optional[torch.Tensor], x_out: torch.Tensor, w1: torch.Tensor,
+                     w2: torch.Tensor, eps: float, out1: torch.Tensor, out2: torch.Tensor) -> None:
+    """x_out = x + delta (``x_out`` may be ``x``); out1, out2 = its RMS norm times ``w1``, ``w2``, in 32-bit."""
+    require_cuda(x, delta, x_out, w1, w2, out1, out2)
+    N, H = x.shape
+    for t in (x, x_out):
+        if t.dtype != torch.float32 or t.shape != (N, H) or not t.is_contiguous():
+            raise KernelError("add_rmsnorm_pair: x and x_out must be contiguous float32 [N, H]")
+    for t in (out1, out2, delta):
+        if t is not None and (t.shape != (N, H) or t.dtype != out1.dtype or not t.is_contiguous()):
+            raise KernelError("add_rmsnorm_pair: delta and the outputs must be contiguous [N, H] of one dtype")
+    for w in (w1, w2):
+        if w.shape != (H,) or w.dtype != w1.dtype or not w.is_contiguous():
+            raise KernelError("add_rmsnorm_pair: the weights must be contiguous [H] of one dtype")
+    check(core_lib().ib_add_rmsnorm_pair(x.data_ptr(), _ptr(delta), x_out.data_ptr(), w1.data_ptr(), w2.data_ptr(),
+                                         dtype_code(w1.dtype), out1.data_ptr(), out2.data_ptr(), dtype_code(out1.dtype),
+                                         N, H, float(eps), stream_ptr(x)), "add_rmsnorm_pair")
+
+
+def reenter_add(x: torch.Tensor, delta: Optional[torch.Tensor], origin: Optional[torch.Tensor], v: torch.Tensor,
+                out: torch.Tensor) -> None:
+    """out[n] = x[n] (+ delta[n]) (+ origin[n]) + v in 32-bit; ``out`` may be ``x``."""
+    require_cuda(x, delta, origin, v, out)
+    N, W = x.shape
+    for t in (x, origin, out):
+        if t is not None and (t.dtype != torch.float32 or t.shape != (N, W) or not t.is_contiguous()):
+            raise KernelError("reenter_add: x, origin and out must be contiguous float32 [N, W]")
+    if delta is not None and (delta.shape != (N, W) or not delta.is_contiguous()):
+        raise KernelError("reenter_add: delta must be contiguous [N, W]")
+    _f32_vec(v, W, "reenter_add: v")
+    check(core_lib().ib_reenter_add(x.data_ptr(), _ptr(delta), dtype_code(delta.dtype) if delta is not None else 0,
+                                    _ptr(origin), v.data_ptr(), out.data_ptr(), N, W, stream_ptr(x)), "reenter_add")
+
+
+def qk_row_norm_append(x: torch.Tensor, q_weight: Optional[torch.Tensor], k_weight: Optional[torch.Tensor], eps: float,
+                       inv_freq: Optional[torch.Tensor], rotary_dim: int, n_heads: int, n_kv_heads: int, dim: int,
+                       vdim: int, positions: torch.Tensor, row_entry: torch.Tensor, block_tables: torch.Tensor,
+                       k_pool: torch.Tensor, v_pool: torch.Tensor, err: torch.Tensor) -> None:
+    """Rows of ``x``: ``n_heads`` queries and ``n_kv_heads`` keys of ``dim``, ``n_kv_heads`` values of ``vdim``.
+    All of a row's queries are divided by their one root mean square and multiplied by ``q_weight``
+    (float32 [n_heads * dim]; None: neither), its keys likewise; the first ``rotary_dim`` dimensions of
+    every head are rotated (halves paired).  Queries are written back, keys and values to their pages."""
+    require_cuda(x, q_weight, k_weight, inv_freq, positions, row_entry, block_tables, k_pool, v_pool, err)
+    _int32(positions, "positions")
+    _int32(row_entry, "row_entry")
+    _int32(block_tables, "block_tables")
+    _f32_vec(q_weight, n_heads * dim, "qk_row_norm_append: q_weight")
+    _f32_vec(k_weight, n_kv_heads * dim, "qk_row_norm_append: k_weight")
+    num_pages, nkv_pool, page_size, d_pool = k_pool.shape
+    if x.dim() != 2 or x.stride(1) != 1 or x.shape[1] < (n_heads + n_kv_heads) * dim + n_kv_heads * vdim:
+        raise KernelError("qk_row_norm_append: x rows must hold queries, keys and values with unit inner stride")
+    if nkv_pool != n_kv_heads or d_pool != dim or v_pool.shape != (num_pages, n_kv_heads, page_size, vdim) \
+            or k_pool.dtype != x.dtype or v_pool.dtype != x.dtype or not k_pool.is_contiguous() \
+            or not v_pool.is_contiguous():
+        raise KernelError("qk_row_norm_append: pools must be contiguous [pages, kv_heads, page_size, dim | vdim] of x's dtype")
+    if rotary_dim:
+        _f32_vec(inv_freq, rotary_dim // 2, "qk_row_norm_append: inv_freq")
+        if inv_freq is None:
+            raise KernelError("qk_row_norm_append: a rotation needs its frequencies")
+    check(core_lib().ib_qk_row_norm_append(x.data_ptr(), x.stride(0), dtype_code(x.dtype), _ptr(q_weight), _ptr(k_weight),
+                                           float(eps), _ptr(inv_freq), int(rotary_dim), positions.data_ptr(),
+                                           row_entry.data_ptr(), block_tables.data_ptr(), block_tables.shape[1],
+                                           k_pool.data_ptr(), v_pool.data_ptr(), x.shape[0], n_heads, n_kv_heads, dim,
+                                           vdim, page_size, num_pages, err.data_ptr(), stream_ptr(x)),
+          "qk_row_norm_append")
+
+
+def attention_talk(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, out: torch.Tensor, ctx,
+                   block_tables: torch.Tensor, n_heads: int, scale: float, talk: Optional[torch.Tensor],
+                   temp: Optional[torch.Tensor], gate: Optional[torch.Tensor], chunk: int, window: int,
+                   err: torch.Tensor) -> None:
+    """Attention whose heads exchange their scores before the softmax: head h's score is
+    ``sum_g talk[h, g] temp[g] scale (q_g . k)`` over all heads (``talk`` float32 [H, H]; None: its own).
+    Query i sees keys j <= i, with ``chunk`` those of its own run of ``chunk`` positions, with ``window`` the
+    last ``window``.  ``gate`` [N, H] (a view of wider rows is fine): a head's result is multiplied by its
+    sigmoid.  ``q`` rows begin with the queries; ``out`` [N, H * vdim] may be a view of wider rows.  32-bit."""
+    require_cuda(q, k_pool, v_pool, out, talk, temp, gate, block_tables, err)
+    check_talk_arguments(q, k_pool, v_pool, out, block_tables, n_heads, talk, temp, gate)
+    num_pages, nkv, page_size, dim = k_pool.shape
+    check(core_lib().ib_attention_talk(q.data_ptr(), q.stride(0), k_pool.data_ptr(), v_pool.data_ptr(), out.data_ptr(),
+                                       out.stride(0), dtype_code(q.dtype), _ptr(talk), _ptr(temp), _ptr(gate),
+                                       gate.stride(0) if gate is not None else 0, ctx.positions.data_ptr(),
+                                       ctx.row_entry.data_ptr(), block_tables.data_ptr(), block_tables.shape[1],
+                                       q.shape[0], n_heads, nkv, dim, v_pool.shape[3], page_size, num_pages,
+                                       float(scale), int(chunk), int(window), err.data_ptr(), stream_ptr(q)),
+          "attention_talk")
+
+
+def check_talk_arguments(q, k_pool, v_pool, out, block_tables, n_heads, talk, temp, gate) -> None:
+    """What both forms of ``attention_talk`` ask of their tensors."""
+    _int32(block_tables, "block_tables")
+    N = q.shape[0]
+    num_pages, nkv, page_size, dim = k_pool.shape
+    vdim = v_pool.shape[3]
+    if q.dim() != 2 or q.stride(1) != 1 or q.shape[1] < n_heads * dim or out.shape != (N, n_heads * vdim) \
+            or out.stride(1) != 1 or v_pool.shape[:3] != k_pool.shape[:3] or not k_pool.is_contiguous() \
+            or not v_pool.is_contiguous() or not (q.dtype == k_pool.dtype == v_pool.dtype == out.dtype) \
+            or n_heads % nkv:
+        raise KernelError("attention_talk: q rows [heads * dim ...], out [N, heads * vdim] and the pools do not fit")
+    if talk is not None and (talk.dtype != torch.float32 or talk.shape != (n_heads, n_heads) or not talk.is_contiguous()):
+        raise KernelError("attention_talk: talk must be contiguous float32 [heads, heads]")
+    _f32_vec(temp, n_heads, "attention_talk: temp")
+    if gate is not None and (gate.shape != (N, n_heads) or gate.stride(1) != 1 or gate.dtype != q.dtype):
+        raise KernelError("attention_talk: gate must be [N, heads] of q's dtype with unit inner stride")

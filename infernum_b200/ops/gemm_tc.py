@@ -23,7 +23,7 @@ from ..csrc.build import load_module
 from ..errors import KernelError
 from . import core
 
-_c_int, _c_void_p, _c_ll = ctypes.c_int, ctypes.c_void_p, ctypes.c_longlong
+_c_int, _c_void_p, _c_ll, _c_float = ctypes.c_int, ctypes.c_void_p, ctypes.c_longlong, ctypes.c_float
 _lib: Optional[ctypes.CDLL] = None
 _pair_lib: Optional[ctypes.CDLL] = None
 _workspaces: Dict[torch.device, dict] = {}
@@ -31,7 +31,7 @@ _workspaces: Dict[torch.device, dict] = {}
 BM, BK = 128, 64
 # the gate's activation in a fused epilogue, as the kernels number them (0: no gated epilogue;
 # ``swiglu=True`` in the calls below is SiLU)
-GATE_CODES = {"silu": 1, "gelu_tanh": 2}
+GATE_CODES = {"silu": 1, "gelu_tanh": 2, "clamped_swish": 3}
 # What a tile of gemm_pair costs beside its width, in weight rows: its token half is
 # fetched and its prologue and epilogue run whatever the width.
 PAIR_TILE_OVERHEAD = 66
@@ -61,7 +61,7 @@ def lib() -> ctypes.CDLL:
     if _lib is None:
         l = load_module("gemm_tc", ["gemm_tcgen05.cu"])
         l.ib_gemm_tc.argtypes = [_c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_int,
-                                 _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p]
+                                 _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_float, _c_float]
         l.ib_gemm_tc.restype = _c_int
         l.ib_gemm_tc_token_tile.argtypes = [_c_int]
         l.ib_gemm_tc_token_tile.restype = _c_int
@@ -82,7 +82,7 @@ def pair_lib() -> ctypes.CDLL:
         l.ib_gemm_pair.restype = _c_int
         l.ib_gemm_pair_scaled.argtypes = [_c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_int,
                                           _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p,
-                                          _c_int, _c_void_p, _c_void_p]
+                                          _c_int, _c_void_p, _c_void_p, _c_float, _c_float]
         l.ib_gemm_pair_scaled.restype = _c_int
         lib()  # the SM count
         _pair_lib = l
@@ -126,10 +126,12 @@ def eligible(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> bool:
 
 
 def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, splits: Optional[int] = None,
-            err: Optional[torch.Tensor] = None, swiglu: bool = False) -> None:
+            err: Optional[torch.Tensor] = None, swiglu: bool = False, act_limit: float = 0.0,
+            act_alpha: float = 0.0) -> None:
     """Runs the tcgen05 kernel; raises KernelError if the operands do not fit it.
     ``swiglu``: ``w`` holds, per 128 rows, 64 gate rows then their 64 up rows, and
-    ``out`` [T, N/2] receives silu(gate) * up (at most 64 tokens)."""
+    ``out`` [T, N/2] receives silu(gate) * up (at most 64 tokens); a code of ``GATE_CODES`` names another
+    activation (``act_limit`` and ``act_alpha`` are the clamped one's)."""
     core.require_cuda(x, w, out)
     T, K = x.shape
     N = w.shape[0]
@@ -138,7 +140,7 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, splits: Optiona
     code = lib().ib_gemm_tc(x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(),
                             out.stride(0), 1 if out.dtype == torch.float32 else 0, T, N, K, splits,
                             int(swiglu), (err if err is not None else _error_word(x.device)).data_ptr(),
-                            core.stream_ptr(x))
+                            core.stream_ptr(x), float(act_limit), float(act_alpha))
     core.check(code, "gemm_tc")
 
 
@@ -193,7 +195,8 @@ def choose_token_group(T: int, K: int) -> int:
 def gemm_pair(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor,
               err: Optional[torch.Tensor] = None, swiglu: bool = False,
               tiling: Optional[Tuple[int, int, int]] = None, token_group: Optional[int] = None,
-              scale: Optional[torch.Tensor] = None, cols_per_scale: int = 0) -> None:
+              scale: Optional[torch.Tensor] = None, cols_per_scale: int = 0, act_limit: float = 0.0,
+              act_alpha: float = 0.0) -> None:
     """The product for many tokens: tiles of 256 tokens x up to 256 weight rows,
     each computed by two SMs as one (tcgen05 ``cta_group::2``); bf16 out.
     ``swiglu`` as in ``gemm_tc``, for any number of tokens.  ``scale`` (with
@@ -216,7 +219,7 @@ def gemm_pair(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor,
                                           token_group or choose_token_group(T, K), POLICY["sm_count"],
                                           scale.data_ptr() if scale is not None else None, int(cols_per_scale),
                                           (err if err is not None else _error_word(x.device)).data_ptr(),
-                                          core.stream_ptr(x))
+                                          core.stream_ptr(x), float(act_limit), float(act_alpha))
     core.check(code, "gemm_pair")
 
 
@@ -243,7 +246,8 @@ def route(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, err: Optional[tor
 
 def swiglu_route(x: torch.Tensor, w_interleaved: torch.Tensor, out: torch.Tensor,
                  err: Optional[torch.Tensor] = None, activation: str = "silu",
-                 scale: Optional[torch.Tensor] = None, cols_per_scale: int = 0) -> bool:
+                 scale: Optional[torch.Tensor] = None, cols_per_scale: int = 0, act_limit: float = 0.0,
+                 act_alpha: float = 0.0) -> bool:
     """The gate/up product with SiLU(gate) * up applied in its epilogue, when
     the policy and the operands allow; ``out`` is [T, I].  Up to 64 tokens go to
     the kernel that streams the weights once (decode), prompts to the kernel on
@@ -263,10 +267,11 @@ def swiglu_route(x: torch.Tensor, w_interleaved: torch.Tensor, out: torch.Tensor
     if T <= min(POLICY["max_tokens"], 64):
         if scale is not None:
             return False
-        gemm_tc(x, w_interleaved, out, splits=1, swiglu=code, err=err)
+        gemm_tc(x, w_interleaved, out, splits=1, swiglu=code, err=err, act_limit=act_limit, act_alpha=act_alpha)
         return True
     if pair_suits(T, fused_activation=True):
-        gemm_pair(x, w_interleaved, out, swiglu=code, err=err, scale=scale, cols_per_scale=cols_per_scale)
+        gemm_pair(x, w_interleaved, out, swiglu=code, err=err, scale=scale, cols_per_scale=cols_per_scale,
+                  act_limit=act_limit, act_alpha=act_alpha)
         return True
     return False
 

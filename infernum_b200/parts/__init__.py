@@ -7,4 +7,4 @@ from .base import (BLOCKS, EMBEDDINGS, ENTRIES, FEED_FORWARDS, HEADS, MIXERS, NO
                    WeightSpec, build_layer, register_block, register_feed_forward, register_mixer,
                    register_norm, register_position_encoding)
 from . import (attention, block, diff_attention, embedding, latent_attention, mlp, moe, norm, parallel, recurrent,  # noqa: F401  (registration)
-               reentry, rope)
+               reentry, rope, talking_attention)

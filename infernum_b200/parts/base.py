@@ -123,13 +123,16 @@ class PagedCacheSpec:
     the mixer keeps no values of their own (a latent cache, where keys and
     values are made from the one cached vector): only the key pool exists.
     ``keep_first`` (with a window): the first so many tokens of a request stay
-    visible however far back they lie, so the pages that hold them are kept."""
+    visible however far back they lie, so the pages that hold them are kept.
+    ``chunk`` > 0: a query reads only tokens of its own run of ``chunk`` positions
+    (counted from position 0), so pages of earlier runs can be given back."""
 
     kv_heads: int
     head_dim: int
     window: int = 0
     v_head_dim: Optional[int] = None
     keep_first: int = 0
+    chunk: int = 0
 
     @property
     def value_dim(self) -> int:
@@ -340,10 +343,16 @@ class ResidualStream:
         self.pending = delta
         self.pending_write = write
 
+    def own(self) -> None:
+        """Makes the residual one that may be written over: a copy, when it still is the embedding's output."""
+        if self.origin is not None and self.origin.data_ptr() == self.residual.data_ptr():
+            self.residual = self.residual.clone()
+
     def flush(self) -> None:
         if self.pending is not None:
             from ..ops import core
 
+            self.own()
             if self.pending_write is not None:
                 mix, out_coef = self.pending_write
                 core.hc_norm(self.residual, self.pending, mix, out_coef, None, None, None, 1.0, None)

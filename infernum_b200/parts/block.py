@@ -25,6 +25,9 @@ of the embedding's output and all layers' results so far.
 ``x <- x + mult * norm1b(g1 * mixer(c1(norm1(x))))``, then the same with ``ffn``;
 ``c`` adds a short causal convolution of the normed rows to them, ``g`` is a
 sigmoid gate computed from the normed rows.
+
+``parallel_prenorm``: mixer and feed-forward side by side, ``x <- x +
+(mixer(norm1(x)) + ffn(norm2(x)))``, both of the same x.
 """
 
 from __future__ import annotations
@@ -277,3 +280,63 @@ class SandwichBlock(Block):
                 core.conv_state_update(h, self.taps, state, off, ctx)
             y = p[role].forward(u, ctx, cache) if role == "mixer" else p[role].forward(u, ctx)
             p[post].add_gated(stream, y, g, gate[1] if gate is not None else None, self.mult)
+
+
+@BLOCKS.register("parallel_prenorm")
+class ParallelPreNormBlock(Block):
+    """``x <- x + (mixer(norm1(x)) + ffn(norm2(x)))``.  The sum into x is pending on the
+    stream until the next norm folds it in.
+
+    Two RMS norms of one eps are one kernel (``forward_pair``).  When mixer and
+    feed-forward both end in a plain product and can hand over what it reads
+    (``forward_hidden`` and ``out_proj``), the two products are one: the rows
+    ``[mixer's | feed-forward's]`` times the two weights side by side, whose one
+    32-bit accumulator holds the sum.
+
+    Parts: ``norm1``, ``mixer``, and optionally ``ffn`` with ``norm2`` (a ``norm2``
+    without a feed-forward is not used).
+    """
+
+    def __init__(self, params, rt, parts):
+        super().__init__(params, rt, parts)
+        missing = [r for r in ("norm1", "mixer") if r not in parts]
+        if "ffn" in parts and "norm2" not in parts:
+            missing.append("norm2")
+        if missing:
+            raise ConfigError(f"parallel_prenorm block {params.get('name', '')!r} lacks parts {missing}")
+        self.joint = None
+
+    def bind(self, weights) -> None:
+        super().bind(weights)
+        ends = [getattr(self.parts.get(r), "out_proj", None) for r in ("mixer", "ffn")]
+        if any(e is None or not hasattr(self.parts[r], "forward_hidden") for e, r in zip(ends, ("mixer", "ffn"))):
+            return
+        a, b = ends
+        if a.weight.dtype != b.weight.dtype or a.weight.shape[1] % 8 or b.weight.shape[1] % 8:
+            return
+        # the parts keep views of the joint weight, so nothing is held twice
+        self.joint = Linear(torch.cat([a.weight, b.weight], dim=1), self.rt)
+        k = a.weight.shape[1]
+        a.weight, b.weight = self.joint.weight[:, :k], self.joint.weight[:, k:]
+
+    def forward(self, stream: ResidualStream, ctx, cache) -> None:
+        p = self.parts
+        mixer, ffn, norm1 = p["mixer"], p.get("ffn"), p["norm1"]
+        if ffn is None:
+            stream.push(mixer.forward(norm1.forward(stream), ctx, cache))
+            return
+        if hasattr(norm1, "forward_pair") and norm1.pairs_with(p["norm2"]):
+            h1, h2 = norm1.forward_pair(stream, p["norm2"])
+        else:
+            h1 = norm1.forward(stream)
+            h2 = p["norm2"].forward(stream)  # (nothing is pending any more: the same sum)
+        if self.joint is not None:
+            k = mixer.out_proj.weight.shape[1]
+            rows = torch.empty((h1.shape[0], self.joint.weight.shape[1]), dtype=h1.dtype, device=h1.device)
+            mixer.forward_hidden(h1, ctx, cache, rows[:, :k])
+            ffn.forward_hidden(h2, ctx, rows[:, k:])
+            stream.push(self.joint(rows))
+            return
+        y = mixer.forward(h1, ctx, cache)
+        core.pointwise(y, ffn.forward(h2, ctx), "axpby", 1.0, 1.0)
+        stream.push(y)

@@ -1,6 +1,6 @@
 """Token embedding and output head.
 
-Embedding: ``h[t, :] = E[id_t, :]`` with no scaling
+Embedding: ``h[t, :] = E[id_t, :]``, unscaled unless a model asks for a factor
 (infernum-llama/src/graph_builder.rs:442; infernum-cuda/kernels/embed.cu:36-50),
 written straight into the float32 residual stream.
 
@@ -32,7 +32,8 @@ class TokenEmbedding(Embedding):
     for layers that hand on a weighted sum of them); ``norm`` (a norm spec {"kind",
     "params"} with ``apply_f32``: the looked-up rows are normed, in 32-bit, before
     they become the stream); ``keep_origin`` (True: the stream keeps the embedding's
-    output, as this part leaves it, in ``stream.origin``)."""
+    output, as this part leaves it, in ``stream.origin``); ``scale`` (the rows are
+    multiplied by it as they are looked up; not together with ``act`` or ``result_slots``)."""
 
     def __init__(self, params, rt: Runtime):
         super().__init__(params, rt)
@@ -42,6 +43,9 @@ class TokenEmbedding(Embedding):
         self.with_act = bool(params.get("act", False))
         self.result_slots = int(params.get("result_slots") or 0)
         self.keep_origin = bool(params.get("keep_origin", False))
+        self.scale = float(params.get("scale", 1.0))
+        if self.scale != 1.0 and (self.with_act or self.result_slots):
+            raise ConfigError("token embedding: a scaled embedding keeps no activation copy or results")
         self.norm = None
         if params.get("norm"):
             from .base import NORMS
@@ -93,7 +97,7 @@ class TokenEmbedding(Embedding):
     def forward(self, token_ids: torch.Tensor) -> torch.Tensor:
         out = torch.empty((token_ids.numel(), self.hidden_size), dtype=torch.float32,
                           device=token_ids.device)
-        core.embed(token_ids, self.weight, out, self.rt.err)
+        core.embed(token_ids, self.weight, out, self.rt.err, self.scale)
         return out
 
 

@@ -11,8 +11,10 @@ kept.
 Parameters: ``hidden_size``, ``intermediate_size``, ``prefix`` (checkpoint
 prefix, e.g. "model.layers.0.mlp."), ``names`` (the three tensors' names
 behind the prefix, default gate_proj.weight / up_proj.weight /
-down_proj.weight), ``activation`` of the gate: "silu" (default) or
-"gelu_tanh", ``0.5 g (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3)))``.
+down_proj.weight), ``activation`` of the gate: "silu" (default),
+"gelu_tanh", ``0.5 g (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3)))``, or "clamped_swish",
+``g' sigmoid(alpha g') (u' + 1)`` for the whole with ``g' = min(g, limit)`` and ``u'`` the
+up held to [-limit, limit] (parameters ``limit``, None for none, and ``alpha``).
 """
 
 from __future__ import annotations
@@ -40,6 +42,8 @@ class SwiGLU(FeedForward):
         if self.activation not in core.ACTIVATIONS:
             raise ConfigError(f"gated feed-forward: unknown activation {self.activation!r}; "
                               f"known: {sorted(core.ACTIVATIONS)}")
+        limit = params.get("limit")
+        self.act_args = {"limit": float("inf") if limit is None else float(limit), "alpha": float(params.get("alpha", 1.0))}
         self.gate_up: Optional[Linear] = None
         self.down: Optional[Linear] = None
 
@@ -69,14 +73,24 @@ class SwiGLU(FeedForward):
     def weight_bytes(self) -> int:
         return self.gate_up.nbytes + self.down.nbytes
 
+    # the product that ends the sub-layer, for arrangements that end two sub-layers in one product
+    @property
+    def out_proj(self) -> Linear:
+        return self.down
+
     def forward(self, x: torch.Tensor, ctx=None) -> torch.Tensor:
         act = torch.empty((x.shape[0], self.intermediate_size), dtype=x.dtype, device=x.device)
+        self.forward_hidden(x, ctx, act)
+        return self.down(act)
+
+    def forward_hidden(self, x: torch.Tensor, ctx, act: torch.Tensor) -> None:
+        """What the last product reads, into ``act`` [N, intermediate] (may lie in wider rows)."""
         fused = False
         if self.block == 64 and x.dtype == torch.bfloat16 and self.gate_up.weight.dtype == torch.bfloat16:
             from ..ops import gemm_tc
 
             fused = gemm_tc.swiglu_route(x, self.gate_up.weight, act, self.gate_up.err,
-                                         activation=self.activation)
+                                         activation=self.activation, act_limit=self.act_args["limit"],
+                                         act_alpha=self.act_args["alpha"])
         if not fused:
-            core.gated_act(self.gate_up(x), act, self.activation, block=self.block)
-        return self.down(act)
+            core.gated_act(self.gate_up(x), act, self.activation, block=self.block, **self.act_args)

@@ -3,7 +3,8 @@ directly, no ``1 + w``), sum of squares and rsqrt in 32-bit, one rounding at
 the store.  Reference: infernum-cuda/kernels/rmsnorm.cu:64-94 and, fused with
 the residual add, infernum-cuda/kernels/add_rmsnorm.cu:78-108.
 
-Parameters: ``hidden_size``, ``eps``, ``weight`` (checkpoint tensor name).
+Parameters: ``hidden_size``, ``eps``, ``weight`` (checkpoint tensor name), ``optional``
+(the checkpoint may leave the weight out; the norm is then not used).
 """
 
 from __future__ import annotations
@@ -23,18 +24,22 @@ class RMSNorm(Norm):
         self.hidden_size = int(params["hidden_size"])
         self.eps = float(params["eps"])
         self.weight_name = params["weight"]
+        self.optional = bool(params.get("optional", False))
         self.weight: Optional[torch.Tensor] = None
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
-        return {self.weight_name: WeightSpec((self.hidden_size,), init="norm")}
+        return {self.weight_name: WeightSpec((self.hidden_size,), init="norm", optional=self.optional)}
 
     def bind(self, weights) -> None:
-        self.weight = weights[self.weight_name].contiguous()
+        w = weights.get(self.weight_name) if self.optional else weights[self.weight_name]
+        self.weight = w.contiguous() if w is not None else None
 
     def weight_bytes(self) -> int:
-        return self.weight.numel() * self.weight.element_size()
+        return self.weight.numel() * self.weight.element_size() if self.weight is not None else 0
 
     def forward(self, stream: ResidualStream, row_idx: Optional[torch.Tensor] = None) -> torch.Tensor:
+        if stream.pending is not None and row_idx is None:
+            stream.own()
         residual = stream.residual
         n_out = residual.shape[0] if row_idx is None else row_idx.numel()
         out = torch.empty((n_out, self.hidden_size), dtype=self.rt.dtype, device=residual.device)
@@ -43,6 +48,23 @@ class RMSNorm(Norm):
         if row_idx is None:
             stream.pending = None
         return out
+
+    def pairs_with(self, other: Norm) -> bool:
+        """Whether ``forward_pair`` with this other norm is one kernel."""
+        return type(other) is type(self) and other.eps == self.eps and other.hidden_size == self.hidden_size \
+            and other.weight is not None and self.weight is not None and other.weight.dtype == self.weight.dtype \
+            and (self.hidden_size % 4 == 0 or self.hidden_size <= 8192) and self.hidden_size <= 16384
+
+    def forward_pair(self, stream: ResidualStream, other: "RMSNorm"):
+        """Folds the stream's pending delta into its residual and returns this norm's and the
+        other's rows of the sum (one root mean square, two weights, one kernel)."""
+        x, delta = stream.residual, stream.pending
+        fresh = delta is not None and stream.origin is not None and stream.origin.data_ptr() == x.data_ptr()
+        x_out = torch.empty_like(x) if fresh else x  # (the embedding's output is never written over)
+        outs = [torch.empty(x.shape, dtype=self.rt.dtype, device=x.device) for _ in range(2)]
+        core.add_rmsnorm_pair(x, delta, x_out, self.weight, other.weight, self.eps, *outs)
+        stream.residual, stream.pending = x_out, None
+        return outs[0], outs[1]
 
     def apply(self, x: torch.Tensor) -> torch.Tensor:
         out = torch.empty(x.shape, dtype=self.rt.dtype, device=x.device)

@@ -9,6 +9,12 @@ the activation dtype and returns 32-bit, which is the new stream; the vector
 is added in 32-bit.
 
 Parameters: ``hidden_size``, ``passes``, ``weight``, ``step`` (tensor names).
+
+``add_reentry``: before pass t the stream becomes ``x + x0 + s_t`` - in the first
+pass ``x + s_0`` - all sums in 32-bit, what the layer before still has pending
+included, in one kernel.
+
+Parameters: ``hidden_size``, ``passes``, ``step`` (a tensor name).
 """
 
 from __future__ import annotations
@@ -59,3 +65,33 @@ class ConcatReentry(Part):
         core.add_row(out, self.step[number])
         stream.residual = out
         stream.act = None
+
+
+@ENTRIES.register("add_reentry")
+class AddReentry(Part):
+    def __init__(self, params, rt: Runtime):
+        super().__init__(params, rt)
+        self.hidden_size = int(params["hidden_size"])
+        self.passes = int(params["passes"])
+        self.step_name = params["step"]
+        self.step: Optional[torch.Tensor] = None
+
+    def weight_specs(self) -> Dict[str, WeightSpec]:
+        return {self.step_name: WeightSpec((self.passes, self.hidden_size), std=0.1)}
+
+    def bind(self, weights) -> None:
+        self.step = weights[self.step_name].to(torch.float32).contiguous()
+
+    def weight_bytes(self) -> int:
+        return self.hidden_size * 4
+
+    def forward(self, stream: ResidualStream, number: int) -> None:
+        if stream.origin is None:
+            raise ConfigError("a pass entry needs the embedding's output (the embedding keeps none)")
+        if not 0 <= number < self.passes:
+            raise ConfigError(f"pass {number} is outside the {self.passes} the model has")
+        x = stream.residual
+        # (the embedding's output is never written over)
+        out = torch.empty_like(x) if stream.origin.data_ptr() == x.data_ptr() else x
+        core.reenter_add(x, stream.pending, stream.origin if number > 0 else None, self.step[number], out)
+        stream.residual, stream.pending, stream.act = out, None, None

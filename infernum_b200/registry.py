@@ -72,3 +72,5 @@ def _ensure_builtin() -> None:
         from .models import bolovik  # noqa: F401
     if "Vodatar" not in _ARCHITECTURES:
         from .models import vodatar  # noqa: F401
+    if "Menitar" not in _ARCHITECTURES:
+        from .models import menitar  # noqa: F401
