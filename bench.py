@@ -118,13 +118,15 @@ class ClockSampler:
 
 def decode_bytes(model, cache, live_tokens: int, batch: int = 0) -> int:
     """Bytes one decode step has to move: every weight it uses once, the keys and
-    values of the live requests (inside their windows), and the requests' fixed-size
+    values of the live requests (inside their windows or runs), and the requests' fixed-size
     state, read and written."""
     per_token = 0
     el = 2 if model.rt.dtype != __import__("torch").float32 else 4
     per_request = live_tokens / max(batch, 1)
     for g in cache.groups:
         seen = min(per_request, g.spec.window) if g.spec.window > 0 and batch else per_request
+        if g.spec.chunk > 0 and batch:
+            seen = min(seen, per_request % g.spec.chunk)  # (the tokens of the run the next one is in)
         per_token += g.spec.elements_per_token() * el * len(g.positions) * (seen / per_request if per_request else 1)
     return int(model.step_weight_bytes() + per_token * live_tokens + 2 * batch * cache.state_bytes_per_request())
 
@@ -488,6 +490,39 @@ def vodatar_prefill_flops(cfg: dict, T: int) -> float:
     return total + 2.0 * D * cfg["vocab"]
 
 
+def menitar_config(width, layers, heads, kv_heads, ff, vocab, chunk=2048):
+    """Parallel layers: attention within runs of ``chunk`` positions whose heads exchange their scores
+    (heads of 128, half of each rotated) beside a gated feed-forward with a clamped swish.  The first two
+    layers are walked twice, so ``layers`` runs come from ``layers - 2`` layers."""
+    att = {"heads": heads, "kv_heads": kv_heads, "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+           "mask": {"size": chunk}, "rot": {"dims": 64, "base": 500000.0}}
+    n = max(layers - 2, 2)
+    return {"architecture": "Menitar", "vocab": vocab, "width": width, "logit_scale": 1.0, "norm": {"eps": 1e-6},
+            "embedding": {"scale": 1.0}, "loop": {"start": 0, "stop": 2, "times": 2},
+            "layers": [{"type": "attention", "mixer": att, "mlp": {"kind": "dense", "ff": ff, "limit": 7.0}}
+                       for _ in range(n)], "max_position": 8192}
+
+
+def menitar_prefill_flops(cfg: dict, T: int) -> float:
+    """Multiply-adds x 2 of one prompt step: the products of every run of a layer, and scores, their
+    exchange among the heads and the weighted values over the keys a query sees."""
+    D, total = cfg["width"], 0.0
+    loop = cfg.get("loop")
+    runs = list(range(len(cfg["layers"])))
+    if loop:
+        runs = list(range(loop["start"])) + list(range(loop["start"], loop["stop"])) * loop["times"] \
+            + list(range(loop["stop"], len(cfg["layers"])))
+    for i in runs:
+        m, mlp = cfg["layers"][i]["mixer"], cfg["layers"][i].get("mlp")
+        H, G, d, v = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+        c = (m.get("mask") or {}).get("size", 0)
+        keys = sum(t % c + 1 if c else t + 1 for t in range(T))
+        total += 2.0 * T * D * (H * d + G * d + G * v + H) + 2.0 * T * H * v * D + 2.0 * H * (d + H + v) * keys
+        if mlp:
+            total += 6.0 * T * D * mlp["ff"]
+    return total + 2.0 * D * cfg["vocab"]
+
+
 DESIGN_SIZES = {
     # name: (width, layers, heads, feed-forward, vocabulary, q_rank, llama kv heads)
     "2b-shape": (2048, 8, 16, 8192, 32000, 768, 4),
@@ -532,6 +567,9 @@ def design_compare(args, peaks) -> dict:
             other_flops = vodatar_prefill_flops
             beside, beside_cfg, beside_flops = "rugesun", rugesun_config(width, layers, heads, ff, vocab, q_rank), \
                 rugesun_prefill_flops
+        elif args.design == "menitar":
+            other = menitar_config(width, layers, heads, kv_heads, ff, vocab)
+            other_flops = menitar_prefill_flops
         else:
             other = rugesun_config(width, layers, heads, ff, vocab, q_rank)
             other_flops = rugesun_prefill_flops
@@ -651,7 +689,7 @@ def main() -> int:
     ap.add_argument("--only", choices=["decode", "prefill"], default=None,
                     help="run one part only and print its numbers (for profiling)")
     ap.add_argument("--no-cuda-graph", action="store_true", help="launch decode steps kernel by kernel")
-    ap.add_argument("--design", choices=["rugesun", "nadozen", "bolovik", "vodatar"], default=None,
+    ap.add_argument("--design", choices=["rugesun", "nadozen", "bolovik", "vodatar", "menitar"], default=None,
                     help="instead of the default workload: prefill and decode of this design at a few sizes,\n"
                          "beside the Llama decoder (bolovik: the Nadozen decoder; vodatar: the Rugesun decoder) at equal sizes; prints one JSON line {\"design\": ...}")
     ap.add_argument("--size", default=None, help="with --design: one of its sizes only")

@@ -6,6 +6,10 @@ counters (without that flag ncu locks the clocks of a GPU that others share).
     python -m infernum_b200.cli.kernel_bench attention-decode --batch 64 --kv-len 1100
     python -m infernum_b200.cli.kernel_bench attention-prefill --tokens 2048
     python -m infernum_b200.cli.kernel_bench attention-prefill --tokens 512 --prefix 3584
+    python -m infernum_b200.cli.kernel_bench talk-prefill --tokens 2048 --chunk 1024
+    python -m infernum_b200.cli.kernel_bench talk-decode --batch 8 --kv-len 1100
+    python -m infernum_b200.cli.kernel_bench qk-row-norm --tokens 2048 --rotary 64
+    python -m infernum_b200.cli.kernel_bench norm-pair --tokens 2048 --hidden 4096
     python -m infernum_b200.cli.kernel_bench gemm --tokens 8 --n 4096 --k 4096
     python -m infernum_b200.cli.kernel_bench norm --tokens 2048 --hidden 4096
     python -m infernum_b200.cli.kernel_bench rope --tokens 2048
@@ -90,7 +94,8 @@ def _attention_case(batch, rows, kv_len, nh, nkv, hd, page_size, device):
 
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawTextHelpFormatter)
-    ap.add_argument("kernel", choices=["attention-decode", "attention-prefill", "gemm", "norm", "rope", "silu"])
+    ap.add_argument("kernel", choices=["attention-decode", "attention-prefill", "talk-decode", "talk-prefill", "gemm", "norm",
+                                       "norm-pair", "qk-row-norm", "rope", "silu"])
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--tokens", type=int, default=2048)
     ap.add_argument("--kv-len", type=int, default=1100)
@@ -98,12 +103,14 @@ def main(argv=None) -> int:
     ap.add_argument("--heads", type=int, default=32)
     ap.add_argument("--kv-heads", type=int, default=8)
     ap.add_argument("--head-dim", type=int, default=128)
+    ap.add_argument("--chunk", type=int, default=0, help="talk-*: positions in a run that see one another")
+    ap.add_argument("--rotary", type=int, default=64, help="qk-row-norm: rotated dimensions of a head")
     ap.add_argument("--hidden", type=int, default=4096)
     ap.add_argument("--intermediate", type=int, default=14336)
     ap.add_argument("--n", type=int, default=4096)
     ap.add_argument("--k", type=int, default=4096)
     ap.add_argument("--page-size", type=int, default=16)
-    ap.add_argument("--splits", type=int, default=0, help="force a slice count (attention-decode, attention-prefill, gemm)")
+    ap.add_argument("--splits", type=int, default=0, help="force a slice count (attention-*, talk-*, gemm)")
     ap.add_argument("--reps", type=int, default=50)
     ap.add_argument("--warmup", type=int, default=5)
     ap.add_argument("--library", action="store_true", help="gemm: time the library product instead")
@@ -157,6 +164,30 @@ def main(argv=None) -> int:
             flops = 4.0 * nh * hd * (rows * (rows + 1) / 2 + rows * args.prefix)
             out.update(tokens=rows, prefix=args.prefix, us=us, tflops=flops / us / 1e6,
                        frac_of_bf16=flops / us / 1e6 / peaks["bf16_tflops"])
+    elif args.kernel in ("talk-decode", "talk-prefill"):
+        from ..ops import attention_talk
+
+        decode = args.kernel == "talk-decode"
+        batch, rows = (args.batch, 1) if decode else (1, args.tokens)
+        kv_len = args.kv_len if decode else args.tokens + args.prefix
+        cases = [_attention_case(batch, rows, kv_len, nh, nkv, hd, args.page_size, dev) for _ in range(3 if decode else 1)]
+        outs = torch.empty(batch * rows, nh * hd, dtype=torch.bfloat16, device=dev)
+        talk = (torch.randn(nh, nh, device=dev) * nh ** -0.5).bfloat16().float().contiguous()
+        temp = torch.rand(nh, device=dev)
+        gate = torch.randn(batch * rows, nh, device=dev).to(torch.bfloat16)
+        if args.splits:
+            rt.options["talk_splits"] = args.splits
+        fns = [lambda q=q, kp=kp, vp=vp, tables=tables, ctx=ctx: attention_talk.run(
+            q, kp, vp, outs, ctx, tables, nh, hd ** -0.5, talk, temp, gate, args.chunk, 0, rt)
+            for q, kp, vp, tables, ctx in cases]
+        us = _time(fns, args.reps, args.warmup, not args.no_graph)
+        c = args.chunk
+        keys = sum(p % c + 1 if c else p + 1 for p in range(kv_len - rows, kv_len))
+        plan = next(v for k, v in cases[0][4].scratch.items() if isinstance(k, tuple))
+        out.update(batch=batch, rows=rows, kv_len=kv_len, chunk=c, plan=list(plan), us=us)
+        nbytes, flops = batch * keys * nkv * hd * 2 * 2, batch * 2.0 * nh * (2 * hd + nh) * keys
+        out.update(gbs=nbytes / us / 1e3, frac_of_hbm=nbytes / us / 1e3 / peaks["hbm_gbs"]) if decode else \
+            out.update(tflops=flops / us / 1e6, frac_of_bf16=flops / us / 1e6 / peaks["bf16_tflops"])
     elif args.kernel == "gemm":
         T, N, K = args.tokens, args.n, args.k
         copies = max(2, int(300e6 / (N * K * 2)) + 1)
@@ -191,6 +222,33 @@ def main(argv=None) -> int:
         nbytes = T * H * (4 + 2 + 4 + 2)
         out.update(tokens=T, hidden=H, us=us, gbs=nbytes / us / 1e3,
                    frac_of_hbm=nbytes / us / 1e3 / peaks["hbm_gbs"])
+    elif args.kernel == "norm-pair":
+        T, H = args.tokens, args.hidden
+        n = max(2, int(300e6 / (T * H * 14)) + 1)
+        res = [torch.randn(T, H, device=dev) for _ in range(n)]
+        delta = [torch.randn(T, H, device=dev).to(torch.bfloat16) for _ in range(n)]
+        w = torch.ones(H, dtype=torch.bfloat16, device=dev)
+        o1, o2 = (torch.empty(T, H, dtype=torch.bfloat16, device=dev) for _ in range(2))
+        fns = [lambda r=r, d=d: core.add_rmsnorm_pair(r, d, r, w, w, 1e-5, o1, o2) for r, d in zip(res, delta)]
+        us = _time(fns, args.reps, args.warmup, not args.no_graph)
+        nbytes = T * H * (4 + 2 + 4 + 2 + 2)
+        out.update(tokens=T, hidden=H, us=us, gbs=nbytes / us / 1e3, frac_of_hbm=nbytes / us / 1e3 / peaks["hbm_gbs"])
+    elif args.kernel == "qk-row-norm":
+        T, ps = args.tokens, args.page_size
+        n = max(2, int(300e6 / (T * (nh + 2 * nkv) * hd * 2)) + 1)
+        xs = [torch.randn(T, (nh + 2 * nkv) * hd + nh, device=dev).to(torch.bfloat16) for _ in range(n)]
+        pages = -(-T // ps)
+        kp, vp = (torch.zeros(pages, nkv, ps, hd, dtype=torch.bfloat16, device=dev) for _ in range(2))
+        pos = torch.arange(T, dtype=torch.int32, device=dev)
+        ent = torch.zeros(T, dtype=torch.int32, device=dev)
+        tables = torch.arange(pages, dtype=torch.int32, device=dev).view(1, pages)
+        inv = torch.rand(args.rotary // 2, device=dev)
+        qw, kw = torch.ones(nh * hd, device=dev), torch.ones(nkv * hd, device=dev)
+        fns = [lambda x=x: core.qk_row_norm_append(x, qw, kw, 1e-5, inv, args.rotary, nh, nkv, hd, hd, pos, ent, tables, kp,
+                                                   vp, rt.err) for x in xs]
+        us = _time(fns, args.reps, args.warmup, not args.no_graph)
+        nbytes = T * (nh + 2 * nkv) * hd * 2 * 2
+        out.update(tokens=T, us=us, gbs=nbytes / us / 1e3, frac_of_hbm=nbytes / us / 1e3 / peaks["hbm_gbs"])
     elif args.kernel == "rope":
         T = args.tokens
         width = (nh + 2 * nkv) * hd

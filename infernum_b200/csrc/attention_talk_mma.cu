@@ -5,23 +5,24 @@
 //   r_g(i, j) = (q_g(i) . k_g(j)) * scale * temp_g        s_h(i, j) = sum_g talk[h, g] r_g(i, j)
 //   out_h(i)  = sum_j softmax_j(s_h(i, .)) v_h(j) * sigmoid(gate_h(i))
 //
-// The exchange runs over all heads, so a CTA holds all heads of its eight queries: keys of every
-// key/value head come in tiles of BN that start at absolute multiples of BN whatever the step's cut.
-// A tile is worked on in three passes with a barrier between them:
+// The exchange runs over all heads, so a CTA holds all heads of its BQ queries (8; for decoded tokens as
+// many as fill eight columns of one key/value head): keys of every key/value head come in tiles of BN that
+// start at absolute multiples of BN whatever the step's cut.  The columns of a key/value head are its
+// (query, head) pairs, query by query; a unit is eight of them, and a warp owns UW units.  A tile is
+// worked on in three passes with a barrier between them:
 //
-//   1  a warp owns HW consecutive heads and computes S^T = K Q^T for each, [keys x 8 queries]; the
-//      scaled scores go to shared memory as three bf16 numbers that add up to the 32-bit score (8
-//      mantissa bits each), one plane a number, [query][key][head].
-//   2  a warp takes a query: [heads x heads] (bf16, exact) times [heads x keys], the three planes one
-//      after the other into one 32-bit accumulator: the exchange at 32-bit precision on the tensor
-//      cores.  The result replaces the query's planes as 32-bit, [head][key].
-//   3  a warp takes its heads again: running softmax over the tile and O^T += V^T P^T, [values x 8
-//      queries] in registers.
+//   1  S^T = K Q^T per unit, [keys x 8 columns]; the scaled scores go to shared memory as three bf16
+//      numbers that add up to the 32-bit score (8 mantissa bits each), one plane a number,
+//      [query][key][head].
+//   2  per query, 16 heads and 16 keys: [heads x heads] (bf16, exact) times [heads x keys], the three
+//      planes one after the other into one 32-bit accumulator: the exchange at 32-bit precision on the
+//      tensor cores.  The result goes to shared memory as 32-bit, [query][head][key].
+//   3  per unit: running softmax over the tile and O^T += V^T P^T, [values x 8 columns] in registers.
 //
-// K has one stage (free after pass 1), V two; both of the next tile are fetched by cp.async during
-// passes 2 and 3.  Key places are looked up in the block table once per tile, two tiles ahead.  Where
-// all heads' accumulators do not fit the registers the values are cut in ES column blocks over CTAs,
-// each of which computes the scores.
+// Keys have one stage, fetched by cp.async while passes 2 and 3 of the tile before run, and so have the
+// values, fetched during passes 1 and 2.  Key places are looked up in the block table once per tile, two
+// tiles ahead.  Where the accumulators do not fit the registers the values are cut in ES column blocks
+// over CTAs, each of which computes the scores.
 //
 // Steps of few rows cut the keys in slices over CTAs; each writes its maxima, denominators and
 // unnormed sums in 32-bit and a second kernel weighs them.
@@ -40,43 +41,50 @@ namespace {
 constexpr int H = TALK_H, G = TALK_G, D = TALK_D, E = TALK_E, R = H / G;
 static_assert(H % G == 0 && D % 16 == 0 && E % 16 == 0 && D >= 16 && E >= 16, "sizes this kernel takes");
 constexpr int gcd_of(int a, int b) { return b == 0 ? a : gcd_of(b, a % b); }
-constexpr int BQ = 8;                               // queries of a CTA
-constexpr int WARPS = H >= 8 ? 8 : 4, THREADS = WARPS * 32;
-constexpr int HW = (H + WARPS - 1) / WARPS;         // heads of a warp
-constexpr int SEG = gcd_of(HW, R);                  // of those, runs that share a key/value head
 constexpr int HP = (H + 15) / 16 * 16;              // heads padded to the exchange's 16 x 16 pieces
-constexpr int value_block() {
-    for (int e = E; e >= 16; e -= 16)
-        if (E % e == 0 && HW * e <= 512) return e;
-    return 16;
-}
-constexpr int EB = value_block(), ES = E / EB;      // values in ES blocks of EB columns
-constexpr int QS = D + 8, KS = D + 8, VS = EB + 8, SR = HP + 8;  // row strides (elements): 16 bytes of padding
+constexpr int KT = HP / 16;
+constexpr int SR = HP + 8, QS = D + 8, KS = D + 8;  // row strides (elements): 16 bytes of padding
 constexpr int PLANES = 3;
-constexpr bool alias_of(int bn) { return bn / 8 * (HP / 16) * 2 * PLANES <= 48; }
-// Bytes of a query's region: the planes, and the exchanged scores in their place or behind them; the
-// stride between queries is 8 words beyond a multiple of 32 banks.
-constexpr int plane_bytes(int bn) { return bn * SR * 2; }
-constexpr int mix_bytes(int bn) { return H * (bn + 8) * 4; }
-constexpr int region_bytes(int bn) {
-    int b = alias_of(bn) ? (PLANES * plane_bytes(bn) > mix_bytes(bn) ? PLANES * plane_bytes(bn) : mix_bytes(bn))
-                         : PLANES * plane_bytes(bn) + mix_bytes(bn);
-    b = (b + 127) / 128 * 128 + 32;
-    return b;
-}
-constexpr int OUT_STAGE = WARPS * 8 * VS * 2;
-constexpr int smem_bytes(int bn) {
-    const int b = BQ * H * QS * 2 + G * bn * KS * 2 + 2 * G * bn * VS * 2 + BQ * region_bytes(bn) + HP * SR * 2 +
-                  (H + 3) / 4 * 16 + 3 * bn * 4;
-    return b > OUT_STAGE ? b : OUT_STAGE;
-}
 constexpr int SMEM_MAX = 227 * 1024;
-constexpr int BN = smem_bytes(32) <= SMEM_MAX ? 32 : 16;  // keys of a tile
-constexpr int SMEM = smem_bytes(BN);
-constexpr bool FITS = SMEM <= SMEM_MAX && HW * EB <= 512;
-constexpr bool ALIAS = alias_of(BN);
-constexpr int QR = region_bytes(BN), PLANE = plane_bytes(BN), MIX_AT = ALIAS ? 0 : PLANES * PLANE, MS = BN + 8;
-constexpr int MT = BN / 16, ET = EB / 16, KT = HP / 16;
+constexpr int BQ_FEW = R >= 8 ? 1 : 8 / R;          // queries of a CTA when every entry has few rows
+
+template <int BQ>
+struct Cfg {
+    static constexpr int UPG = (BQ * R + 7) / 8;    // units of a key/value head
+    static constexpr int NU = G * UPG;
+    static constexpr int WARPS = NU >= 16 && BQ == 8 ? 16 : (NU >= 8 ? 8 : 4);
+    static constexpr int THREADS = WARPS * 32;
+    static constexpr int UW = (NU + WARPS - 1) / WARPS;
+    static constexpr int SEG = gcd_of(UW, UPG);     // of a warp's units, runs that share a key/value head
+    static constexpr int MOST = WARPS == 16 ? 256 : 512;  // UW * EB: accumulators that fit the registers
+    static constexpr int value_block() {
+        for (int e = E; e >= 16; e -= 16)
+            if (E % e == 0 && UW * e <= MOST) return e;
+        return 16;
+    }
+    static constexpr int EB = value_block(), ES = E / EB;  // values in ES blocks of EB columns
+    static constexpr int VS = EB + 8, ET = EB / 16;
+    static constexpr int plane_bytes(int bn) { return bn * SR * 2; }
+    // A query's region: the planes, then the exchanged scores; 8 words beyond a multiple of the 32 banks.
+    static constexpr int region_bytes(int bn) { return (PLANES * plane_bytes(bn) + H * (bn + 8) * 4 + 127) / 128 * 128 + 32; }
+    static constexpr int smem_bytes(int bn) {
+        const int b = G * UPG * 8 * QS * 2 + G * bn * KS * 2 + G * bn * VS * 2 + BQ * region_bytes(bn) + HP * SR * 2 +
+                      (H + 3) / 4 * 16 + 3 * bn * 4;
+        const int st = WARPS * 8 * VS * 2;
+        return b > st ? b : st;
+    }
+    // keys of a tile: for few rows as many as leave room for a second CTA on the SM, if any do
+    static constexpr int pick() {
+        if (BQ != 8 || BQ_FEW == 8) {
+            if (smem_bytes(32) <= SMEM_MAX / 2 - 1024) return 32;
+            if (smem_bytes(16) <= SMEM_MAX / 2 - 1024) return 16;
+        }
+        return smem_bytes(32) <= SMEM_MAX ? 32 : 16;
+    }
+    static constexpr int BN = pick(), SMEM = smem_bytes(BN), QR = region_bytes(BN), PLANE = plane_bytes(BN),
+                         MIX_AT = PLANES * PLANE, MS = BN + 8, MT = BN / 16;
+    static constexpr bool FITS = SMEM <= SMEM_MAX && UW * EB <= MOST;
+};
 
 __device__ __forceinline__ unsigned smem_addr(const void* p) { return (unsigned)__cvta_generic_to_shared(p); }
 __device__ __forceinline__ void ldsm_x4(unsigned& r0, unsigned& r1, unsigned& r2, unsigned& r3, const bf16* p) {
@@ -102,6 +110,8 @@ __device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
 __device__ __forceinline__ void cp_async16(bf16* smem, const bf16* gmem) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(smem_addr(smem)), "l"(gmem));
 }
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;\n" ::: "memory"); }
+__device__ __forceinline__ void cp_async_wait_but_one() { asm volatile("cp.async.wait_group 1;\n" ::: "memory"); }
 __device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_all;\n" ::: "memory"); }
 
 struct Params {
@@ -115,16 +125,20 @@ struct Params {
     float *stats, *part;  // [splits][rows][H][2], [splits][rows][H][E]
 };
 
-template <bool SPLIT>
-__global__ void __launch_bounds__(THREADS, 1) attention_talk_mma_kernel(const Params p) {
+template <int BQ, bool SPLIT>
+__global__ void __launch_bounds__(Cfg<BQ>::THREADS, 1) attention_talk_mma_kernel(const Params p) {
+    using C = Cfg<BQ>;
+    constexpr int UPG = C::UPG, NU = C::NU, WARPS = C::WARPS, THREADS = C::THREADS, UW = C::UW, SEG = C::SEG, EB = C::EB,
+                  VS = C::VS, ET = C::ET, BN = C::BN, QR = C::QR, PLANE = C::PLANE, MIX_AT = C::MIX_AT, MS = C::MS,
+                  MT = C::MT;
     pdl_trigger();
     extern __shared__ __align__(128) unsigned char smem_raw[];
-    bf16* qs = reinterpret_cast<bf16*>(smem_raw);          // [H][8][QS]
-    bf16* ks = qs + H * BQ * QS;                           // [G][BN][KS]
-    bf16* vs_all = ks + G * BN * KS;                       // [2][G][BN][VS]
-    unsigned char* regions = reinterpret_cast<unsigned char*>(vs_all + 2 * G * BN * VS);  // [8][QR]
-    bf16* ts = reinterpret_cast<bf16*>(regions + BQ * QR);  // [HP][SR]
-    float* hs = reinterpret_cast<float*>(ts + HP * SR);     // [H] (padded to 4): scale * temperature
+    bf16* qs = reinterpret_cast<bf16*>(smem_raw);            // [NU * 8 columns][QS]
+    bf16* ks = qs + NU * 8 * QS;                             // [G][BN][KS]
+    bf16* vs = ks + G * BN * KS;                             // [G][BN][VS]
+    unsigned char* regions = reinterpret_cast<unsigned char*>(vs + G * BN * VS);  // [BQ][QR]
+    bf16* ts = reinterpret_cast<bf16*>(regions + BQ * QR);   // [HP][SR]
+    float* hs = reinterpret_cast<float*>(ts + HP * SR);      // [H] (padded to 4): scale * temperature
     int* places = reinterpret_cast<int*>(hs + (H + 3) / 4 * 4);  // [3][BN]: a key's row in the pool, -1: none
 
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gq = lane >> 2, tq = lane & 3;
@@ -135,6 +149,13 @@ __global__ void __launch_bounds__(THREADS, 1) attention_talk_mma_kernel(const Pa
         ts[h * SR + g] = __float2bfloat16_rn(v);
     }
     for (int i = tid; i < H; i += THREADS) hs[i] = p.scale * (p.temp ? p.temp[i] : 1.f);
+    if (HP != H) {  // heads that only fill up a piece: zeros, or what lies there would meet a zero weight
+        constexpr int PADS = HP == H ? 1 : HP - H;
+        for (int i = tid; i < BQ * PLANES * BN * PADS; i += THREADS) {
+            const int c = i % PADS, key = i / PADS % (PLANES * BN), qi = i / (PADS * PLANES * BN);
+            reinterpret_cast<bf16*>(regions + qi * QR)[key * SR + H + c] = __float2bfloat16_rn(0.f);
+        }
+    }
     pdl_wait();
 
     const int en = blockIdx.y, sp = SPLIT ? blockIdx.z % p.splits : 0, eb = SPLIT ? blockIdx.z / p.splits : blockIdx.z;
@@ -172,9 +193,9 @@ __global__ void __launch_bounds__(THREADS, 1) attention_talk_mma_kernel(const Pa
             places[t % 3 * BN + tid] = at;
         }
     };
-    auto fetch = [&](int t) {
+    auto fetch_keys = [&](int t) {
         const int* pl = places + t % 3 * BN;
-        constexpr int KC = D / 8, VC = EB / 8;
+        constexpr int KC = D / 8;
         for (int c = tid; c < G * BN * KC; c += THREADS) {
             const int part = c % KC, key = c / KC % BN, g = c / (KC * BN), at = pl[key];
             bf16* dst = ks + (g * BN + key) * KS + part * 8;
@@ -183,7 +204,11 @@ __global__ void __launch_bounds__(THREADS, 1) attention_talk_mma_kernel(const Pa
             else
                 *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
         }
-        bf16* vs = vs_all + (t & 1) * G * BN * VS;
+        cp_async_commit();
+    };
+    auto fetch_values = [&](int t) {
+        const int* pl = places + t % 3 * BN;
+        constexpr int VC = EB / 8;
         for (int c = tid; c < G * BN * VC; c += THREADS) {
             const int part = c % VC, key = c / VC % BN, g = c / (VC * BN), at = pl[key];
             bf16* dst = vs + (g * BN + key) * VS + part * 8;
@@ -192,31 +217,32 @@ __global__ void __launch_bounds__(THREADS, 1) attention_talk_mma_kernel(const Pa
             else
                 *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
         }
+        cp_async_commit();
     };
 
     {
         constexpr int QC = D / 8;
-        for (int c = tid; c < BQ * H * QC; c += THREADS) {
-            const int part = c % QC, h = c / QC % H, qi = c / (QC * H);
-            bf16* dst = qs + (h * BQ + qi) * QS + part * 8;
+        for (int c = tid; c < NU * 8 * QC; c += THREADS) {
+            const int part = c % QC, col = c / QC % (UPG * 8), g = c / (QC * UPG * 8), qi = col / R;
+            bf16* dst = qs + (g * UPG * 8 + col) * QS + part * 8;
             if (qi < nq)
-                cp_async16(dst, q_rows + (size_t)qi * p.q_stride + h * D + part * 8);
+                cp_async16(dst, q_rows + (size_t)qi * p.q_stride + (g * R + col % R) * D + part * 8);
             else
                 *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
         }
+        cp_async_commit();
     }
     if (n_tiles > 0) {
         look_up(0);
         look_up(1);
         __syncthreads();
-        fetch(0);
+        fetch_keys(0);
     }
 
-    // this thread's query in pass 3 (a column of S^T and O^T is a query)
-    const int my_pos = gq < nq ? pos0 + gq : -1, my_lo = gq < nq ? first_key(pos0 + gq) : 0;
-    float o[HW][ET][4], mx[HW], den[HW];
+    // this thread's columns in pass 3 (column gq of every unit)
+    float o[UW][ET][4], mx[UW], den[UW];
 #pragma unroll
-    for (int a = 0; a < HW; ++a) {
+    for (int a = 0; a < UW; ++a) {
         mx[a] = -INFINITY;
         den[a] = 0.f;
 #pragma unroll
@@ -229,12 +255,15 @@ __global__ void __launch_bounds__(THREADS, 1) attention_talk_mma_kernel(const Pa
         const int j0 = klo + t * BN;
         cp_async_wait_all();
         __syncthreads();
-        // ---- pass 1: every head's scores
+        fetch_values(t);
+        // ---- pass 1: the scores of every unit
 #pragma unroll
-        for (int a = 0; a < HW; a += SEG) {
-            const int h0 = warp * HW + a;
-            if (h0 >= H) break;  // (the whole warp; a run of SEG heads exists or does not)
-            const bf16* kg = ks + (h0 / R) * BN * KS + (lane & 15) * KS + (lane >> 4) * 8;
+        for (int a = 0; a < UW; a += SEG) {
+            const int u0 = warp * UW + a;
+            if (u0 >= NU) break;  // (the whole warp; a run of SEG units exists or does not)
+            const int g = u0 / UPG;
+            const bf16* kg = ks + g * BN * KS + (lane & 15) * KS + (lane >> 4) * 8;
+            const bf16* qu = qs + (u0 * 8 + (lane & 7)) * QS;
             float s[SEG][MT][4];
 #pragma unroll
             for (int x = 0; x < SEG; ++x)
@@ -242,149 +271,125 @@ __global__ void __launch_bounds__(THREADS, 1) attention_talk_mma_kernel(const Pa
                 for (int m = 0; m < MT; ++m)
 #pragma unroll
                     for (int i = 0; i < 4; ++i) s[x][m][i] = 0.f;
-#pragma unroll 4
-            for (int kk = 0; kk < D / 16; ++kk) {
-                unsigned ka[MT][4];
+            // two steps of 16 at a time: one load of a unit's columns serves both
+#pragma unroll 2
+            for (int kk = 0; kk + 2 <= D / 16; kk += 2) {
+                unsigned ka[2][MT][4], b[SEG][4];
 #pragma unroll
-                for (int m = 0; m < MT; ++m) ldsm_x4(ka[m][0], ka[m][1], ka[m][2], ka[m][3], kg + m * 16 * KS + kk * 16);
-                if (SEG % 2 == 0) {
+                for (int m = 0; m < MT; ++m)
 #pragma unroll
-                    for (int x = 0; x < SEG; x += 2) {
-                        unsigned b0, b1, b2, b3;
-                        ldsm_x4(b0, b1, b2, b3,
-                                qs + ((h0 + x + (lane >> 4)) * BQ + (lane & 7)) * QS + kk * 16 + ((lane >> 3) & 1) * 8);
+                    for (int y = 0; y < 2; ++y)
+                        ldsm_x4(ka[y][m][0], ka[y][m][1], ka[y][m][2], ka[y][m][3], kg + m * 16 * KS + (kk + y) * 16);
 #pragma unroll
-                        for (int m = 0; m < MT; ++m) {
-                            mma_bf16(s[x][m], ka[m], b0, b1);
-                            mma_bf16(s[x + (SEG > 1)][m], ka[m], b2, b3);
-                        }
-                    }
-                } else {
+                for (int x = 0; x < SEG; ++x)
+                    ldsm_x4(b[x][0], b[x][1], b[x][2], b[x][3], qu + x * 8 * QS + kk * 16 + (lane >> 3) * 8);
+#pragma unroll
+                for (int y = 0; y < 2; ++y)
+#pragma unroll
+                    for (int x = 0; x < SEG; ++x)
+#pragma unroll
+                        for (int m = 0; m < MT; ++m) mma_bf16(s[x][m], ka[y][m], b[x][2 * y], b[x][2 * y + 1]);
+            }
+            if (D / 16 % 2) {
+                constexpr int kk = D / 16 - 1;
+                unsigned ka[4];
+#pragma unroll
+                for (int m = 0; m < MT; ++m) {
+                    ldsm_x4(ka[0], ka[1], ka[2], ka[3], kg + m * 16 * KS + kk * 16);
 #pragma unroll
                     for (int x = 0; x < SEG; ++x) {
                         unsigned b0, b1;
-                        ldsm_x2(b0, b1, qs + ((h0 + x) * BQ + (lane & 7)) * QS + kk * 16 + ((lane >> 3) & 1) * 8);
-#pragma unroll
-                        for (int m = 0; m < MT; ++m) mma_bf16(s[x][m], ka[m], b0, b1);
+                        ldsm_x2(b0, b1, qu + x * 8 * QS + kk * 16 + ((lane >> 3) & 1) * 8);
+                        mma_bf16(s[x][m], ka, b0, b1);
                     }
                 }
             }
             // scaled, in three bf16 numbers each (the differences are exact)
 #pragma unroll
-            for (int m = 0; m < MT; ++m)
+            for (int x = 0; x < SEG; ++x) {
+                const int c0 = (u0 + x) % UPG * 8 + 2 * tq;  // this thread's columns: c0 and c0 + 1
+                const int qa = c0 / R, ha = g * R + c0 % R, qb = (c0 + 1) / R, hb = g * R + (c0 + 1) % R;
+                const bool in_a = BQ * R % 8 == 0 || c0 < BQ * R, in_b = BQ * R % 8 == 0 || c0 + 1 < BQ * R;
+                const float fa = in_a ? hs[ha] : 0.f, fb = in_b ? hs[hb] : 0.f;
+                bf16* da = reinterpret_cast<bf16*>(regions + qa * QR) + gq * SR + ha;
+                bf16* db = reinterpret_cast<bf16*>(regions + qb * QR) + gq * SR + hb;
 #pragma unroll
-                for (int i = 0; i < 4; ++i) {
-                    const int key = m * 16 + gq + (i >> 1) * 8, qi = 2 * tq + (i & 1);
-                    bf16* dst = reinterpret_cast<bf16*>(regions + qi * QR) + key * SR + h0;
-                    bf16 w[PLANES][SEG];
+                for (int m = 0; m < MT; ++m)
 #pragma unroll
-                    for (int x = 0; x < SEG; ++x) {
-                        float v = s[x][m][i] * hs[h0 + x];
+                    for (int i = 0; i < 2; ++i) {
+                        float va = s[x][m][2 * i] * fa, vb = s[x][m][2 * i + 1] * fb;
+                        const int at = (m * 16 + i * 8) * SR;
 #pragma unroll
                         for (int l = 0; l < PLANES; ++l) {
-                            w[l][x] = __float2bfloat16_rn(v);
-                            v -= __bfloat162float(w[l][x]);
-                        }
-                    }
-#pragma unroll
-                    for (int l = 0; l < PLANES; ++l) {
-                        bf16* d = dst + l * (PLANE / 2);
-                        if (SEG % 4 == 0) {
-#pragma unroll
-                            for (int x = 0; x < SEG; x += 4) {
-                                uint2 u;
-                                u.x = (unsigned)__bfloat16_as_ushort(w[l][x]) |
-                                      (unsigned)__bfloat16_as_ushort(w[l][x + (SEG > 1)]) << 16;
-                                u.y = (unsigned)__bfloat16_as_ushort(w[l][x + 2 * (SEG > 2)]) |
-                                      (unsigned)__bfloat16_as_ushort(w[l][x + 3 * (SEG > 3)]) << 16;
-                                *reinterpret_cast<uint2*>(d + x) = u;
+                            const __nv_bfloat162 w = __floats2bfloat162_rn(va, vb);
+                            va -= __low2float(w);
+                            vb -= __high2float(w);
+                            if (R % 2 == 0) {
+                                if (in_a) *reinterpret_cast<__nv_bfloat162*>(da + at + l * (PLANE / 2)) = w;
+                            } else {
+                                if (in_a) da[at + l * (PLANE / 2)] = __low2bfloat16(w);
+                                if (in_b) db[at + l * (PLANE / 2)] = __high2bfloat16(w);
                             }
-                        } else if (SEG % 2 == 0) {
-#pragma unroll
-                            for (int x = 0; x < SEG; x += 2)
-                                *reinterpret_cast<unsigned*>(d + x) =
-                                    (unsigned)__bfloat16_as_ushort(w[l][x]) |
-                                    (unsigned)__bfloat16_as_ushort(w[l][x + (SEG > 1)]) << 16;
-                        } else {
-#pragma unroll
-                            for (int x = 0; x < SEG; ++x) d[x] = w[l][x];
                         }
                     }
-                }
-        }
-        if (HP != H) {  // heads that only fill up a piece: zeros, or what lies there would meet a zero weight
-            constexpr int PADS = HP == H ? 1 : HP - H;
-            for (int i = tid; i < BQ * BN * PADS; i += THREADS) {
-                const int c = i % PADS, key = i / PADS % BN, qi = i / (PADS * BN);
-                bf16* d = reinterpret_cast<bf16*>(regions + qi * QR) + key * SR + H + c;
-#pragma unroll
-                for (int l = 0; l < PLANES; ++l) d[l * (PLANE / 2)] = __float2bfloat16_rn(0.f);
             }
         }
         __syncthreads();
         if (t + 2 < n_tiles) look_up(t + 2);
-        if (t + 1 < n_tiles) fetch(t + 1);
-        // ---- pass 2: the exchange, a query at a time
-        for (int qi = warp; qi < nq; qi += WARPS) {
-            const bf16* raw = reinterpret_cast<const bf16*>(regions + qi * QR);
+        if (t + 1 < n_tiles) fetch_keys(t + 1);
+        // ---- pass 2: the exchange; an item is a query, 16 heads and 16 keys
+        for (int it = warp; it < nq * KT * MT; it += WARPS) {
+            const int n0 = it % MT * 2, m = it / MT % KT, qi = it / (MT * KT);
+            const bf16* raw = reinterpret_cast<const bf16*>(regions + qi * QR) + (n0 * 8 + (lane & 7)) * SR + ((lane >> 3) & 1) * 8;
             float* mix = reinterpret_cast<float*>(regions + qi * QR + MIX_AT);
-            constexpr int NT = BN / 8, GROUP = ALIAS ? NT : 2;  // tiles of 8 keys taken together
+            float c[2][4];
 #pragma unroll
-            for (int n0 = 0; n0 < NT; n0 += GROUP) {
-                unsigned b[GROUP][KT][6];
+            for (int n = 0; n < 2; ++n)
 #pragma unroll
-                for (int n = 0; n < GROUP; ++n)
+                for (int i = 0; i < 4; ++i) c[n][i] = 0.f;
+#pragma unroll 2
+            for (int kk = 0; kk < KT; ++kk) {
+                unsigned a[4], b[PLANES][4];
+                ldsm_x4(a[0], a[1], a[2], a[3], ts + (m * 16 + (lane & 15)) * SR + kk * 16 + (lane >> 4) * 8);
 #pragma unroll
-                    for (int kk = 0; kk < KT; ++kk) {
-                        const bf16* src = raw + ((n0 + n) * 8 + (lane & 7)) * SR + kk * 16 + ((lane >> 3) & 1) * 8;
-                        ldsm_x4(b[n][kk][0], b[n][kk][1], b[n][kk][2], b[n][kk][3], src + (lane >> 4) * (PLANE / 2));
-                        ldsm_x2(b[n][kk][4], b[n][kk][5], src + 2 * (PLANE / 2));
-                    }
-                if (ALIAS) __syncwarp();  // (every lane has read before the planes are written over)
+                for (int l = 0; l < PLANES; ++l)  // both tiles of 8 keys
+                    ldsm_x4(b[l][0], b[l][1], b[l][2], b[l][3], raw + (lane >> 4) * 8 * SR + kk * 16 + l * (PLANE / 2));
 #pragma unroll
-                for (int m = 0; m < KT; ++m) {
-                    float c[GROUP][4];
+                for (int l = PLANES - 1; l >= 0; --l)
 #pragma unroll
-                    for (int n = 0; n < GROUP; ++n)
-#pragma unroll
-                        for (int i = 0; i < 4; ++i) c[n][i] = 0.f;
-#pragma unroll
-                    for (int kk = 0; kk < KT; ++kk) {
-                        unsigned a[4];
-                        ldsm_x4(a[0], a[1], a[2], a[3], ts + (m * 16 + (lane & 15)) * SR + kk * 16 + (lane >> 4) * 8);
-#pragma unroll
-                        for (int l = PLANES - 1; l >= 0; --l)
-#pragma unroll
-                            for (int n = 0; n < GROUP; ++n) mma_bf16(c[n], a, b[n][kk][2 * l], b[n][kk][2 * l + 1]);
-                    }
-#pragma unroll
-                    for (int n = 0; n < GROUP; ++n)
-#pragma unroll
-                        for (int i = 0; i < 2; ++i) {
-                            const int h = m * 16 + gq + i * 8;
-                            if (HP == H || h < H)
-                                *reinterpret_cast<float2*>(mix + h * MS + (n0 + n) * 8 + 2 * tq) =
-                                    make_float2(c[n][2 * i], c[n][2 * i + 1]);
-                        }
-                }
+                    for (int n = 0; n < 2; ++n) mma_bf16(c[n], a, b[l][2 * n], b[l][2 * n + 1]);
             }
+#pragma unroll
+            for (int n = 0; n < 2; ++n)
+#pragma unroll
+                for (int i = 0; i < 2; ++i) {
+                    const int h = m * 16 + gq + i * 8;
+                    if (HP == H || h < H)
+                        *reinterpret_cast<float2*>(mix + h * MS + (n0 + n) * 8 + 2 * tq) = make_float2(c[n][2 * i], c[n][2 * i + 1]);
+                }
         }
+        if (t + 1 < n_tiles) cp_async_wait_but_one();  // the values are here; the next keys need not be
+        else cp_async_wait_all();
         __syncthreads();
         // ---- pass 3: softmax and values
-        const bf16* vs = vs_all + (t & 1) * G * BN * VS;
-        const float* mine = reinterpret_cast<const float*>(regions + gq * QR + MIX_AT);
 #pragma unroll
-        for (int a = 0; a < HW; a += SEG) {
-            const int h0 = warp * HW + a;
-            if (h0 >= H) break;
+        for (int a = 0; a < UW; a += SEG) {
+            const int u0 = warp * UW + a;
+            if (u0 >= NU) break;
+            const int g = u0 / UPG;
             unsigned pb[SEG][MT][2];
 #pragma unroll
             for (int x = 0; x < SEG; ++x) {
+                const int c = (u0 + x) % UPG * 8 + gq, qi = c / R;
+                const bool live = qi < nq;
+                const int pos = live ? pos0 + qi : -1, lo = live ? first_key(pos) : 0;
+                const float* mine = reinterpret_cast<const float*>(regions + (live ? qi : 0) * QR + MIX_AT) +
+                                    (g * R + c % R) * MS + 2 * tq;
                 float s[MT][4], top = -INFINITY;
 #pragma unroll
                 for (int m = 0; m < MT; ++m) {
-                    const float2 u = *reinterpret_cast<const float2*>(mine + (h0 + x) * MS + m * 16 + 2 * tq);
-                    const float2 v = *reinterpret_cast<const float2*>(mine + (h0 + x) * MS + m * 16 + 2 * tq + 8);
+                    const float2 u = *reinterpret_cast<const float2*>(mine + m * 16);
+                    const float2 v = *reinterpret_cast<const float2*>(mine + m * 16 + 8);
                     s[m][0] = u.x;
                     s[m][1] = u.y;
                     s[m][2] = v.x;
@@ -392,7 +397,7 @@ __global__ void __launch_bounds__(THREADS, 1) attention_talk_mma_kernel(const Pa
 #pragma unroll
                     for (int i = 0; i < 4; ++i) {
                         const int j = j0 + m * 16 + 2 * tq + (i & 1) + (i >> 1) * 8;
-                        if (j > my_pos || j < my_lo) s[m][i] = -INFINITY;
+                        if (j > pos || j < lo) s[m][i] = -INFINITY;
                         top = fmaxf(top, s[m][i]);
                     }
                 }
@@ -400,13 +405,14 @@ __global__ void __launch_bounds__(THREADS, 1) attention_talk_mma_kernel(const Pa
                 top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, 2));
                 const float now = fmaxf(mx[a + x], top);
                 const float f = now == mx[a + x] ? 1.f : __expf(mx[a + x] - now);  // (exp(-inf) = 0 on the first keys)
+                const float from = now == -INFINITY ? 0.f : now;
                 mx[a + x] = now;
                 float sum = 0.f;
 #pragma unroll
                 for (int m = 0; m < MT; ++m) {
 #pragma unroll
                     for (int i = 0; i < 4; ++i) {
-                        s[m][i] = s[m][i] == -INFINITY ? 0.f : __expf(s[m][i] - now);
+                        s[m][i] = __expf(s[m][i] - from);  // (exp(-inf) = 0 for keys that are not seen)
                         sum += s[m][i];
                     }
                     pb[x][m][0] = pack_bf16(s[m][0], s[m][1]);
@@ -424,7 +430,7 @@ __global__ void __launch_bounds__(THREADS, 1) attention_talk_mma_kernel(const Pa
                     }
                 }
             }
-            const bf16* vg = vs + (h0 / R) * BN * VS + ((lane & 7) + (lane >> 4) * 8) * VS + ((lane >> 3) & 1) * 8;
+            const bf16* vg = vs + g * BN * VS + ((lane & 7) + (lane >> 4) * 8) * VS + ((lane >> 3) & 1) * 8;
 #pragma unroll
             for (int n = 0; n < ET; ++n)
 #pragma unroll
@@ -438,28 +444,29 @@ __global__ void __launch_bounds__(THREADS, 1) attention_talk_mma_kernel(const Pa
     }
 
 #pragma unroll
-    for (int a = 0; a < HW; ++a) {
+    for (int a = 0; a < UW; ++a) {
         den[a] += __shfl_xor_sync(0xffffffffu, den[a], 1);
         den[a] += __shfl_xor_sync(0xffffffffu, den[a], 2);
     }
     if (SPLIT) {
         cp_async_wait_all();  // (the queries, when the slice held no key)
 #pragma unroll
-        for (int a = 0; a < HW; ++a) {
-            const int h = warp * HW + a;
-            if (h >= H) break;
+        for (int a = 0; a < UW; ++a) {
+            const int u = warp * UW + a;
+            if (u >= NU) break;
+            const int g = u / UPG, c0 = u % UPG * 8;
             const size_t base = (size_t)sp * p.n_rows + row0 + tile0;
-            if (eb == 0 && tq == 0 && gq < nq) {
-                float* st = p.stats + ((base + gq) * H + h) * 2;
+            if (eb == 0 && tq == 0 && (c0 + gq) / R < nq) {
+                float* st = p.stats + ((base + (c0 + gq) / R) * H + g * R + (c0 + gq) % R) * 2;
                 st[0] = mx[a];
                 st[1] = den[a];
             }
             if (n_tiles == 0) continue;
 #pragma unroll
             for (int i = 0; i < 2; ++i) {
-                const int qi = 2 * tq + i;
-                if (qi >= nq) continue;
-                float* dst = p.part + ((base + qi) * H + h) * E + eb * EB;
+                const int c = c0 + 2 * tq + i;
+                if (c / R >= nq) continue;
+                float* dst = p.part + ((base + c / R) * H + g * R + c % R) * E + eb * EB;
 #pragma unroll
                 for (int n = 0; n < ET; ++n) {
                     dst[n * 16 + gq] = o[a][n][i];
@@ -473,12 +480,13 @@ __global__ void __launch_bounds__(THREADS, 1) attention_talk_mma_kernel(const Pa
     __syncthreads();
     bf16* st = reinterpret_cast<bf16*>(smem_raw) + warp * 8 * VS;
 #pragma unroll
-    for (int a = 0; a < HW; ++a) {
-        const int h = warp * HW + a;
-        if (h >= H) break;
+    for (int a = 0; a < UW; ++a) {
+        const int u = warp * UW + a;
+        if (u >= NU) break;
+        const int g = u / UPG, c0 = u % UPG * 8;
         float f = den[a] > 0.f ? 1.f / den[a] : 0.f;
-        if (p.gate && gq < nq) {
-            const float z = __bfloat162float(p.gate[(size_t)(row0 + tile0 + gq) * p.gate_stride + h]);
+        if (p.gate && (c0 + gq) / R < nq) {
+            const float z = __bfloat162float(p.gate[(size_t)(row0 + tile0 + (c0 + gq) / R) * p.gate_stride + g * R + (c0 + gq) % R]);
             f *= 1.f / (1.f + expf(-z));
         }
         const float f0 = __shfl_sync(0xffffffffu, f, 8 * tq), f1 = __shfl_sync(0xffffffffu, f, 8 * tq + 4);
@@ -491,10 +499,11 @@ __global__ void __launch_bounds__(THREADS, 1) attention_talk_mma_kernel(const Pa
         }
         __syncwarp();
         constexpr int OC = EB / 8;
-        for (int c = lane; c < nq * OC; c += 32) {
-            const int qi = c / OC, part = c % OC;
-            *reinterpret_cast<uint4*>(p.out + (size_t)(row0 + tile0 + qi) * p.out_stride + h * E + eb * EB + part * 8) =
-                *reinterpret_cast<const uint4*>(st + qi * VS + part * 8);
+        for (int x = lane; x < 8 * OC; x += 32) {
+            const int col = x / OC, part = x % OC, qi = (c0 + col) / R;
+            if (qi < nq)
+                *reinterpret_cast<uint4*>(p.out + (size_t)(row0 + tile0 + qi) * p.out_stride + (g * R + (c0 + col) % R) * E +
+                                          eb * EB + part * 8) = *reinterpret_cast<const uint4*>(st + col * VS + part * 8);
         }
         __syncwarp();
     }
@@ -544,12 +553,45 @@ __global__ void attention_talk_merge_kernel(const float* __restrict__ stats, con
         out[(size_t)row * out_stride + h * E + c] =
             __float2bfloat16_rn((((sh_o[0][c] + sh_o[1][c]) + sh_o[2][c]) + sh_o[3][c]) * f);
 }
+
+template <int BQ>
+int launch_talk(const Params& p, int n_entries, int max_rows, cudaStream_t s) {
+    using C = Cfg<BQ>;
+    if (!C::FITS) return IB_ERR_UNSUPPORTED;
+    if ((long long)p.splits * C::ES > 65535) return IB_ERR_TOO_LARGE;
+    if (p.splits > 1 && (p.slice_len <= 0 || p.slice_len % C::BN)) return IB_ERR_BAD_ARG;
+    static bool configured = false;
+    if (!configured) {
+        cudaError_t ce = cudaFuncSetAttribute(attention_talk_mma_kernel<BQ, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM);
+        if (ce == cudaSuccess)
+            ce = cudaFuncSetAttribute(attention_talk_mma_kernel<BQ, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM);
+        if (ce != cudaSuccess) return (int)ce;
+        configured = true;
+    }
+    const dim3 grid((max_rows + BQ - 1) / BQ, n_entries, C::ES * p.splits);
+    cudaError_t le = p.splits == 1
+        ? launch_kernel(attention_talk_mma_kernel<BQ, false>, grid, dim3(C::THREADS), C::SMEM, s, p)
+        : launch_kernel(attention_talk_mma_kernel<BQ, true>, grid, dim3(C::THREADS), C::SMEM, s, p);
+    if (le != cudaSuccess) return (int)le;
+    if (p.splits > 1) {
+        le = launch_kernel(attention_talk_merge_kernel, dim3((unsigned)((long long)p.n_rows * H)), dim3(128), 0, s,
+                           (const float*)p.stats, (const float*)p.part, p.gate, p.gate_stride, p.out, p.out_stride, p.splits,
+                           p.n_rows);
+        if (le != cudaSuccess) return (int)le;
+    }
+    IB_LAUNCH_CHECK();
+    return IB_OK;
+}
 }  // namespace
 
-// What was compiled: sizes, keys of a tile, blocks of the values, whether the shared memory suffices.
-IB_EXPORT int ib_attention_talk_mma_info(int what) {
-    const int v[] = {H, G, D, E, BN, ES, FITS ? 1 : 0, SMEM};
-    return what >= 0 && what < 8 ? v[what] : -1;
+// What was compiled: sizes, then for eight queries a CTA (few = 0) or for few rows an entry (few = 1) the queries
+// of a CTA, the keys of a tile, the blocks of the values, the bytes of shared memory, whether it can run.
+IB_EXPORT int ib_attention_talk_mma_info(int what, int few) {
+    using A = Cfg<8>;
+    using B = Cfg<BQ_FEW>;
+    const int v[] = {H, G, D, E, few ? BQ_FEW : 8, few ? B::BN : A::BN, few ? B::ES : A::ES, few ? B::SMEM : A::SMEM,
+                     (few ? B::FITS : A::FITS) ? 1 : 0};
+    return what >= 0 && what < 9 ? v[what] : -1;
 }
 
 IB_EXPORT long long ib_attention_talk_mma_scratch_bytes(int n_rows, int splits) {
@@ -558,32 +600,25 @@ IB_EXPORT long long ib_attention_talk_mma_scratch_bytes(int n_rows, int splits) 
 
 // q rows begin with H * D queries (row stride q_stride), out rows hold H * E (stride out_stride); talk float32 [H, H]
 // whose values are exact in bf16, or null; temp float32 [H] or null; gate bf16, one per (row, head), or null.
-// max_rows: an upper bound on the rows of any entry (the grid's width).  splits > 1: the keys from the first
-// that a CTA's first query sees, rounded down to the key tile, in slices of `slice_len` (a multiple of the key
-// tile; together they must reach the last query) over that many CTAs, through `scratch`; n_rows: all rows.
+// max_rows: an upper bound on the rows of any entry (the grid's width); few: the variant for few rows an entry.
+// splits > 1: the keys from the first that a CTA's first query sees, rounded down to the key tile, in slices of
+// `slice_len` (a multiple of the key tile; together they must reach the last query) over that many CTAs, through
+// `scratch`; n_rows: all rows.
 IB_EXPORT int ib_attention_talk_mma(const void* q, int q_stride, const void* k_pool, const void* v_pool, void* out,
                                     int out_stride, const float* talk, const float* temp, const void* gate,
                                     int gate_stride, const int* cu_rows, const int* positions, const int* block_tables,
                                     int max_blocks, int n_entries, int max_rows, int page_size, int num_pages,
-                                    float scale, int chunk, int window, unsigned* err, int n_rows, int splits,
+                                    float scale, int chunk, int window, unsigned* err, int n_rows, int few, int splits,
                                     int slice_len, void* scratch, long long scratch_bytes, void* stream) {
     if (n_entries <= 0 || max_rows <= 0 || n_rows <= 0) return IB_OK;
     if (!q || !k_pool || !v_pool || !out || !cu_rows || !positions || !block_tables || !err) return IB_ERR_BAD_ARG;
     if (page_size <= 0 || num_pages <= 0 || max_blocks <= 0 || chunk < 0 || window < 0 || splits < 1 ||
         q_stride < H * D || out_stride < H * E || (gate && gate_stride < H))
         return IB_ERR_BAD_ARG;
-    if (!FITS || q_stride % 8 || out_stride % 8 || (((uintptr_t)q | (uintptr_t)k_pool | (uintptr_t)v_pool | (uintptr_t)out) & 15))
+    if (q_stride % 8 || out_stride % 8 || (((uintptr_t)q | (uintptr_t)k_pool | (uintptr_t)v_pool | (uintptr_t)out) & 15))
         return IB_ERR_UNSUPPORTED;
-    if (n_entries > 65535 || (long long)splits * ES > 65535 || (long long)num_pages * G * page_size > 0x7fffffffLL)
-        return IB_ERR_TOO_LARGE;
-    static bool configured = false;
-    if (!configured) {
-        cudaError_t ce = cudaFuncSetAttribute(attention_talk_mma_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
-        if (ce == cudaSuccess)
-            ce = cudaFuncSetAttribute(attention_talk_mma_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
-        if (ce != cudaSuccess) return (int)ce;
-        configured = true;
-    }
+    if (n_entries > 65535 || (long long)num_pages * G * page_size > 0x7fffffffLL) return IB_ERR_TOO_LARGE;
+    if (splits > 1 && (!scratch || scratch_bytes < ib_attention_talk_mma_scratch_bytes(n_rows, splits))) return IB_ERR_BAD_ARG;
     Params p;
     p.q = (const bf16*)q;
     p.k_pool = (const bf16*)k_pool;
@@ -608,26 +643,8 @@ IB_EXPORT int ib_attention_talk_mma(const void* q, int q_stride, const void* k_p
     p.n_rows = n_rows;
     p.scale = scale;
     p.err = err;
-    p.stats = nullptr;
-    p.part = nullptr;
-    cudaStream_t s = (cudaStream_t)stream;
-    const dim3 grid((max_rows + BQ - 1) / BQ, n_entries, ES * splits);
-    cudaError_t le;
-    if (splits == 1) {
-        le = launch_kernel(attention_talk_mma_kernel<false>, grid, dim3(THREADS), SMEM, s, p);
-        if (le != cudaSuccess) return (int)le;
-        IB_LAUNCH_CHECK();
-        return IB_OK;
-    }
-    if (!scratch || slice_len <= 0 || slice_len % BN || scratch_bytes < ib_attention_talk_mma_scratch_bytes(n_rows, splits))
-        return IB_ERR_BAD_ARG;
     p.stats = (float*)scratch;
-    p.part = p.stats + (size_t)splits * n_rows * H * 2;
-    le = launch_kernel(attention_talk_mma_kernel<true>, grid, dim3(THREADS), SMEM, s, p);
-    if (le != cudaSuccess) return (int)le;
-    le = launch_kernel(attention_talk_merge_kernel, dim3((unsigned)((long long)n_rows * H)), dim3(128), 0, s,
-                       (const float*)p.stats, (const float*)p.part, p.gate, gate_stride, p.out, out_stride, splits, n_rows);
-    if (le != cudaSuccess) return (int)le;
-    IB_LAUNCH_CHECK();
-    return IB_OK;
+    p.part = scratch ? p.stats + (size_t)splits * n_rows * H * 2 : nullptr;
+    return few ? launch_talk<BQ_FEW>(p, n_entries, max_rows, (cudaStream_t)stream)
+               : launch_talk<8>(p, n_entries, max_rows, (cudaStream_t)stream);
 }

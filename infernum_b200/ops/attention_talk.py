@@ -7,8 +7,9 @@ sizes multiples of 16, at most 256; all heads of eight queries and one tile of k
 in an SM's shared memory) or ``rt.options["attention"] == "plain"``; the caller
 then takes the plain 32-bit kernel (``core.attention_talk``).
 
-A CTA takes eight rows of an entry with all heads.  A step of few rows would
-leave SMs idle: ``choose_splits`` then cuts the keys in slices over several CTAs.
+A CTA takes eight rows of an entry with all heads, or - when no entry has more
+rows than fill eight (row, head) columns of a key/value head, decoded tokens - those.
+A step of few rows would leave SMs idle: ``choose_splits`` then cuts the keys in slices over several CTAs.
 The plan and the scratch buffer are worked out once per step and kept in
 ``ctx.scratch``.
 """
@@ -31,7 +32,7 @@ _libs: Dict[Tuple[int, int, int, int], ctypes.CDLL] = {}
 PLAIN_SMEM = 220 * 1024  # what the plain kernel may hold of a row, in bytes
 SMEM_MAX = 227 * 1024
 SM_COUNT_FALLBACK = 148
-ROW_TILE, MAX_SPLITS = 8, 64
+MAX_SPLITS = 64
 
 
 def plain_floats(heads: int, dim: int, vdim: int) -> int:
@@ -39,34 +40,41 @@ def plain_floats(heads: int, dim: int, vdim: int) -> int:
     return heads * (dim + vdim) + heads * 2 * 33 + 3 * heads
 
 
-def layout(heads: int, kv_heads: int, dim: int, vdim: int) -> Tuple[int, int, int]:
-    """(keys of a tile, blocks of the values, bytes of shared memory) of the kernel compiled for
-    these sizes; restates the constants at the head of ``attention_talk_mma.cu``."""
-    warps = 8 if heads >= 8 else 4
-    per_warp = -(-heads // warps)
+def queries_of_few(heads: int, kv_heads: int) -> int:
+    """Queries of a CTA in the variant for few rows: as many as fill eight columns of a key/value head."""
+    return max(1, 8 // (heads // kv_heads))
+
+
+def layout(heads: int, kv_heads: int, dim: int, vdim: int, queries: int) -> Tuple[int, int, int, bool]:
+    """(keys of a tile, blocks of the values, bytes of shared memory, whether it can run) of the kernel
+    for these sizes with this many queries a CTA; restates ``Cfg`` in ``attention_talk_mma.cu``."""
+    per_kv = heads // kv_heads
+    units_of_kv = -(-queries * per_kv // 8)
+    units = kv_heads * units_of_kv
+    warps = 16 if units >= 16 and queries == 8 else (8 if units >= 8 else 4)
+    mine = -(-units // warps)
+    most = 256 if warps == 16 else 512
     padded = -(-heads // 16) * 16
-    block = next((e for e in range(vdim, 15, -16) if vdim % e == 0 and per_warp * e <= 512), 16)
+    block = next((e for e in range(vdim, 15, -16) if vdim % e == 0 and mine * e <= most), 16)
 
     def smem(bn: int) -> int:
-        plane, mix = bn * (padded + 8) * 2, heads * (bn + 8) * 4
-        alias = bn // 8 * (padded // 16) * 6 <= 48
-        region = (max(3 * plane, mix) if alias else 3 * plane + mix)
-        region = -(-region // 128) * 128 + 32
-        total = 8 * heads * (dim + 8) * 2 + kv_heads * bn * (dim + 8) * 2 + 2 * kv_heads * bn * (block + 8) * 2 \
-            + 8 * region + padded * (padded + 8) * 2 + -(-heads // 4) * 16 + 3 * bn * 4
+        region = -(-(3 * bn * (padded + 8) * 2 + heads * (bn + 8) * 4) // 128) * 128 + 32
+        total = units * 8 * (dim + 8) * 2 + kv_heads * bn * ((dim + 8) + (block + 8)) * 2 + queries * region \
+            + padded * (padded + 8) * 2 + -(-heads // 4) * 16 + 3 * bn * 4
         return max(total, warps * 8 * (block + 8) * 2)
 
     bn = 32 if smem(32) <= SMEM_MAX else 16
-    return bn, vdim // block, smem(bn)
+    if queries != 8 or queries_of_few(heads, kv_heads) == 8:
+        # few rows: as many keys as leave room for a second CTA on the SM, if any do
+        half = SMEM_MAX // 2 - 1024
+        bn = 32 if smem(32) <= half else (16 if smem(16) <= half else bn)
+    return bn, vdim // block, smem(bn), smem(bn) <= SMEM_MAX and mine * block <= most
 
 
 def supported(heads: int, kv_heads: int, dim: int, vdim: int) -> bool:
-    if dim % 16 or vdim % 16 or not 16 <= dim <= 256 or not 16 <= vdim <= 256 or heads % kv_heads:
+    if dim % 16 or vdim % 16 or not 16 <= dim <= 256 or not 16 <= vdim <= 256 or heads % kv_heads or heads > 96:
         return False
-    bn, blocks, smem = layout(heads, kv_heads, dim, vdim)
-    per_warp = -(-heads // (8 if heads >= 8 else 4))
-    # the exchange keeps a query's planes of one piece of heads after the other in registers
-    return smem <= SMEM_MAX and per_warp * (vdim // blocks) <= 512 and heads <= 96
+    return all(layout(heads, kv_heads, dim, vdim, n)[3] for n in (8, queries_of_few(heads, kv_heads)))
 
 
 def lib_for(heads: int, kv_heads: int, dim: int, vdim: int) -> ctypes.CDLL:
@@ -78,23 +86,23 @@ def lib_for(heads: int, kv_heads: int, dim: int, vdim: int) -> ctypes.CDLL:
         lib.ib_attention_talk_mma.argtypes = [
             _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int,
             _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_void_p,
-            _c_int, _c_int, _c_int, _c_void_p, _c_ll, _c_void_p]
+            _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_ll, _c_void_p]
         lib.ib_attention_talk_mma.restype = _c_int
         lib.ib_attention_talk_mma_scratch_bytes.argtypes = [_c_int, _c_int]
         lib.ib_attention_talk_mma_scratch_bytes.restype = _c_ll
-        lib.ib_attention_talk_mma_info.argtypes = [_c_int]
+        lib.ib_attention_talk_mma_info.argtypes = [_c_int, _c_int]
         lib.ib_attention_talk_mma_info.restype = _c_int
-        built = tuple(lib.ib_attention_talk_mma_info(i) for i in range(8))
-        bn, blocks, smem = layout(*key)
-        if built != (*key, bn, blocks, 1, smem):
-            raise KernelError(f"the module for heads and sizes {key} was built as {built}")
+        for few, queries in ((0, 8), (1, queries_of_few(heads, kv_heads))):
+            built = [lib.ib_attention_talk_mma_info(i, few) for i in range(9)]
+            if built != [*key, queries, *(int(v) for v in layout(*key, queries))]:
+                raise KernelError(f"the module for heads and sizes {key} was built as {built}")
         _libs[key] = lib
     return lib
 
 
-def key_span(max_kv_len: int, max_rows: int, chunk: int, window: int, bn: int) -> int:
+def key_span(max_kv_len: int, max_rows: int, chunk: int, window: int, bn: int, queries: int = 8) -> int:
     """The most keys between the first that a row tile reads, rounded down to a key tile, and its last row."""
-    span, behind = max_kv_len, min(max_rows, ROW_TILE) - 1
+    span, behind = max_kv_len, min(max_rows, queries) - 1
     if chunk > 0:
         span = min(span, chunk + behind)
     if window > 0:
@@ -102,10 +110,11 @@ def key_span(max_kv_len: int, max_rows: int, chunk: int, window: int, bn: int) -
     return span + bn - 1
 
 
-def choose_splits(max_rows: int, n_entries: int, blocks: int, span: int, bn: int, slots: int) -> Tuple[int, int]:
+def choose_splits(max_rows: int, n_entries: int, blocks: int, span: int, bn: int, slots: int,
+                  queries: int = 8) -> Tuple[int, int]:
     """(slices of the keys, keys per slice): one when the row tiles fill the SMs' ``slots`` for CTAs or there
     are few keys, else as many as fill them about twice, each of at least two tiles of keys."""
-    ctas = max(1, -(-max_rows // ROW_TILE) * n_entries * blocks)
+    ctas = max(1, -(-max_rows // queries) * n_entries * blocks)
     want = min(-(-2 * slots // ctas), span // (2 * bn), MAX_SPLITS, 65535 // blocks)
     if ctas >= slots or want < 2:
         return 1, 0
@@ -129,19 +138,24 @@ def run(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, out: torch.
     key = ("talk_plan", n_heads, nkv, dim, vdim, chunk, window)
     plan = ctx.scratch.get(key) if hasattr(ctx, "scratch") else None
     if plan is None:
-        bn, blocks, smem = layout(n_heads, nkv, dim, vdim)
+        # entries whose (row, head) pairs fill no more than eight columns of a key/value head
+        few = int(ctx.max_rows_per_entry <= queries_of_few(n_heads, nkv))
+        if rt.options.get("talk_few") is not None:
+            few = int(rt.options["talk_few"])
+        queries = queries_of_few(n_heads, nkv) if few else 8
+        bn, blocks, smem, _ = layout(n_heads, nkv, dim, vdim, queries)
         sms = rt.options.get("sm_count") or SM_COUNT_FALLBACK
         forced = rt.options.get("talk_splits")
-        span = key_span(ctx.max_kv_len, ctx.max_rows_per_entry, chunk, window, bn)
+        span = key_span(ctx.max_kv_len, ctx.max_rows_per_entry, chunk, window, bn, queries)
         if forced:
             slice_len = -(-math.ceil(span / forced) // bn) * bn
-            plan = (-(-span // slice_len), slice_len)
+            plan = (-(-span // slice_len), slice_len, few)
         else:
-            plan = choose_splits(ctx.max_rows_per_entry, ctx.n_entries, blocks, span, bn,
-                                 sms * max(1, min(2, SMEM_MAX // smem)))
+            plan = (*choose_splits(ctx.max_rows_per_entry, ctx.n_entries, blocks, span, bn,
+                                   sms * (2 if 2 * (smem + 1024) <= SMEM_MAX else 1), queries), few)
         if hasattr(ctx, "scratch"):
             ctx.scratch[key] = plan
-    splits, slice_len = plan
+    splits, slice_len, few = plan
     N = q.shape[0]
     scratch_ptr, scratch_bytes = None, 0
     if splits > 1:
@@ -156,7 +170,7 @@ def run(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, out: torch.
         q.data_ptr(), q.stride(0), k_pool.data_ptr(), v_pool.data_ptr(), out.data_ptr(), out.stride(0),
         core._ptr(talk), core._ptr(temp), core._ptr(gate), gate.stride(0) if gate is not None else 0,
         ctx.cu_rows.data_ptr(), ctx.positions.data_ptr(), tables.data_ptr(), tables.shape[1], ctx.n_entries,
-        ctx.max_rows_per_entry, page_size, num_pages, float(scale), int(chunk), int(window), rt.err.data_ptr(), N, splits,
-        slice_len, scratch_ptr, scratch_bytes, core.stream_ptr(q))
+        ctx.max_rows_per_entry, page_size, num_pages, float(scale), int(chunk), int(window), rt.err.data_ptr(), N, few,
+        splits, slice_len, scratch_ptr, scratch_bytes, core.stream_ptr(q))
     core.check(code, "attention_talk_mma")
     return True

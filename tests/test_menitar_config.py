@@ -215,9 +215,11 @@ def test_slices_of_the_keys():
 
 
 def test_sizes_with_a_tensor_core_variant():
-    from infernum_b200.ops.attention_talk import layout, supported
+    from infernum_b200.ops.attention_talk import layout, queries_of_few, supported
     assert supported(16, 4, 64, 64) and supported(32, 8, 128, 128) and supported(5, 5, 64, 16) and supported(1, 1, 16, 256)
     assert not supported(4, 2, 24, 32) and not supported(4, 2, 32, 40) and not supported(64, 64, 128, 128)
     for h, g, d, e in [(16, 4, 64, 64), (12, 4, 16, 32), (10, 1, 16, 80), (32, 8, 128, 128)]:
-        bn, blocks, smem = layout(h, g, d, e)
-        assert bn in (16, 32) and e % (blocks * 16) == 0 and smem <= 227 * 1024
+        for queries in (8, queries_of_few(h, g)):
+            bn, blocks, smem, fits = layout(h, g, d, e, queries)
+            assert fits and bn in (16, 32) and e % (blocks * 16) == 0 and smem <= 227 * 1024
+    assert [queries_of_few(h, g) for h, g in ((32, 8), (8, 8), (16, 1), (12, 4))] == [2, 8, 1, 2]

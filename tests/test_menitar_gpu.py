@@ -455,6 +455,20 @@ def test_exchanged_scores_on_the_tensor_cores(H, G, d, e, page, chunk):
         rt.options["talk_splits"] = splits
         check_talk(torch.bfloat16, H, G, d, e, page, chunk, lens, few, run, 2e-2)
         check_talk(torch.bfloat16, H, G, d, e, page, chunk, lens, rows, run, 2e-2, window=37)
+    # the variant for few rows an entry: as many as fill eight columns of a key/value head, and one
+    for n in {1, attention_talk.queries_of_few(H, G)}:
+        least = [min(n, t, r) if r else 0 for t, r in zip(lens, few)]
+        for splits in (1, 2, 20):
+            rt.options["talk_splits"] = splits
+            check_talk(torch.bfloat16, H, G, d, e, page, chunk, lens, least, run, 2e-2)
+            check_talk(torch.bfloat16, H, G, d, e, page, chunk, lens, least, run, 2e-2, window=37)
+        check_talk(torch.bfloat16, H, G, d, e, page, chunk, lens, least, run, 2e-2, bare=True)
+        rt.options["talk_few"] = 0  # and the other one on the same rows
+        check_talk(torch.bfloat16, H, G, d, e, page, chunk, lens, least, run, 2e-2)
+        del rt.options["talk_few"]
+    rt.options["talk_few"] = 1  # and on rows that take several of its CTAs
+    check_talk(torch.bfloat16, H, G, d, e, page, chunk, lens, few, run, 2e-2)
+    del rt.options["talk_few"]
     del rt.options["talk_splits"]
     check_talk(torch.bfloat16, H, G, d, e, page, chunk, lens, few, run, 2e-2)
     assert int(rt.err.item()) == 0
