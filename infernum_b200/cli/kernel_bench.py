@@ -173,12 +173,11 @@ def main(argv=None) -> int:
         cases = [_attention_case(batch, rows, kv_len, nh, nkv, hd, args.page_size, dev) for _ in range(3 if decode else 1)]
         outs = torch.empty(batch * rows, nh * hd, dtype=torch.bfloat16, device=dev)
         talk = (torch.randn(nh, nh, device=dev) * nh ** -0.5).bfloat16().float().contiguous()
-        temp = torch.rand(nh, device=dev)
         gate = torch.randn(batch * rows, nh, device=dev).to(torch.bfloat16)
         if args.splits:
             rt.options["talk_splits"] = args.splits
         fns = [lambda q=q, kp=kp, vp=vp, tables=tables, ctx=ctx: attention_talk.run(
-            q, kp, vp, outs, ctx, tables, nh, hd ** -0.5, talk, temp, gate, args.chunk, 0, rt)
+            q, kp, vp, outs, ctx, tables, nh, talk, gate, args.chunk, 0, rt)
             for q, kp, vp, tables, ctx in cases]
         us = _time(fns, args.reps, args.warmup, not args.no_graph)
         c = args.chunk
@@ -243,8 +242,9 @@ def main(argv=None) -> int:
         ent = torch.zeros(T, dtype=torch.int32, device=dev)
         tables = torch.arange(pages, dtype=torch.int32, device=dev).view(1, pages)
         inv = torch.rand(args.rotary // 2, device=dev)
-        qw, kw = torch.ones(nh * hd, device=dev), torch.ones(nkv * hd, device=dev)
-        fns = [lambda x=x: core.qk_row_norm_append(x, qw, kw, 1e-5, inv, args.rotary, nh, nkv, hd, hd, pos, ent, tables, kp,
+        qw, kw = (torch.ones(n * hd, device=dev).to(torch.bfloat16) for n in (nh, nkv))
+        qs = torch.ones(nh, device=dev)
+        fns = [lambda x=x: core.qk_row_norm_append(x, qw, kw, 1e-5, qs, inv, args.rotary, nh, nkv, hd, hd, pos, ent, tables, kp,
                                                    vp, rt.err) for x in xs]
         us = _time(fns, args.reps, args.warmup, not args.no_graph)
         nbytes = T * (nh + 2 * nkv) * hd * 2 * 2

@@ -3,8 +3,7 @@
 //
 // With H query heads over G key/value heads (head a reads key/value head a / (H / G)):
 //
-//   r_g(i, j) = (q_g(i) . k_g(j)) * scale * temp_g
-//   s_h(i, j) = sum_g talk[h, g] r_g(i, j)            (all H heads, across key/value heads)
+//   s_h(i, j) = sum_g talk[h, g] (q_g(i) . k_g(j))    (all H heads, across key/value heads)
 //   o_h(i)    = sum_j softmax_j(s_h(i, .)) v_h(j) * sigmoid(gate_h(i))
 //
 // Query i sees keys j <= i; with `chunk` > 0 only those of its own run of `chunk` positions
@@ -14,7 +13,8 @@
 //   qk_row_norm_append  rows [q : H d | k : G d | v : G e | ...] as projected: all of q is divided by
 //                       its one root mean square and multiplied by a weight of H d values, k likewise
 //                       (each when it has a weight); then the first rd dimensions of every head are
-//                       rotated (element i with i + rd/2, angle = position * f_i).  Queries are
+//                       rotated (element i with i + rd/2, angle = position * f_i); query head h is
+//                       multiplied by q_scale[h] (what scales its scores).  Queries are
 //                       written back in place, keys and values to their pages.  32-bit, one rounding.
 //   attention_talk      one CTA per row, all heads: keys in tiles of 32 that start at absolute
 //                       multiples of 32; the heads' scores, their combination, the running softmax
@@ -24,9 +24,10 @@
 
 using namespace ib;
 
-template <typename T>
-__global__ void qk_row_norm_append_kernel(T* __restrict__ x, int x_stride, const float* __restrict__ qw,
-                                          const float* __restrict__ kw, float eps, const float* __restrict__ inv_freq,
+template <typename T, typename TW>
+__global__ void qk_row_norm_append_kernel(T* __restrict__ x, int x_stride, const TW* __restrict__ qw,
+                                          const TW* __restrict__ kw, float eps, const float* __restrict__ q_scale,
+                                          const float* __restrict__ inv_freq,
                                           int rd, const int* __restrict__ positions, const int* __restrict__ row_entry,
                                           const int* __restrict__ block_tables, int max_blocks, T* __restrict__ k_pool,
                                           T* __restrict__ v_pool, int nh, int nkv, int d, int e, int page_size,
@@ -66,20 +67,20 @@ __global__ void qk_row_norm_append_kernel(T* __restrict__ x, int x_stride, const
         const int head = it / per_head, i = it % per_head;
         const bool is_q = head < nh;
         const int base = head * d;  // (keys follow the queries)
-        const float f = is_q ? fq : fk;
-        const float* w = is_q ? (qw ? qw + base : nullptr) : (kw ? kw + base - qc : nullptr);
+        const float f = is_q ? fq * (q_scale ? q_scale[head] : 1.f) : fk;
+        const TW* w = is_q ? (qw ? qw + base : nullptr) : (kw ? kw + base - qc : nullptr);
         T* dst = is_q ? xr + base : k_pool + (at + (size_t)(head - nh) * page_size) * d;
         if (!is_q && bad) continue;
         if (i < half) {
-            const float a = to_f32(xr[base + i]) * f * (w ? w[i] : 1.f);
-            const float b = to_f32(xr[base + i + half]) * f * (w ? w[i + half] : 1.f);
+            const float a = to_f32(xr[base + i]) * f * (w ? to_f32(w[i]) : 1.f);
+            const float b = to_f32(xr[base + i + half]) * f * (w ? to_f32(w[i + half]) : 1.f);
             float sn, cs;
             sincosf((float)pos * inv_freq[i], &sn, &cs);
             dst[i] = from_f32<T>(a * cs - b * sn);
             dst[i + half] = from_f32<T>(b * cs + a * sn);
         } else {
             const int c = i + half;
-            dst[c] = from_f32<T>(to_f32(xr[base + c]) * f * (w ? w[c] : 1.f));
+            dst[c] = from_f32<T>(to_f32(xr[base + c]) * f * (w ? to_f32(w[c]) : 1.f));
         }
     }
 }
@@ -100,6 +101,7 @@ __device__ __forceinline__ uint4 pack8(const float (&v)[8]) {
     for (int i = 0; i < 4; ++i) p[i] = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
     return raw;
 }
+__device__ __forceinline__ void load8(const bf16* p, float (&v)[8]) { unpack8(*reinterpret_cast<const uint4*>(p), v); }
 __device__ __forceinline__ void load8(const float* p, float (&v)[8]) {
     *reinterpret_cast<float4*>(v) = *reinterpret_cast<const float4*>(p);
     *reinterpret_cast<float4*>(v + 4) = *reinterpret_cast<const float4*>(p + 4);
@@ -110,8 +112,9 @@ __device__ __forceinline__ void load8(const float* p, float (&v)[8]) {
 // thread keeps the first ROW_HOLD of its 16-byte pieces in registers between the two passes.
 constexpr int ROW_MAX_PAIRS = 256;
 constexpr int ROW_HOLD = 3;
-__global__ void qk_row_norm_append_vec8_kernel(bf16* __restrict__ x, int x_stride, const float* __restrict__ qw,
-                                               const float* __restrict__ kw, float eps,
+template <typename TW>
+__global__ void qk_row_norm_append_vec8_kernel(bf16* __restrict__ x, int x_stride, const TW* __restrict__ qw,
+                                               const TW* __restrict__ kw, float eps, const float* __restrict__ q_scale,
                                                const float* __restrict__ inv_freq, int rd,
                                                const int* __restrict__ positions, const int* __restrict__ row_entry,
                                                const int* __restrict__ block_tables, int max_blocks,
@@ -199,8 +202,8 @@ __global__ void qk_row_norm_append_vec8_kernel(bf16* __restrict__ x, int x_strid
         const int head = item / per_head, p = item % per_head;
         const bool is_q = head < nh;
         if (!is_q && bad) return;
-        const float f = is_q ? fq : fk;
-        const float* w = is_q ? (qw ? qw + head * d : nullptr) : (kw ? kw + (head - nh) * d : nullptr);
+        const float f = is_q ? fq * (q_scale ? q_scale[head] : 1.f) : fk;
+        const TW* w = is_q ? (qw ? qw + head * d : nullptr) : (kw ? kw + (head - nh) * d : nullptr);
         bf16* dst = is_q ? xr + head * d : k_pool + (at + (size_t)(head - nh) * page_size) * d;
         const int c = p < rot ? p << 3 : rd + ((p - rot) << 3);
         float a[8], wv[8];
@@ -243,38 +246,41 @@ __global__ void qk_row_norm_append_vec8_kernel(bf16* __restrict__ x, int x_strid
     }
 }
 
-// x rows: [nh * d | nkv * d | nkv * e | anything]; qw float32 [nh * d] / kw float32 [nkv * d], or null: not normed.
-IB_EXPORT int ib_qk_row_norm_append(void* x, int x_stride, int dtype, const float* qw, const float* kw, float eps,
-                                    const float* inv_freq, int rd, const int* positions, const int* row_entry,
-                                    const int* block_tables, int max_blocks, void* k_pool, void* v_pool, int n_rows,
-                                    int nh, int nkv, int d, int e, int page_size, int num_pages, unsigned* err,
-                                    void* stream) {
+// x rows: [nh * d | nkv * d | nkv * e | anything]; qw [nh * d] / kw [nkv * d] of type w_dtype (0 float32, 1 bf16), or
+// null: not normed; q_scale float32 [nh] or null.
+IB_EXPORT int ib_qk_row_norm_append(void* x, int x_stride, int dtype, const void* qw, const void* kw, int w_dtype, float eps,
+                                    const float* q_scale, const float* inv_freq, int rd, const int* positions,
+                                    const int* row_entry, const int* block_tables, int max_blocks, void* k_pool,
+                                    void* v_pool, int n_rows, int nh, int nkv, int d, int e, int page_size, int num_pages,
+                                    unsigned* err, void* stream) {
     if (n_rows <= 0) return IB_OK;
     if (!x || !positions || !row_entry || !block_tables || !k_pool || !v_pool || !err) return IB_ERR_BAD_ARG;
     if (nh <= 0 || nkv <= 0 || d <= 0 || e <= 0 || page_size <= 0 || num_pages <= 0 || max_blocks <= 0 || rd < 0 ||
-        (rd & 1) || rd > d || (rd > 0 && !inv_freq) || ((qw || kw) && !(eps > 0.f)))
+        (rd & 1) || rd > d || (rd > 0 && !inv_freq) || ((qw || kw) && !(eps > 0.f)) || w_dtype < 0 || w_dtype > 1)
         return IB_ERR_BAD_ARG;
     if (x_stride < (nh + nkv) * d + nkv * e) return IB_ERR_BAD_ARG;
     cudaStream_t s = (cudaStream_t)stream;
     cudaError_t le;
+#define IB_ROW(KERNEL, T, TW, THREADS)                                                                                   \
+    le = launch_kernel(KERNEL, dim3(n_rows), dim3(THREADS), 0, s, (T*)x, x_stride, (const TW*)qw, (const TW*)kw, eps, q_scale, \
+                       inv_freq, rd, positions, row_entry, block_tables, max_blocks, (T*)k_pool, (T*)v_pool, nh, nkv, d, e, \
+                       page_size, num_pages, err)
     if (dtype == 1 && d % 8 == 0 && e % 8 == 0 && rd % 16 == 0 && rd / 2 <= ROW_MAX_PAIRS && x_stride % 8 == 0 &&
         !(((uintptr_t)x | (uintptr_t)k_pool | (uintptr_t)v_pool | (uintptr_t)qw | (uintptr_t)kw) & 15)) {
         const int items = (nh + nkv) * ((rd >> 4) + ((d - rd) >> 3)) + nkv * (e >> 3);
         const int threads = items <= 256 ? 128 : (items <= 1024 ? 256 : 512);
-        le = launch_kernel(qk_row_norm_append_vec8_kernel, dim3(n_rows), dim3(threads), 0, s, (bf16*)x, x_stride, qw, kw,
-                           eps, inv_freq, rd, positions, row_entry, block_tables, max_blocks, (bf16*)k_pool,
-                           (bf16*)v_pool, nh, nkv, d, e, page_size, num_pages, err);
+        if (w_dtype == 0) IB_ROW(qk_row_norm_append_vec8_kernel<float>, bf16, float, threads);
+        else IB_ROW(qk_row_norm_append_vec8_kernel<bf16>, bf16, bf16, threads);
     } else if (dtype == 0) {
-        le = launch_kernel(qk_row_norm_append_kernel<float>, dim3(n_rows), dim3(256), 0, s, (float*)x, x_stride, qw, kw,
-                           eps, inv_freq, rd, positions, row_entry, block_tables, max_blocks, (float*)k_pool,
-                           (float*)v_pool, nh, nkv, d, e, page_size, num_pages, err);
+        if (w_dtype == 0) IB_ROW((qk_row_norm_append_kernel<float, float>), float, float, 256);
+        else IB_ROW((qk_row_norm_append_kernel<float, bf16>), float, bf16, 256);
     } else if (dtype == 1) {
-        le = launch_kernel(qk_row_norm_append_kernel<bf16>, dim3(n_rows), dim3(256), 0, s, (bf16*)x, x_stride, qw, kw,
-                           eps, inv_freq, rd, positions, row_entry, block_tables, max_blocks, (bf16*)k_pool,
-                           (bf16*)v_pool, nh, nkv, d, e, page_size, num_pages, err);
+        if (w_dtype == 0) IB_ROW((qk_row_norm_append_kernel<bf16, float>), bf16, float, 256);
+        else IB_ROW((qk_row_norm_append_kernel<bf16, bf16>), bf16, bf16, 256);
     } else {
         return IB_ERR_UNSUPPORTED;
     }
+#undef IB_ROW
     if (le != cudaSuccess) return (int)le;
     IB_LAUNCH_CHECK();
     return IB_OK;
@@ -283,11 +289,10 @@ IB_EXPORT int ib_qk_row_norm_append(void* x, int x_stride, int dtype, const floa
 template <typename T>
 __global__ void attention_talk_kernel(const T* __restrict__ q, int q_stride, const T* __restrict__ k_pool,
                                       const T* __restrict__ v_pool, T* __restrict__ out, int out_stride,
-                                      const float* __restrict__ talk, const float* __restrict__ temp,
-                                      const T* __restrict__ gate, int gate_stride, const int* __restrict__ positions,
+                                      const float* __restrict__ talk, const T* __restrict__ gate, int gate_stride, const int* __restrict__ positions,
                                       const int* __restrict__ row_entry, const int* __restrict__ block_tables,
                                       int max_blocks, int nh, int nkv, int d, int e, int page_size, int num_pages,
-                                      float scale, int chunk, int window, unsigned* __restrict__ err) {
+                                      int chunk, int window, unsigned* __restrict__ err) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ float sm[];
@@ -333,8 +338,6 @@ __global__ void attention_talk_kernel(const T* __restrict__ q, int q_stride, con
                 const T* kp = k_pool + (size_t)(at + (long long)(h / R) * page_size) * d;
                 const float* qh = qs + h * d;
                 for (int c = 0; c < d; ++c) a = fmaf(qh[c], to_f32(kp[c]), a);
-                a *= scale;
-                if (temp) a *= temp[h];
             }
             raw[h * SS + t] = a;
         }
@@ -390,12 +393,12 @@ __global__ void attention_talk_kernel(const T* __restrict__ q, int q_stride, con
 }
 
 // q rows of nh * d (stride q_stride), out rows of nh * e; talk float32 [nh, nh] or null (scores stay with their
-// head), temp float32 [nh] or null, gate: one value of the activation dtype per (row, head) or null.
+// head), gate: one value of the activation dtype per (row, head) or null.
 IB_EXPORT int ib_attention_talk(const void* q, int q_stride, const void* k_pool, const void* v_pool, void* out,
-                                int out_stride, int dtype, const float* talk, const float* temp, const void* gate,
+                                int out_stride, int dtype, const float* talk, const void* gate,
                                 int gate_stride, const int* positions, const int* row_entry, const int* block_tables,
                                 int max_blocks, int n_rows, int nh, int nkv, int d, int e, int page_size, int num_pages,
-                                float scale, int chunk, int window, unsigned* err, void* stream) {
+                                int chunk, int window, unsigned* err, void* stream) {
     if (n_rows <= 0) return IB_OK;
     if (!q || !k_pool || !v_pool || !out || !positions || !row_entry || !block_tables || !err) return IB_ERR_BAD_ARG;
     if (nh <= 0 || nkv <= 0 || nh % nkv || d <= 0 || e <= 0 || page_size <= 0 || num_pages <= 0 || max_blocks <= 0 ||
@@ -415,14 +418,14 @@ IB_EXPORT int ib_attention_talk(const void* q, int q_stride, const void* k_pool,
     cudaError_t le;
     if (dtype == 0)
         le = launch_kernel(attention_talk_kernel<float>, dim3(n_rows), dim3(256), smem, s, (const float*)q, q_stride,
-                           (const float*)k_pool, (const float*)v_pool, (float*)out, out_stride, talk, temp,
+                           (const float*)k_pool, (const float*)v_pool, (float*)out, out_stride, talk,
                            (const float*)gate, gate_stride, positions, row_entry, block_tables, max_blocks, nh, nkv, d, e,
-                           page_size, num_pages, scale, chunk, window, err);
+                           page_size, num_pages, chunk, window, err);
     else if (dtype == 1)
         le = launch_kernel(attention_talk_kernel<bf16>, dim3(n_rows), dim3(256), smem, s, (const bf16*)q, q_stride,
-                           (const bf16*)k_pool, (const bf16*)v_pool, (bf16*)out, out_stride, talk, temp,
+                           (const bf16*)k_pool, (const bf16*)v_pool, (bf16*)out, out_stride, talk,
                            (const bf16*)gate, gate_stride, positions, row_entry, block_tables, max_blocks, nh, nkv, d, e,
-                           page_size, num_pages, scale, chunk, window, err);
+                           page_size, num_pages, chunk, window, err);
     else
         return IB_ERR_UNSUPPORTED;
     if (le != cudaSuccess) return (int)le;

@@ -2,8 +2,10 @@
 // m16n8k16), for prompts and decoded tokens alike.  Compiled per (TALK_H, TALK_G, TALK_D, TALK_E): query
 // heads, key/value heads, size of a key, size of a value.
 //
-//   r_g(i, j) = (q_g(i) . k_g(j)) * scale * temp_g        s_h(i, j) = sum_g talk[h, g] r_g(i, j)
+//   s_h(i, j) = sum_g talk[h, g] (q_g(i) . k_g(j))
 //   out_h(i)  = sum_j softmax_j(s_h(i, .)) v_h(j) * sigmoid(gate_h(i))
+//
+// (scales of the scores are in the queries, which qk_row_norm_append scales before it rounds them).
 //
 // The exchange runs over all heads, so a CTA holds all heads of its BQ queries (8; for decoded tokens as
 // many as fill eight columns of one key/value head): keys of every key/value head come in tiles of BN that
@@ -11,7 +13,7 @@
 // (query, head) pairs, query by query; a unit is eight of them, and a warp owns UW units.  A tile is
 // worked on in three passes with a barrier between them:
 //
-//   1  S^T = K Q^T per unit, [keys x 8 columns]; the scaled scores go to shared memory as three bf16
+//   1  S^T = K Q^T per unit, [keys x 8 columns]; the scores go to shared memory as three bf16
 //      numbers that add up to the 32-bit score (8 mantissa bits each), one plane a number,
 //      [query][key][head].
 //   2  per query, 16 heads and 16 keys: [heads x heads] (bf16, exact) times [heads x keys], the three
@@ -69,7 +71,7 @@ struct Cfg {
     static constexpr int region_bytes(int bn) { return (PLANES * plane_bytes(bn) + H * (bn + 8) * 4 + 127) / 128 * 128 + 32; }
     static constexpr int smem_bytes(int bn) {
         const int b = G * UPG * 8 * QS * 2 + G * bn * KS * 2 + G * bn * VS * 2 + BQ * region_bytes(bn) + HP * SR * 2 +
-                      (H + 3) / 4 * 16 + 3 * bn * 4;
+                      3 * bn * 4;
         const int st = WARPS * 8 * VS * 2;
         return b > st ? b : st;
     }
@@ -114,15 +116,26 @@ __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commi
 __device__ __forceinline__ void cp_async_wait_but_one() { asm volatile("cp.async.wait_group 1;\n" ::: "memory"); }
 __device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_all;\n" ::: "memory"); }
 
+template <int N>
+struct Int {
+    static constexpr int value = N;
+};
+// 2^x by the special function unit, results below the normal range as zero; log2(e)
+__device__ __forceinline__ float exp2_fast(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
+    return y;
+}
+constexpr float LOG2E = 1.4426950408889634f;
+
 struct Params {
     const bf16 *q, *k_pool, *v_pool, *gate;
     bf16* out;
-    const float *talk, *temp;
+    const float* talk;
     const int *cu_rows, *positions, *block_tables;
     int q_stride, out_stride, gate_stride, max_blocks, page_size, num_pages, chunk, window, splits, slice_len, n_rows;
-    float scale;
     unsigned* err;
-    float *stats, *part;  // [splits][rows][H][2], [splits][rows][H][E]
+    float *stats, *part;  // [splits][rows][H][2] (maxima times log2(e)), [splits][rows][H][E]
 };
 
 template <int BQ, bool SPLIT>
@@ -138,8 +151,7 @@ __global__ void __launch_bounds__(Cfg<BQ>::THREADS, 1) attention_talk_mma_kernel
     bf16* vs = ks + G * BN * KS;                             // [G][BN][VS]
     unsigned char* regions = reinterpret_cast<unsigned char*>(vs + G * BN * VS);  // [BQ][QR]
     bf16* ts = reinterpret_cast<bf16*>(regions + BQ * QR);   // [HP][SR]
-    float* hs = reinterpret_cast<float*>(ts + HP * SR);      // [H] (padded to 4): scale * temperature
-    int* places = reinterpret_cast<int*>(hs + (H + 3) / 4 * 4);  // [3][BN]: a key's row in the pool, -1: none
+    int* places = reinterpret_cast<int*>(ts + HP * SR);      // [3][BN]: a key's row in the pool, -1: none
 
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gq = lane >> 2, tq = lane & 3;
     for (int i = tid; i < HP * HP; i += THREADS) {
@@ -148,7 +160,6 @@ __global__ void __launch_bounds__(Cfg<BQ>::THREADS, 1) attention_talk_mma_kernel
         if (h < H && g < H) v = p.talk ? p.talk[h * H + g] : (h == g ? 1.f : 0.f);
         ts[h * SR + g] = __float2bfloat16_rn(v);
     }
-    for (int i = tid; i < H; i += THREADS) hs[i] = p.scale * (p.temp ? p.temp[i] : 1.f);
     if (HP != H) {  // heads that only fill up a piece: zeros, or what lies there would meet a zero weight
         constexpr int PADS = HP == H ? 1 : HP - H;
         for (int i = tid; i < BQ * PLANES * BN * PADS; i += THREADS) {
@@ -193,32 +204,35 @@ __global__ void __launch_bounds__(Cfg<BQ>::THREADS, 1) attention_talk_mma_kernel
             places[t % 3 * BN + tid] = at;
         }
     };
-    auto fetch_keys = [&](int t) {
-        const int* pl = places + t % 3 * BN;
-        constexpr int KC = D / 8;
-        for (int c = tid; c < G * BN * KC; c += THREADS) {
-            const int part = c % KC, key = c / KC % BN, g = c / (KC * BN), at = pl[key];
-            bf16* dst = ks + (g * BN + key) * KS + part * 8;
-            if (at >= 0)
-                cp_async16(dst, p.k_pool + ((size_t)at + (size_t)g * p.page_size) * D + part * 8);
-            else
-                *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
+    // rows of W elements of all key/value heads, 16 bytes a copy; where the threads cover whole tiles of one
+    // key/value head a thread's key stays the same from one to the next
+    auto fetch_rows = [&](bf16* dst, int dst_stride, const bf16* pool, int pool_width, auto width, const int* pl) {
+        constexpr int PARTS = decltype(width)::value / 8, HEAD = BN * PARTS;
+        const size_t head_step = (size_t)p.page_size * pool_width;
+        if constexpr (THREADS % HEAD == 0) {
+            const int part = tid % PARTS, key = tid / PARTS % BN, at = pl[key];
+            bf16* d = dst + (tid / HEAD * BN + key) * dst_stride + part * 8;
+            const bf16* src = pool + (size_t)(at < 0 ? 0 : at) * pool_width + part * 8 + tid / HEAD * head_step;
+#pragma unroll
+            for (int g = 0; g < G; g += THREADS / HEAD) {
+                if (G % (THREADS / HEAD) != 0 && g + tid / HEAD >= G) break;
+                if (at >= 0) cp_async16(d, src);
+                else *reinterpret_cast<uint4*>(d) = make_uint4(0, 0, 0, 0);
+                d += THREADS / HEAD * BN * dst_stride;
+                src += THREADS / HEAD * head_step;
+            }
+        } else {
+            for (int c = tid; c < G * HEAD; c += THREADS) {
+                const int part = c % PARTS, key = c / PARTS % BN, g = c / HEAD, at = pl[key];
+                bf16* d = dst + (g * BN + key) * dst_stride + part * 8;
+                if (at >= 0) cp_async16(d, pool + (size_t)at * pool_width + g * head_step + part * 8);
+                else *reinterpret_cast<uint4*>(d) = make_uint4(0, 0, 0, 0);
+            }
         }
         cp_async_commit();
     };
-    auto fetch_values = [&](int t) {
-        const int* pl = places + t % 3 * BN;
-        constexpr int VC = EB / 8;
-        for (int c = tid; c < G * BN * VC; c += THREADS) {
-            const int part = c % VC, key = c / VC % BN, g = c / (VC * BN), at = pl[key];
-            bf16* dst = vs + (g * BN + key) * VS + part * 8;
-            if (at >= 0)
-                cp_async16(dst, p.v_pool + ((size_t)at + (size_t)g * p.page_size) * E + eb * EB + part * 8);
-            else
-                *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
-        }
-        cp_async_commit();
-    };
+    auto fetch_keys = [&](int t) { fetch_rows(ks, KS, p.k_pool, D, Int<D>{}, places + t % 3 * BN); };
+    auto fetch_values = [&](int t) { fetch_rows(vs, VS, p.v_pool + eb * EB, E, Int<EB>{}, places + t % 3 * BN); };
 
     {
         constexpr int QC = D / 8;
@@ -239,7 +253,22 @@ __global__ void __launch_bounds__(Cfg<BQ>::THREADS, 1) attention_talk_mma_kernel
         fetch_keys(0);
     }
 
-    // this thread's columns in pass 3 (column gq of every unit)
+    // Per unit: where this thread's two columns of S^T (pass 1) go, what its one column of P^T (pass 3: column gq)
+    // reads and sees.  Columns that only fill up a unit, and queries beyond the entry's last, write nowhere
+    // and see nothing.
+    int raw_a[UW], raw_b[UW], mix_at[UW], sees_lo[UW], sees_hi[UW];
+#pragma unroll
+    for (int a = 0; a < UW; ++a) {
+        const int u = warp * UW + a, g = u / UPG, c0 = u % UPG * 8 + 2 * tq, c = u % UPG * 8 + gq;
+        raw_a[a] = c0 < BQ * R ? c0 / R * QR + gq * SR * 2 + (g * R + c0 % R) * 2 : -1;
+        raw_b[a] = c0 + 1 < BQ * R ? (c0 + 1) / R * QR + gq * SR * 2 + (g * R + (c0 + 1) % R) * 2 : -1;
+        const bool live = u < NU && c / R < nq;
+        mix_at[a] = (live ? c / R * QR + (g * R + c % R) * MS * 4 : 0) + MIX_AT + 8 * tq;
+        sees_hi[a] = live ? pos0 + c / R - 2 * tq : -1 - 2 * tq;
+        sees_lo[a] = live ? first_key(pos0 + c / R) - 2 * tq : 0;
+    }
+    const int lo_last = first_key(last);
+    // mx: running maximum, in units of log2(e)
     float o[UW][ET][4], mx[UW], den[UW];
 #pragma unroll
     for (int a = 0; a < UW; ++a) {
@@ -304,35 +333,34 @@ __global__ void __launch_bounds__(Cfg<BQ>::THREADS, 1) attention_talk_mma_kernel
                     }
                 }
             }
-            // scaled, in three bf16 numbers each (the differences are exact)
+            // in three bf16 numbers each: the leading bits, twice, and the rest (the differences are exact)
 #pragma unroll
-            for (int x = 0; x < SEG; ++x) {
-                const int c0 = (u0 + x) % UPG * 8 + 2 * tq;  // this thread's columns: c0 and c0 + 1
-                const int qa = c0 / R, ha = g * R + c0 % R, qb = (c0 + 1) / R, hb = g * R + (c0 + 1) % R;
-                const bool in_a = BQ * R % 8 == 0 || c0 < BQ * R, in_b = BQ * R % 8 == 0 || c0 + 1 < BQ * R;
-                const float fa = in_a ? hs[ha] : 0.f, fb = in_b ? hs[hb] : 0.f;
-                bf16* da = reinterpret_cast<bf16*>(regions + qa * QR) + gq * SR + ha;
-                bf16* db = reinterpret_cast<bf16*>(regions + qb * QR) + gq * SR + hb;
+            for (int x = 0; x < SEG; ++x)
 #pragma unroll
                 for (int m = 0; m < MT; ++m)
 #pragma unroll
                     for (int i = 0; i < 2; ++i) {
-                        float va = s[x][m][2 * i] * fa, vb = s[x][m][2 * i + 1] * fb;
-                        const int at = (m * 16 + i * 8) * SR;
+                        float va = s[x][m][2 * i], vb = s[x][m][2 * i + 1];
+                        const int at = (m * 16 + i * 8) * SR * 2;
 #pragma unroll
                         for (int l = 0; l < PLANES; ++l) {
-                            const __nv_bfloat162 w = __floats2bfloat162_rn(va, vb);
-                            va -= __low2float(w);
-                            vb -= __high2float(w);
+                            const unsigned ia = __float_as_uint(va), ib = __float_as_uint(vb);
+                            const unsigned w = __byte_perm(ia, ib, 0x7632);  // both upper halves
+                            if (l + 1 < PLANES) {
+                                va -= __uint_as_float(ia & 0xffff0000u);
+                                vb -= __uint_as_float(ib & 0xffff0000u);
+                            }
+                            unsigned char* d = regions + at + l * PLANE;
                             if (R % 2 == 0) {
-                                if (in_a) *reinterpret_cast<__nv_bfloat162*>(da + at + l * (PLANE / 2)) = w;
+                                if (BQ * R % 8 == 0 || raw_a[a + x] >= 0) *reinterpret_cast<unsigned*>(d + raw_a[a + x]) = w;
                             } else {
-                                if (in_a) da[at + l * (PLANE / 2)] = __low2bfloat16(w);
-                                if (in_b) db[at + l * (PLANE / 2)] = __high2bfloat16(w);
+                                if (BQ * R % 8 == 0 || raw_a[a + x] >= 0)
+                                    *reinterpret_cast<unsigned short*>(d + raw_a[a + x]) = (unsigned short)w;
+                                if (BQ * R % 8 == 0 || raw_b[a + x] >= 0)
+                                    *reinterpret_cast<unsigned short*>(d + raw_b[a + x]) = (unsigned short)(w >> 16);
                             }
                         }
                     }
-            }
         }
         __syncthreads();
         if (t + 2 < n_tiles) look_up(t + 2);
@@ -372,6 +400,7 @@ __global__ void __launch_bounds__(Cfg<BQ>::THREADS, 1) attention_talk_mma_kernel
         else cp_async_wait_all();
         __syncthreads();
         // ---- pass 3: softmax and values
+        const bool all_seen = nq == BQ && j0 >= lo_last && j0 + BN - 1 <= pos0;
 #pragma unroll
         for (int a = 0; a < UW; a += SEG) {
             const int u0 = warp * UW + a;
@@ -380,11 +409,7 @@ __global__ void __launch_bounds__(Cfg<BQ>::THREADS, 1) attention_talk_mma_kernel
             unsigned pb[SEG][MT][2];
 #pragma unroll
             for (int x = 0; x < SEG; ++x) {
-                const int c = (u0 + x) % UPG * 8 + gq, qi = c / R;
-                const bool live = qi < nq;
-                const int pos = live ? pos0 + qi : -1, lo = live ? first_key(pos) : 0;
-                const float* mine = reinterpret_cast<const float*>(regions + (live ? qi : 0) * QR + MIX_AT) +
-                                    (g * R + c % R) * MS + 2 * tq;
+                const float* mine = reinterpret_cast<const float*>(regions + mix_at[a + x]);
                 float s[MT][4], top = -INFINITY;
 #pragma unroll
                 for (int m = 0; m < MT; ++m) {
@@ -394,17 +419,24 @@ __global__ void __launch_bounds__(Cfg<BQ>::THREADS, 1) attention_talk_mma_kernel
                     s[m][1] = u.y;
                     s[m][2] = v.x;
                     s[m][3] = v.y;
-#pragma unroll
-                    for (int i = 0; i < 4; ++i) {
-                        const int j = j0 + m * 16 + 2 * tq + (i & 1) + (i >> 1) * 8;
-                        if (j > pos || j < lo) s[m][i] = -INFINITY;
-                        top = fmaxf(top, s[m][i]);
-                    }
                 }
+                if (!all_seen) {
+#pragma unroll
+                    for (int m = 0; m < MT; ++m)
+#pragma unroll
+                        for (int i = 0; i < 4; ++i) {
+                            const int j = j0 + m * 16 + (i & 1) + (i >> 1) * 8;
+                            if (j > sees_hi[a + x] || j < sees_lo[a + x]) s[m][i] = -INFINITY;
+                        }
+                }
+#pragma unroll
+                for (int m = 0; m < MT; ++m)
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) top = fmaxf(top, s[m][i]);
                 top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, 1));
                 top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, 2));
-                const float now = fmaxf(mx[a + x], top);
-                const float f = now == mx[a + x] ? 1.f : __expf(mx[a + x] - now);  // (exp(-inf) = 0 on the first keys)
+                const float now = fmaxf(mx[a + x], top * LOG2E);
+                const float f = now == mx[a + x] ? 1.f : exp2_fast(mx[a + x] - now);  // (2^-inf = 0 on the first keys)
                 const float from = now == -INFINITY ? 0.f : now;
                 mx[a + x] = now;
                 float sum = 0.f;
@@ -412,7 +444,7 @@ __global__ void __launch_bounds__(Cfg<BQ>::THREADS, 1) attention_talk_mma_kernel
                 for (int m = 0; m < MT; ++m) {
 #pragma unroll
                     for (int i = 0; i < 4; ++i) {
-                        s[m][i] = __expf(s[m][i] - from);  // (exp(-inf) = 0 for keys that are not seen)
+                        s[m][i] = exp2_fast(fmaf(s[m][i], LOG2E, -from));  // (2^-inf = 0 for keys that are not seen)
                         sum += s[m][i];
                     }
                     pb[x][m][0] = pack_bf16(s[m][0], s[m][1]);
@@ -530,7 +562,7 @@ __global__ void attention_talk_merge_kernel(const float* __restrict__ stats, con
     for (int k = warp; k < splits; k += 4) {
         const float mk = stats[(k * step + item) * 2];
         if (mk == -INFINITY) continue;  // (the slice held no key of this row)
-        const float f = expf(mk - best);
+        const float f = exp2_fast(mk - best);
         sum = fmaf(stats[(k * step + item) * 2 + 1], f, sum);
         const float* src = part + (k * step + item) * E;
 #pragma unroll
@@ -599,16 +631,16 @@ IB_EXPORT long long ib_attention_talk_mma_scratch_bytes(int n_rows, int splits) 
 }
 
 // q rows begin with H * D queries (row stride q_stride), out rows hold H * E (stride out_stride); talk float32 [H, H]
-// whose values are exact in bf16, or null; temp float32 [H] or null; gate bf16, one per (row, head), or null.
+// whose values are exact in bf16, or null; gate bf16, one per (row, head), or null.
 // max_rows: an upper bound on the rows of any entry (the grid's width); few: the variant for few rows an entry.
 // splits > 1: the keys from the first that a CTA's first query sees, rounded down to the key tile, in slices of
 // `slice_len` (a multiple of the key tile; together they must reach the last query) over that many CTAs, through
 // `scratch`; n_rows: all rows.
 IB_EXPORT int ib_attention_talk_mma(const void* q, int q_stride, const void* k_pool, const void* v_pool, void* out,
-                                    int out_stride, const float* talk, const float* temp, const void* gate,
+                                    int out_stride, const float* talk, const void* gate,
                                     int gate_stride, const int* cu_rows, const int* positions, const int* block_tables,
                                     int max_blocks, int n_entries, int max_rows, int page_size, int num_pages,
-                                    float scale, int chunk, int window, unsigned* err, int n_rows, int few, int splits,
+                                    int chunk, int window, unsigned* err, int n_rows, int few, int splits,
                                     int slice_len, void* scratch, long long scratch_bytes, void* stream) {
     if (n_entries <= 0 || max_rows <= 0 || n_rows <= 0) return IB_OK;
     if (!q || !k_pool || !v_pool || !out || !cu_rows || !positions || !block_tables || !err) return IB_ERR_BAD_ARG;
@@ -626,7 +658,6 @@ IB_EXPORT int ib_attention_talk_mma(const void* q, int q_stride, const void* k_p
     p.gate = (const bf16*)gate;
     p.out = (bf16*)out;
     p.talk = talk;
-    p.temp = temp;
     p.cu_rows = cu_rows;
     p.positions = positions;
     p.block_tables = block_tables;
@@ -641,7 +672,6 @@ IB_EXPORT int ib_attention_talk_mma(const void* q, int q_stride, const void* k_p
     p.splits = splits;
     p.slice_len = slice_len;
     p.n_rows = n_rows;
-    p.scale = scale;
     p.err = err;
     p.stats = (float*)scratch;
     p.part = scratch ? p.stats + (size_t)splits * n_rows * H * 2 : nullptr;

@@ -26,7 +26,7 @@ from ..csrc.build import load_module
 from ..errors import KernelError
 from . import core
 
-_c_int, _c_float, _c_void_p, _c_ll = ctypes.c_int, ctypes.c_float, ctypes.c_void_p, ctypes.c_longlong
+_c_int, _c_void_p, _c_ll = ctypes.c_int, ctypes.c_void_p, ctypes.c_longlong
 _libs: Dict[Tuple[int, int, int, int], ctypes.CDLL] = {}
 
 PLAIN_SMEM = 220 * 1024  # what the plain kernel may hold of a row, in bytes
@@ -60,7 +60,7 @@ def layout(heads: int, kv_heads: int, dim: int, vdim: int, queries: int) -> Tupl
     def smem(bn: int) -> int:
         region = -(-(3 * bn * (padded + 8) * 2 + heads * (bn + 8) * 4) // 128) * 128 + 32
         total = units * 8 * (dim + 8) * 2 + kv_heads * bn * ((dim + 8) + (block + 8)) * 2 + queries * region \
-            + padded * (padded + 8) * 2 + -(-heads // 4) * 16 + 3 * bn * 4
+            + padded * (padded + 8) * 2 + 3 * bn * 4
         return max(total, warps * 8 * (block + 8) * 2)
 
     bn = 32 if smem(32) <= SMEM_MAX else 16
@@ -84,8 +84,8 @@ def lib_for(heads: int, kv_heads: int, dim: int, vdim: int) -> ctypes.CDLL:
         lib = load_module(f"attn_talk_h{heads}_g{kv_heads}_d{dim}_e{vdim}", ["attention_talk_mma.cu"],
                           [f"-DTALK_H={heads}", f"-DTALK_G={kv_heads}", f"-DTALK_D={dim}", f"-DTALK_E={vdim}"])
         lib.ib_attention_talk_mma.argtypes = [
-            _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int,
-            _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_void_p,
+            _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p,
+            _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p,
             _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_ll, _c_void_p]
         lib.ib_attention_talk_mma.restype = _c_int
         lib.ib_attention_talk_mma_scratch_bytes.argtypes = [_c_int, _c_int]
@@ -123,7 +123,7 @@ def choose_splits(max_rows: int, n_entries: int, blocks: int, span: int, bn: int
 
 
 def run(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, out: torch.Tensor, ctx, tables: torch.Tensor,
-        n_heads: int, scale: float, talk, temp, gate, chunk: int, window: int, rt) -> bool:
+        n_heads: int, talk, gate, chunk: int, window: int, rt) -> bool:
     """Arguments as ``core.attention_talk``; entries and their rows come from ``ctx.cu_rows`` and
     ``ctx.positions`` (an entry's rows are consecutive positions)."""
     num_pages, nkv, page_size, dim = k_pool.shape
@@ -132,8 +132,8 @@ def run(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, out: torch.
             or not supported(n_heads, nkv, dim, vdim) or q.stride(0) % 8 or out.stride(0) % 8 \
             or q.data_ptr() % 16 or out.data_ptr() % 16:
         return False
-    core.require_cuda(q, k_pool, v_pool, out, talk, temp, gate, tables)
-    core.check_talk_arguments(q, k_pool, v_pool, out, tables, n_heads, talk, temp, gate)
+    core.require_cuda(q, k_pool, v_pool, out, talk, gate, tables)
+    core.check_talk_arguments(q, k_pool, v_pool, out, tables, n_heads, talk, gate)
     lib = lib_for(n_heads, nkv, dim, vdim)
     key = ("talk_plan", n_heads, nkv, dim, vdim, chunk, window)
     plan = ctx.scratch.get(key) if hasattr(ctx, "scratch") else None
@@ -168,9 +168,9 @@ def run(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, out: torch.
         scratch_ptr, scratch_bytes = buf.data_ptr(), buf.numel() * 4
     code = lib.ib_attention_talk_mma(
         q.data_ptr(), q.stride(0), k_pool.data_ptr(), v_pool.data_ptr(), out.data_ptr(), out.stride(0),
-        core._ptr(talk), core._ptr(temp), core._ptr(gate), gate.stride(0) if gate is not None else 0,
+        core._ptr(talk), core._ptr(gate), gate.stride(0) if gate is not None else 0,
         ctx.cu_rows.data_ptr(), ctx.positions.data_ptr(), tables.data_ptr(), tables.shape[1], ctx.n_entries,
-        ctx.max_rows_per_entry, page_size, num_pages, float(scale), int(chunk), int(window), rt.err.data_ptr(), N, few,
+        ctx.max_rows_per_entry, page_size, num_pages, int(chunk), int(window), rt.err.data_ptr(), N, few,
         splits, slice_len, scratch_ptr, scratch_bytes, core.stream_ptr(q))
     core.check(code, "attention_talk_mma")
     return True

@@ -187,12 +187,12 @@ def core_lib() -> ctypes.CDLL:
                                             _c_void_p, _c_int, _c_int, _c_int, _c_float, _c_void_p]
         lib.ib_reenter_add.argtypes = [_c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int,
                                        _c_void_p]
-        lib.ib_qk_row_norm_append.argtypes = [_c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_float, _c_void_p, _c_int,
-                                              _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_int,
+        lib.ib_qk_row_norm_append.argtypes = [_c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_int, _c_float, _c_void_p,
+                                              _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_int,
                                               _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p]
         lib.ib_attention_talk.argtypes = [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_void_p,
-                                          _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int,
-                                          _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int,
+                                          _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int,
+                                          _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
                                           _c_void_p, _c_void_p]
         for fn in ("ib_embed_scaled", "ib_gated_act_strided", "ib_add_rmsnorm_pair", "ib_reenter_add",
                    "ib_qk_row_norm_append", "ib_attention_talk"):
@@ -1399,19 +1399,24 @@ def reenter_add(x: torch.Tensor, delta: Optional[torch.Tensor], origin: Optional
 
 
 def qk_row_norm_append(x: torch.Tensor, q_weight: Optional[torch.Tensor], k_weight: Optional[torch.Tensor], eps: float,
-                       inv_freq: Optional[torch.Tensor], rotary_dim: int, n_heads: int, n_kv_heads: int, dim: int,
+                       q_scale: Optional[torch.Tensor], inv_freq: Optional[torch.Tensor], rotary_dim: int, n_heads: int, n_kv_heads: int, dim: int,
                        vdim: int, positions: torch.Tensor, row_entry: torch.Tensor, block_tables: torch.Tensor,
                        k_pool: torch.Tensor, v_pool: torch.Tensor, err: torch.Tensor) -> None:
     """Rows of ``x``: ``n_heads`` queries and ``n_kv_heads`` keys of ``dim``, ``n_kv_heads`` values of ``vdim``.
     All of a row's queries are divided by their one root mean square and multiplied by ``q_weight``
-    (float32 [n_heads * dim]; None: neither), its keys likewise; the first ``rotary_dim`` dimensions of
-    every head are rotated (halves paired).  Queries are written back, keys and values to their pages."""
-    require_cuda(x, q_weight, k_weight, inv_freq, positions, row_entry, block_tables, k_pool, v_pool, err)
+    ([n_heads * dim], float32 or bfloat16; None: neither), its keys likewise; the first ``rotary_dim``
+    dimensions of every head are rotated (halves paired); query head h is multiplied by ``q_scale[h]``
+    (float32; None: 1).  All of it in 32-bit with one rounding at the end.  Queries are written back, keys and values to their pages."""
+    require_cuda(x, q_weight, k_weight, q_scale, inv_freq, positions, row_entry, block_tables, k_pool, v_pool, err)
     _int32(positions, "positions")
     _int32(row_entry, "row_entry")
     _int32(block_tables, "block_tables")
-    _f32_vec(q_weight, n_heads * dim, "qk_row_norm_append: q_weight")
-    _f32_vec(k_weight, n_kv_heads * dim, "qk_row_norm_append: k_weight")
+    for w, n in ((q_weight, n_heads * dim), (k_weight, n_kv_heads * dim)):
+        if w is not None and (w.shape != (n,) or not w.is_contiguous() or w.dtype not in (torch.float32, torch.bfloat16)):
+            raise KernelError(f"qk_row_norm_append: a norm's weight must be contiguous float32 or bfloat16 [{n}]")
+    if q_weight is not None and k_weight is not None and q_weight.dtype != k_weight.dtype:
+        raise KernelError("qk_row_norm_append: both norms' weights must have one dtype")
+    _f32_vec(q_scale, n_heads, "qk_row_norm_append: q_scale")
     num_pages, nkv_pool, page_size, d_pool = k_pool.shape
     if x.dim() != 2 or x.stride(1) != 1 or x.shape[1] < (n_heads + n_kv_heads) * dim + n_kv_heads * vdim:
         raise KernelError("qk_row_norm_append: x rows must hold queries, keys and values with unit inner stride")
@@ -1424,35 +1429,36 @@ def qk_row_norm_append(x: torch.Tensor, q_weight: Optional[torch.Tensor], k_weig
         if inv_freq is None:
             raise KernelError("qk_row_norm_append: a rotation needs its frequencies")
     check(core_lib().ib_qk_row_norm_append(x.data_ptr(), x.stride(0), dtype_code(x.dtype), _ptr(q_weight), _ptr(k_weight),
-                                           float(eps), _ptr(inv_freq), int(rotary_dim), positions.data_ptr(),
-                                           row_entry.data_ptr(), block_tables.data_ptr(), block_tables.shape[1],
+                                           next((dtype_code(w.dtype) for w in (q_weight, k_weight) if w is not None), 0),
+                                           float(eps), _ptr(q_scale), _ptr(inv_freq), int(rotary_dim),
+                                           positions.data_ptr(), row_entry.data_ptr(), block_tables.data_ptr(), block_tables.shape[1],
                                            k_pool.data_ptr(), v_pool.data_ptr(), x.shape[0], n_heads, n_kv_heads, dim,
                                            vdim, page_size, num_pages, err.data_ptr(), stream_ptr(x)),
           "qk_row_norm_append")
 
 
 def attention_talk(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, out: torch.Tensor, ctx,
-                   block_tables: torch.Tensor, n_heads: int, scale: float, talk: Optional[torch.Tensor],
-                   temp: Optional[torch.Tensor], gate: Optional[torch.Tensor], chunk: int, window: int,
-                   err: torch.Tensor) -> None:
+                   block_tables: torch.Tensor, n_heads: int, talk: Optional[torch.Tensor],
+                   gate: Optional[torch.Tensor], chunk: int, window: int, err: torch.Tensor) -> None:
     """Attention whose heads exchange their scores before the softmax: head h's score is
-    ``sum_g talk[h, g] temp[g] scale (q_g . k)`` over all heads (``talk`` float32 [H, H]; None: its own).
+    ``sum_g talk[h, g] (q_g . k)`` over all heads (``talk`` float32 [H, H]; None: its own score; what scales
+    scores is in the queries).
     Query i sees keys j <= i, with ``chunk`` those of its own run of ``chunk`` positions, with ``window`` the
     last ``window``.  ``gate`` [N, H] (a view of wider rows is fine): a head's result is multiplied by its
     sigmoid.  ``q`` rows begin with the queries; ``out`` [N, H * vdim] may be a view of wider rows.  32-bit."""
-    require_cuda(q, k_pool, v_pool, out, talk, temp, gate, block_tables, err)
-    check_talk_arguments(q, k_pool, v_pool, out, block_tables, n_heads, talk, temp, gate)
+    require_cuda(q, k_pool, v_pool, out, talk, gate, block_tables, err)
+    check_talk_arguments(q, k_pool, v_pool, out, block_tables, n_heads, talk, gate)
     num_pages, nkv, page_size, dim = k_pool.shape
     check(core_lib().ib_attention_talk(q.data_ptr(), q.stride(0), k_pool.data_ptr(), v_pool.data_ptr(), out.data_ptr(),
-                                       out.stride(0), dtype_code(q.dtype), _ptr(talk), _ptr(temp), _ptr(gate),
+                                       out.stride(0), dtype_code(q.dtype), _ptr(talk), _ptr(gate),
                                        gate.stride(0) if gate is not None else 0, ctx.positions.data_ptr(),
                                        ctx.row_entry.data_ptr(), block_tables.data_ptr(), block_tables.shape[1],
                                        q.shape[0], n_heads, nkv, dim, v_pool.shape[3], page_size, num_pages,
-                                       float(scale), int(chunk), int(window), err.data_ptr(), stream_ptr(q)),
+                                       int(chunk), int(window), err.data_ptr(), stream_ptr(q)),
           "attention_talk")
 
 
-def check_talk_arguments(q, k_pool, v_pool, out, block_tables, n_heads, talk, temp, gate) -> None:
+def check_talk_arguments(q, k_pool, v_pool, out, block_tables, n_heads, talk, gate) -> None:
     """What both forms of ``attention_talk`` ask of their tensors."""
     _int32(block_tables, "block_tables")
     N = q.shape[0]
@@ -1465,6 +1471,5 @@ def check_talk_arguments(q, k_pool, v_pool, out, block_tables, n_heads, talk, te
         raise KernelError("attention_talk: q rows [heads * dim ...], out [N, heads * vdim] and the pools do not fit")
     if talk is not None and (talk.dtype != torch.float32 or talk.shape != (n_heads, n_heads) or not talk.is_contiguous()):
         raise KernelError("attention_talk: talk must be contiguous float32 [heads, heads]")
-    _f32_vec(temp, n_heads, "attention_talk: temp")
     if gate is not None and (gate.shape != (N, n_heads) or gate.stride(1) != 1 or gate.dtype != q.dtype):
         raise KernelError("attention_talk: gate must be [N, heads] of q's dtype with unit inner stride")

@@ -71,7 +71,7 @@ class TalkingAttention(Mixer):
                                                           for k in ("talk", "temp", "gate"))
         self.qkv: Optional[Linear] = None
         self.o: Optional[Linear] = None
-        self.q_norm = self.k_norm = self.talk = self.temp = None
+        self.q_norm = self.k_norm = self.talk = self.q_scale = None
         self.talk_exact = True
 
     # ---- declarations -----------------------------------------------------
@@ -105,8 +105,14 @@ class TalkingAttention(Mixer):
         self.qkv = Linear(torch.cat(mats, dim=0), self.rt)
         self.o = Linear(weights[self.names["o"]], self.rt)
         f32 = lambda name: weights[name].to(torch.float32).contiguous() if name else None  # noqa: E731
-        self.q_norm, self.k_norm = (f32(n) for n in self.norm_names) if self.norm_names else (None, None)
-        self.talk, self.temp = f32(self.talk_name), f32(self.temp_name)
+        if self.norm_names:
+            self.q_norm, self.k_norm = (weights[n].contiguous() for n in self.norm_names)
+            if self.q_norm.dtype != self.k_norm.dtype:
+                self.q_norm, self.k_norm = self.q_norm.float(), self.k_norm.float()
+        self.talk = f32(self.talk_name)
+        # the scores' scale and the heads' temperatures go into the queries, before these are rounded
+        temp = f32(self.temp_name) if self.temp_name else torch.ones(self.heads, device=self.qkv.weight.device)
+        self.q_scale = (temp * self.scale).contiguous()
         # the tensor cores take the exchange's weights in bfloat16: those of a bfloat16 checkpoint are
         self.talk_exact = self.talk is None or bool((self.talk == self.talk.to(torch.bfloat16).float()).all())
 
@@ -130,16 +136,15 @@ class TalkingAttention(Mixer):
             raise ConfigError("talking attention must own its cache")
         tables = ctx.block_tables[cache.group]
         rows = self.qkv(x)
-        core.qk_row_norm_append(rows, self.q_norm, self.k_norm, self.eps, self.inv_freq, self.rotary_dim, self.heads,
-                                self.kv_heads, self.dim, self.vdim, ctx.positions, ctx.row_entry, tables, cache.k_pool,
-                                cache.v_pool, self.rt.err)
+        core.qk_row_norm_append(rows, self.q_norm, self.k_norm, self.eps, self.q_scale, self.inv_freq, self.rotary_dim,
+                                self.heads, self.kv_heads, self.dim, self.vdim, ctx.positions, ctx.row_entry, tables,
+                                cache.k_pool, cache.v_pool, self.rt.err)
         gate = None
         if self.gate_name:
             g0 = (self.heads + self.kv_heads) * self.dim + self.kv_heads * self.vdim
             gate = rows[:, g0: g0 + self.heads]
         # bfloat16 with sizes that have a variant: the tensor-core kernel; everything else the plain 32-bit one
         if not (self.talk_exact and attention_talk.run(rows, cache.k_pool, cache.v_pool, out, ctx, tables, self.heads,
-                                                       self.scale, self.talk, self.temp, gate, self.chunk, self.window,
-                                                       self.rt)):
-            core.attention_talk(rows, cache.k_pool, cache.v_pool, out, ctx, tables, self.heads, self.scale, self.talk,
-                                self.temp, gate, self.chunk, self.window, self.rt.err)
+                                                       self.talk, gate, self.chunk, self.window, self.rt)):
+            core.attention_talk(rows, cache.k_pool, cache.v_pool, out, ctx, tables, self.heads, self.talk, gate,
+                                self.chunk, self.window, self.rt.err)

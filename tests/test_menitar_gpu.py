@@ -394,6 +394,10 @@ def check_talk(dtype, H, G, d, e, page, chunk, lens, rows, run, tol, window=0, b
     step = Step(rows, [t - n for t, n in zip(lens, rows)])
     pick = lambda xs: torch.cat([x[t - n:] for x, t, n in zip(xs, lens, rows)])  # noqa: E731
     wide = torch.full((step.n_rows, H * d + H + 8 - H % 8), float("nan"), dtype=dtype, device=DEV)
+    # (what scales scores is in the queries: rounded once, scaled)
+    factor = scale * (temp if temp is not None else torch.ones(H, dtype=torch.float64))
+    qs = [(q * factor[None, :, None]).to(dtype).double() for q in qs]
+    scale, temp = 1.0, None
     wide[:, : H * d] = pick(qs).reshape(-1, H * d).to(dtype).to(DEV)
     gate = None
     if not bare:
@@ -403,7 +407,7 @@ def check_talk(dtype, H, G, d, e, page, chunk, lens, rows, run, tol, window=0, b
                      zip(qs, ks, vs, gates or [None] * len(lens), lens, rows)])
     out = torch.full((step.n_rows, H * e + 16), float("nan"), dtype=dtype, device=DEV)
     f32 = lambda x: None if x is None else x.float().to(DEV).contiguous()  # noqa: E731
-    run(wide, k_pool, v_pool, out[:, : H * e], step, tables, scale, f32(talk), f32(temp), gate, chunk, window)
+    run(wide, k_pool, v_pool, out[:, : H * e], step, tables, f32(talk), gate, chunk, window)
     assert torch.isfinite(out[:, : H * e]).all() and torch.isnan(out[:, H * e:]).all()
     assert rel_err(out[:, : H * e], ref) < tol
 
@@ -417,8 +421,7 @@ def test_exchanged_scores_with_one_key_that_stands_out(dtype, H, G, d, e, page, 
     rt = runtime(dtype)
 
     def run(q, k_pool, v_pool, out, step, tables, *consts):
-        scale, talk, temp, gate, ch, window = consts
-        core.attention_talk(q, k_pool, v_pool, out, step, tables, H, scale, talk, temp, gate, ch, window, rt.err)
+        core.attention_talk(q, k_pool, v_pool, out, step, tables, H, *consts, rt.err)
 
     lens = [1, 2, page, page + 1, 5 * page - 1, 201, 64, 97, 130]
     rows = [min(t, 5) for t in lens]
@@ -492,7 +495,7 @@ def test_the_exchange_keeps_32_bit_scores():
     k_pool, v_pool, tables = build_pools([k], [v], 16, torch.bfloat16, seed=1)
     step = Step([T])
     out = torch.empty(T, H * e, dtype=torch.bfloat16, device=DEV)
-    args = (1.0, talk.float().to(DEV).contiguous(), temp.float().to(DEV), None, 0, 0)
+    args = (talk.float().to(DEV).contiguous(), None, 0, 0)
     assert attention_talk.run(q.reshape(T, H * d).bfloat16().to(DEV), k_pool, v_pool, out, step, tables, H, *args, rt)
     assert rel_err(out, ref) < 2e-2
 
@@ -514,12 +517,15 @@ def test_norm_over_the_whole_projection_rotation_and_cache_write(dtype, H, G, d,
     x = x.to(dtype)
     qw, kw = torch.rand(H * d, generator=g) + 0.5, torch.rand(G * d, generator=g) + 0.5
     pos = torch.arange(start, start + T)
-    for normed in (True, False):
+    q_scale = torch.rand(H, generator=g) * 3
+    for normed, w_dtype, scaled in ((True, torch.float32, True), (False, torch.float32, False), (True, torch.bfloat16, False)):
+        qw, kw = qw.to(w_dtype), kw.to(w_dtype)
         xd = x.double()
         q, k, v = xd[:, : H * d], xd[:, H * d: (H + G) * d], xd[:, (H + G) * d:]
         if normed:
             q, k = pm.rms_norm(q, qw.double(), eps), pm.rms_norm(k, kw.double(), eps)
-        q = pm.rotate_half(q.reshape(T, H, d), pos, rd, base).reshape(T, -1)
+        q = pm.rotate_half(q.reshape(T, H, d), pos, rd, base)
+        q = (q * q_scale.double()[None, :, None] if scaled else q).reshape(T, -1)
         k = pm.rotate_half(k.reshape(T, G, d), pos, rd, base)
         pages = -(-(start + T) // page)
         k_pool = torch.full((pages + 1, G, page, d), 7.0, dtype=dtype, device=DEV)
@@ -530,7 +536,8 @@ def test_norm_over_the_whole_projection_rotation_and_cache_write(dtype, H, G, d,
         rows = torch.full((T, C + (8 - C % 8) + 8), 3.0, dtype=dtype, device=DEV)
         rows[:, :C] = x.to(DEV)
         inv = torch.tensor([base ** (-2.0 * i / rd) for i in range(rd // 2)], dtype=torch.float32, device=DEV) if rd else None
-        core.qk_row_norm_append(rows, qw.to(DEV) if normed else None, kw.to(DEV) if normed else None, eps, inv, rd, H, G, d, e,
+        core.qk_row_norm_append(rows, qw.to(DEV) if normed else None, kw.to(DEV) if normed else None, eps,
+                                q_scale.to(DEV) if scaled else None, inv, rd, H, G, d, e,
                                 step.positions, step.row_entry, tables, k_pool, v_pool, rt.err)
         tol = 2e-5 if dtype == torch.float32 else 1e-2
         assert rel_err(rows[:, : H * d], q) < tol
@@ -543,7 +550,7 @@ def test_norm_over_the_whole_projection_rotation_and_cache_write(dtype, H, G, d,
         assert bool((k_pool.cpu().transpose(1, 2)[~written] == 7.0).all())
     assert int(rt.err.item()) == 0
     bad = torch.full_like(tables, -1)
-    core.qk_row_norm_append(rows, None, None, eps, inv, rd, H, G, d, e, step.positions, step.row_entry, bad, k_pool, v_pool,
+    core.qk_row_norm_append(rows, None, None, eps, None, inv, rd, H, G, d, e, step.positions, step.row_entry, bad, k_pool, v_pool,
                             rt.err)
     assert int(rt.err.item()) == 2
 
