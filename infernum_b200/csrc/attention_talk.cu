@@ -108,76 +108,87 @@ __device__ __forceinline__ void load8(const float* p, float (&v)[8]) {
 }
 
 // The same on bf16 rows, 16 bytes at a time (d, e, rd / 2 and the row stride multiples of 8, 16-byte aligned
-// bases); the row's sines and cosines are worked out once, before its projection is waited for.  Every
-// thread keeps the first ROW_HOLD of its 16-byte pieces in registers between the two passes.
-constexpr int ROW_MAX_PAIRS = 256;
-constexpr int ROW_HOLD = 3;
+// bases).  An item is 8 pairs that are rotated, 8 elements that are not, or 8 elements of a value; every
+// thread holds the first ROW_HOLD of its items in registers from the sums to the stores.  The row is asked
+// for first; its sines, cosines and place in the pools are worked out (by the last threads, which have the
+// fewest items) while it comes.
+constexpr int ROW_MAX_PAIRS = 256, ROW_HOLD = 3;
+
 template <typename TW>
-__global__ void qk_row_norm_append_vec8_kernel(bf16* __restrict__ x, int x_stride, const TW* __restrict__ qw,
-                                               const TW* __restrict__ kw, float eps, const float* __restrict__ q_scale,
-                                               const float* __restrict__ inv_freq, int rd,
-                                               const int* __restrict__ positions, const int* __restrict__ row_entry,
-                                               const int* __restrict__ block_tables, int max_blocks,
-                                               bf16* __restrict__ k_pool, bf16* __restrict__ v_pool, int nh, int nkv,
-                                               int d, int e, int page_size, int num_pages, unsigned* __restrict__ err) {
+__global__ void __launch_bounds__(256, 4)
+qk_row_norm_append_vec8_kernel(bf16* __restrict__ x, int x_stride, const TW* __restrict__ qw, const TW* __restrict__ kw,
+                               float eps, const float* __restrict__ q_scale, const float* __restrict__ inv_freq, int rd,
+                               const int* __restrict__ positions, const int* __restrict__ row_entry,
+                               const int* __restrict__ block_tables, int max_blocks, bf16* __restrict__ k_pool,
+                               bf16* __restrict__ v_pool, int nh, int nkv, int d, int e, int page_size, int num_pages,
+                               unsigned* __restrict__ err) {
     pdl_trigger();
     __shared__ __align__(16) float sn_s[ROW_MAX_PAIRS];
     __shared__ __align__(16) float cs_s[ROW_MAX_PAIRS];
-    __shared__ float part[2][32];
+    __shared__ float part[2][8];
+    __shared__ long long at_s;  // the row's place among all rows of a pool (key/value head 0), -1: none
     const int row = blockIdx.x;
-    const int pos = positions[row], blk = pos / page_size;
-    const int page = blk < max_blocks ? block_tables[(size_t)row_entry[row] * max_blocks + blk] : -1;
-    const bool bad = page < 0 || page >= num_pages;
-    if (bad && threadIdx.x == 0) atomicOr(err, IB_FLAG_BAD_PAGE);
-    const size_t at = bad ? 0 : ((size_t)page * nkv) * page_size + (pos % page_size);
-    const int half = rd >> 1;
-    for (int j = threadIdx.x; j < half; j += blockDim.x) sincosf((float)pos * inv_freq[j], &sn_s[j], &cs_s[j]);
-    __syncthreads();
+    const int pos = positions[row], entry = row_entry[row];
+    const int qc = nh * d, kc = nkv * d, half = rd >> 1;
+    const int rot = half >> 3, per_head = rot + ((d - rd) >> 3);
+    const int n_qk = (nh + nkv) * per_head, n_all = n_qk + nkv * (e >> 3);
+    bf16* xr = x + (size_t)row * x_stride;
+    // the first element of item `it` of a head (c), and the head (-1: it is one of the values', c counts from theirs)
+    auto place = [&](int it, int& head, int& c) {
+        if (it >= n_qk) {
+            head = -1;
+            c = (it - n_qk) << 3;
+        } else {
+            head = it / per_head;
+            const int p = it - head * per_head;
+            c = p < rot ? p << 3 : rd + ((p - rot) << 3);
+        }
+    };
+    int head_of[ROW_HOLD], c_of[ROW_HOLD];
+#pragma unroll
+    for (int n = 0; n < ROW_HOLD; ++n) place(threadIdx.x + n * blockDim.x, head_of[n], c_of[n]);
     pdl_wait();
 
-    bf16* xr = x + (size_t)row * x_stride;
-    const int qc = nh * d, kc = nkv * d;
-    const int rot = half >> 3, per_head = rot + ((d - rd) >> 3);  // items: 8 pairs, or 8 unrotated elements
-    const int n_qk = (nh + nkv) * per_head, n_all = n_qk + nkv * (e >> 3);
-    uint4 ha[ROW_HOLD], hb[ROW_HOLD];
-    float sq = 0.f, sk = 0.f;
-    int it = threadIdx.x;
-#pragma unroll
-    for (int n = 0; n < ROW_HOLD; ++n, it += blockDim.x) {
-        if (it < n_qk) {
-            const int head = it / per_head, p = it % per_head;
-            const bf16* src = xr + head * d;
-            const int c = p < rot ? p << 3 : rd + ((p - rot) << 3);
-            ha[n] = *reinterpret_cast<const uint4*>(src + c);
-            float v[8], ss = 0.f;
-            unpack8(ha[n], v);
-#pragma unroll
-            for (int i = 0; i < 8; ++i) ss = fmaf(v[i], v[i], ss);
-            if (p < rot) {
-                hb[n] = *reinterpret_cast<const uint4*>(src + c + half);
-                unpack8(hb[n], v);
-#pragma unroll
-                for (int i = 0; i < 8; ++i) ss = fmaf(v[i], v[i], ss);
-            }
-            if (head < nh) sq += ss; else sk += ss;
-        } else if (it < n_all) {
-            ha[n] = *reinterpret_cast<const uint4*>(xr + qc + kc + ((it - n_qk) << 3));
-        }
-    }
-    for (; it < n_qk; it += blockDim.x) {
-        const int head = it / per_head, p = it % per_head;
-        const bf16* src = xr + head * d;
-        const int c = p < rot ? p << 3 : rd + ((p - rot) << 3);
+    auto squares = [&](int head, int c, const uint4& a4, const uint4& b4, float& sq, float& sk) {
         float v[8], ss = 0.f;
-        unpack8(*reinterpret_cast<const uint4*>(src + c), v);
+        unpack8(a4, v);
 #pragma unroll
         for (int i = 0; i < 8; ++i) ss = fmaf(v[i], v[i], ss);
-        if (p < rot) {
-            unpack8(*reinterpret_cast<const uint4*>(src + c + half), v);
+        if (c < half) {
+            unpack8(b4, v);
 #pragma unroll
             for (int i = 0; i < 8; ++i) ss = fmaf(v[i], v[i], ss);
         }
         if (head < nh) sq += ss; else sk += ss;
+    };
+    uint4 ha[ROW_HOLD], hb[ROW_HOLD];
+#pragma unroll
+    for (int n = 0; n < ROW_HOLD; ++n) {
+        if (threadIdx.x + n * blockDim.x >= n_all) break;
+        ha[n] = *reinterpret_cast<const uint4*>(xr + (head_of[n] < 0 ? qc + kc : head_of[n] * d) + c_of[n]);
+        if (head_of[n] >= 0 && c_of[n] < half) hb[n] = *reinterpret_cast<const uint4*>(xr + head_of[n] * d + c_of[n] + half);
+    }
+    {
+        const int back = blockDim.x - 1 - threadIdx.x;
+        if (back == 0) {
+            const int blk = pos / page_size;
+            const int page = blk < max_blocks ? block_tables[(size_t)entry * max_blocks + blk] : -1;
+            const bool bad = page < 0 || page >= num_pages;
+            if (bad) atomicOr(err, IB_FLAG_BAD_PAGE);
+            at_s = bad ? -1 : (long long)page * nkv * page_size + pos % page_size;
+        }
+        for (int j = back; j < half; j += blockDim.x) sincosf((float)pos * inv_freq[j], &sn_s[j], &cs_s[j]);
+    }
+    float sq = 0.f, sk = 0.f;
+#pragma unroll
+    for (int n = 0; n < ROW_HOLD; ++n)
+        if (threadIdx.x + n * blockDim.x < n_qk) squares(head_of[n], c_of[n], ha[n], hb[n], sq, sk);
+    for (int it = threadIdx.x + ROW_HOLD * blockDim.x; it < n_qk; it += blockDim.x) {
+        int head, c;
+        place(it, head, c);
+        const uint4 a4 = *reinterpret_cast<const uint4*>(xr + head * d + c);
+        const uint4 b4 = c < half ? *reinterpret_cast<const uint4*>(xr + head * d + c + half) : make_uint4(0, 0, 0, 0);
+        squares(head, c, a4, b4, sq, sk);
     }
     sq = warp_sum(sq);
     sk = warp_sum(sk);
@@ -186,35 +197,36 @@ __global__ void qk_row_norm_append_vec8_kernel(bf16* __restrict__ x, int x_strid
         part[1][threadIdx.x >> 5] = sk;
     }
     __syncthreads();
+    const int n_warps = blockDim.x >> 5;
     sq = sk = 0.f;
-    for (int w = 0; w < (int)(blockDim.x >> 5); ++w) {
-        sq += part[0][w];
-        sk += part[1][w];
+#pragma unroll
+    for (int w = 0; w < 8; ++w) {
+        sq += w < n_warps ? part[0][w] : 0.f;
+        sk += w < n_warps ? part[1][w] : 0.f;
     }
-    const float fq = qw ? 1.f / sqrtf(sq / (float)qc + eps) : 1.f, fk = kw ? 1.f / sqrtf(sk / (float)kc + eps) : 1.f;
+    const float fq = qw ? rsqrtf(sq / (float)qc + eps) : 1.f, fk = kw ? rsqrtf(sk / (float)kc + eps) : 1.f;
+    const long long at = at_s;
 
-    auto finish = [&](int item, uint4 a4, uint4 b4) {
-        if (item >= n_qk) {
-            const int c = (item - n_qk) << 3, g = c / e;
-            if (!bad) *reinterpret_cast<uint4*>(v_pool + (at + (size_t)g * page_size) * e + c % e) = a4;
+    auto finish = [&](int head, int c, const uint4& a4, const uint4& b4) {
+        if (head < nh && head >= 0 ? false : at < 0) return;  // (no page: only the queries are written)
+        if (head < 0) {
+            const int g = c / e;
+            *reinterpret_cast<uint4*>(v_pool + (at + (long long)g * page_size) * e + (c - g * e)) = a4;
             return;
         }
-        const int head = item / per_head, p = item % per_head;
         const bool is_q = head < nh;
-        if (!is_q && bad) return;
         const float f = is_q ? fq * (q_scale ? q_scale[head] : 1.f) : fk;
-        const TW* w = is_q ? (qw ? qw + head * d : nullptr) : (kw ? kw + (head - nh) * d : nullptr);
-        bf16* dst = is_q ? xr + head * d : k_pool + (at + (size_t)(head - nh) * page_size) * d;
-        const int c = p < rot ? p << 3 : rd + ((p - rot) << 3);
+        const TW* w = is_q ? (qw ? qw + head * d + c : nullptr) : (kw ? kw + (head - nh) * d + c : nullptr);
+        bf16* dst = (is_q ? xr + head * d : k_pool + (at + (long long)(head - nh) * page_size) * d) + c;
         float a[8], wv[8];
         unpack8(a4, a);
-        if (w) load8(w + c, wv);
+        if (w) load8(w, wv);
 #pragma unroll
         for (int i = 0; i < 8; ++i) a[i] *= w ? f * wv[i] : f;
-        if (p < rot) {
+        if (c < half) {
             float b[8], sn[8], cs[8], ra[8], rb[8];
             unpack8(b4, b);
-            if (w) load8(w + c + half, wv);
+            if (w) load8(w + half, wv);
             load8(sn_s + c, sn);
             load8(cs_s + c, cs);
 #pragma unroll
@@ -223,26 +235,21 @@ __global__ void qk_row_norm_append_vec8_kernel(bf16* __restrict__ x, int x_strid
                 ra[i] = a[i] * cs[i] - b[i] * sn[i];
                 rb[i] = b[i] * cs[i] + a[i] * sn[i];
             }
-            *reinterpret_cast<uint4*>(dst + c) = pack8(ra);
-            *reinterpret_cast<uint4*>(dst + c + half) = pack8(rb);
+            *reinterpret_cast<uint4*>(dst) = pack8(ra);
+            *reinterpret_cast<uint4*>(dst + half) = pack8(rb);
         } else {
-            *reinterpret_cast<uint4*>(dst + c) = pack8(a);
+            *reinterpret_cast<uint4*>(dst) = pack8(a);
         }
     };
-    it = threadIdx.x;
 #pragma unroll
-    for (int n = 0; n < ROW_HOLD; ++n, it += blockDim.x)
-        if (it < n_all) finish(it, ha[n], hb[n]);
-    for (; it < n_all; it += blockDim.x) {
-        if (it >= n_qk) {
-            finish(it, *reinterpret_cast<const uint4*>(xr + qc + kc + ((it - n_qk) << 3)), make_uint4(0, 0, 0, 0));
-        } else {
-            const int head = it / per_head, p = it % per_head;
-            const bf16* src = xr + head * d;
-            const int c = p < rot ? p << 3 : rd + ((p - rot) << 3);
-            finish(it, *reinterpret_cast<const uint4*>(src + c),
-                   p < rot ? *reinterpret_cast<const uint4*>(src + c + half) : make_uint4(0, 0, 0, 0));
-        }
+    for (int n = 0; n < ROW_HOLD; ++n)
+        if (threadIdx.x + n * blockDim.x < n_all) finish(head_of[n], c_of[n], ha[n], hb[n]);
+    for (int it = threadIdx.x + ROW_HOLD * blockDim.x; it < n_all; it += blockDim.x) {
+        int head, c;
+        place(it, head, c);
+        const bf16* src = xr + (head < 0 ? qc + kc : head * d) + c;
+        finish(head, c, *reinterpret_cast<const uint4*>(src),
+               head >= 0 && c < half ? *reinterpret_cast<const uint4*>(src + half) : make_uint4(0, 0, 0, 0));
     }
 }
 
@@ -268,7 +275,7 @@ IB_EXPORT int ib_qk_row_norm_append(void* x, int x_stride, int dtype, const void
     if (dtype == 1 && d % 8 == 0 && e % 8 == 0 && rd % 16 == 0 && rd / 2 <= ROW_MAX_PAIRS && x_stride % 8 == 0 &&
         !(((uintptr_t)x | (uintptr_t)k_pool | (uintptr_t)v_pool | (uintptr_t)qw | (uintptr_t)kw) & 15)) {
         const int items = (nh + nkv) * ((rd >> 4) + ((d - rd) >> 3)) + nkv * (e >> 3);
-        const int threads = items <= 256 ? 128 : (items <= 1024 ? 256 : 512);
+        const int threads = items <= 384 && n_rows >= 1024 ? 128 : 256;
         if (w_dtype == 0) IB_ROW(qk_row_norm_append_vec8_kernel<float>, bf16, float, threads);
         else IB_ROW(qk_row_norm_append_vec8_kernel<bf16>, bf16, bf16, threads);
     } else if (dtype == 0) {
