@@ -112,11 +112,11 @@ def key_span(max_kv_len: int, max_rows: int, chunk: int, window: int, bn: int, q
 
 def choose_splits(max_rows: int, n_entries: int, blocks: int, span: int, bn: int, slots: int,
                   queries: int = 8) -> Tuple[int, int]:
-    """(slices of the keys, keys per slice): one when the row tiles fill the SMs' ``slots`` for CTAs or there
-    are few keys, else as many as fill them about twice, each of at least two tiles of keys."""
+    """(slices of the keys, keys per slice): as many slices as the SMs' ``slots`` for CTAs hold at once,
+    each of at least 32 keys; one when the row tiles alone fill more than half of the slots."""
     ctas = max(1, -(-max_rows // queries) * n_entries * blocks)
-    want = min(-(-2 * slots // ctas), span // (2 * bn), MAX_SPLITS, 65535 // blocks)
-    if ctas >= slots or want < 2:
+    want = min(slots // ctas, span // 32, MAX_SPLITS, 65535 // blocks)
+    if want < 2:
         return 1, 0
     slice_len = -(-(-(-span // want)) // bn) * bn
     return -(-span // slice_len), slice_len
