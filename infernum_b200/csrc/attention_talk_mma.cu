@@ -11,7 +11,7 @@
 // many as fill eight columns of one key/value head): keys of every key/value head come in tiles of BN that
 // start at absolute multiples of BN whatever the step's cut.  The columns of a key/value head are its
 // (query, head) pairs, query by query; a unit is eight of them, and a warp owns UW units.  A tile is
-// worked on in three passes with a barrier between them:
+// worked on in three passes:
 //
 //   1  S^T = K Q^T per unit, [keys x 8 columns]; the scores go to shared memory as three bf16
 //      numbers that add up to the 32-bit score (8 mantissa bits each), one plane a number,
@@ -21,8 +21,10 @@
 //      tensor cores.  The result goes to shared memory as 32-bit, [query][head][key].
 //   3  per unit: running softmax over the tile and O^T += V^T P^T, [values x 8 columns] in registers.
 //
-// Keys have one stage, fetched by cp.async while passes 2 and 3 of the tile before run, and so have the
-// values, fetched during passes 1 and 2.  Key places are looked up in the block table once per tile, two
+// For prompts pass 3 of a tile and pass 1 of the next share the stretch between two barriers; keys have two
+// stages then (where they fit), values one, fetched by cp.async during pass 2.  Otherwise keys have one
+// stage, fetched while passes 2 and 3 of the tile before run, and values one, fetched during passes 1 and
+// 2, which leaves room for a second CTA on the SM.  Key places are looked up in the block table once per tile, two
 // tiles ahead.  Where the accumulators do not fit the registers the values are cut in ES column blocks
 // over CTAs, each of which computes the scores.
 //
@@ -69,8 +71,8 @@ struct Cfg {
     static constexpr int plane_bytes(int bn) { return bn * SR * 2; }
     // A query's region: the planes, then the exchanged scores; 8 words beyond a multiple of the 32 banks.
     static constexpr int region_bytes(int bn) { return (PLANES * plane_bytes(bn) + H * (bn + 8) * 4 + 127) / 128 * 128 + 32; }
-    static constexpr int smem_bytes(int bn) {
-        const int b = G * UPG * 8 * QS * 2 + G * bn * KS * 2 + G * bn * VS * 2 + BQ * region_bytes(bn) + HP * SR * 2 +
+    static constexpr int smem_bytes(int bn, int stages = 1) {
+        const int b = G * UPG * 8 * QS * 2 + stages * G * bn * KS * 2 + G * bn * VS * 2 + BQ * region_bytes(bn) + HP * SR * 2 +
                       3 * bn * 4;
         const int st = WARPS * 8 * VS * 2;
         return b > st ? b : st;
@@ -83,7 +85,7 @@ struct Cfg {
         }
         return smem_bytes(32) <= SMEM_MAX ? 32 : 16;
     }
-    static constexpr int BN = pick(), SMEM = smem_bytes(BN), QR = region_bytes(BN), PLANE = plane_bytes(BN),
+    static constexpr int BN = pick(), KST = BQ == 8 && smem_bytes(BN, 2) <= SMEM_MAX ? 2 : 1, SMEM = smem_bytes(BN, KST), QR = region_bytes(BN), PLANE = plane_bytes(BN),
                          MIX_AT = PLANES * PLANE, MS = BN + 8, MT = BN / 16;
     static constexpr bool FITS = SMEM <= SMEM_MAX && UW * EB <= MOST;
 };
@@ -133,7 +135,7 @@ struct Params {
     bf16* out;
     const float* talk;
     const int *cu_rows, *positions, *block_tables;
-    int q_stride, out_stride, gate_stride, max_blocks, page_size, num_pages, chunk, window, splits, slice_len, n_rows;
+    int q_stride, out_stride, gate_stride, max_blocks, page_size, num_pages, chunk, window, splits, slice_len, n_rows, run_tiles;
     unsigned* err;
     float *stats, *part;  // [splits][rows][H][2] (maxima times log2(e)), [splits][rows][H][E]
 };
@@ -147,8 +149,8 @@ __global__ void __launch_bounds__(Cfg<BQ>::THREADS, 1) attention_talk_mma_kernel
     pdl_trigger();
     extern __shared__ __align__(128) unsigned char smem_raw[];
     bf16* qs = reinterpret_cast<bf16*>(smem_raw);            // [NU * 8 columns][QS]
-    bf16* ks = qs + NU * 8 * QS;                             // [G][BN][KS]
-    bf16* vs = ks + G * BN * KS;                             // [G][BN][VS]
+    bf16* ks = qs + NU * 8 * QS;                             // [KST][G][BN][KS]
+    bf16* vs = ks + C::KST * G * BN * KS;                           // [G][BN][VS]
     unsigned char* regions = reinterpret_cast<unsigned char*>(vs + G * BN * VS);  // [BQ][QR]
     bf16* ts = reinterpret_cast<bf16*>(regions + BQ * QR);   // [HP][SR]
     int* places = reinterpret_cast<int*>(ts + HP * SR);      // [3][BN]: a key's row in the pool, -1: none
@@ -171,7 +173,14 @@ __global__ void __launch_bounds__(Cfg<BQ>::THREADS, 1) attention_talk_mma_kernel
 
     const int en = blockIdx.y, sp = SPLIT ? blockIdx.z % p.splits : 0, eb = SPLIT ? blockIdx.z / p.splits : blockIdx.z;
     const int row0 = p.cu_rows[en], n_rows = p.cu_rows[en + 1] - row0;
-    const int tile0 = (int)(gridDim.x - 1 - blockIdx.x) * BQ;  // (the last rows, which may see the most keys, first)
+    // The rows that see the most keys first: the last ones or, with several runs of positions in an entry, the
+    // last of every run, then those before them.
+    int tile = (int)(gridDim.x - 1 - blockIdx.x);
+    if (p.run_tiles > 0) {
+        const int runs = (int)gridDim.x / p.run_tiles;
+        tile = (int)blockIdx.x % runs * p.run_tiles + p.run_tiles - 1 - (int)blockIdx.x / runs;
+    }
+    const int tile0 = tile * BQ;
     if (tile0 >= n_rows) return;
     const int nq = min(BQ, n_rows - tile0);
     const int pos0 = p.positions[row0] + tile0, last = pos0 + nq - 1;  // an entry's rows are consecutive positions
@@ -231,7 +240,7 @@ __global__ void __launch_bounds__(Cfg<BQ>::THREADS, 1) attention_talk_mma_kernel
         }
         cp_async_commit();
     };
-    auto fetch_keys = [&](int t) { fetch_rows(ks, KS, p.k_pool, D, Int<D>{}, places + t % 3 * BN); };
+    auto fetch_keys = [&](int t) { fetch_rows(ks + t % C::KST * G * BN * KS, KS, p.k_pool, D, Int<D>{}, places + t % 3 * BN); };
     auto fetch_values = [&](int t) { fetch_rows(vs, VS, p.v_pool + eb * EB, E, Int<EB>{}, places + t % 3 * BN); };
 
     {
@@ -280,18 +289,14 @@ __global__ void __launch_bounds__(Cfg<BQ>::THREADS, 1) attention_talk_mma_kernel
             for (int i = 0; i < 4; ++i) o[a][n][i] = 0.f;
     }
 
-    for (int t = 0; t < n_tiles; ++t) {
-        const int j0 = klo + t * BN;
-        cp_async_wait_all();
-        __syncthreads();
-        fetch_values(t);
-        // ---- pass 1: the scores of every unit
+    // ---- pass 1: the scores of every unit
+    auto pass1 = [&](const bf16* ks_now) {
 #pragma unroll
         for (int a = 0; a < UW; a += SEG) {
             const int u0 = warp * UW + a;
             if (u0 >= NU) break;  // (the whole warp; a run of SEG units exists or does not)
             const int g = u0 / UPG;
-            const bf16* kg = ks + g * BN * KS + (lane & 15) * KS + (lane >> 4) * 8;
+            const bf16* kg = ks_now + g * BN * KS + (lane & 15) * KS + (lane >> 4) * 8;
             const bf16* qu = qs + (u0 * 8 + (lane & 7)) * QS;
             float s[SEG][MT][4];
 #pragma unroll
@@ -362,10 +367,9 @@ __global__ void __launch_bounds__(Cfg<BQ>::THREADS, 1) attention_talk_mma_kernel
                         }
                     }
         }
-        __syncthreads();
-        if (t + 2 < n_tiles) look_up(t + 2);
-        if (t + 1 < n_tiles) fetch_keys(t + 1);
-        // ---- pass 2: the exchange; an item is a query, 16 heads and 16 keys
+    };
+    // ---- pass 2: the exchange; an item is a query, 16 heads and 16 keys
+    auto pass2 = [&]() {
         for (int it = warp; it < nq * KT * MT; it += WARPS) {
             const int n0 = it % MT * 2, m = it / MT % KT, qi = it / (MT * KT);
             const bf16* raw = reinterpret_cast<const bf16*>(regions + qi * QR) + (n0 * 8 + (lane & 7)) * SR + ((lane >> 3) & 1) * 8;
@@ -396,10 +400,9 @@ __global__ void __launch_bounds__(Cfg<BQ>::THREADS, 1) attention_talk_mma_kernel
                         *reinterpret_cast<float2*>(mix + h * MS + (n0 + n) * 8 + 2 * tq) = make_float2(c[n][2 * i], c[n][2 * i + 1]);
                 }
         }
-        if (t + 1 < n_tiles) cp_async_wait_but_one();  // the values are here; the next keys need not be
-        else cp_async_wait_all();
-        __syncthreads();
-        // ---- pass 3: softmax and values
+    };
+    // ---- pass 3: softmax and values
+    auto pass3 = [&](int j0) {
         const bool all_seen = nq == BQ && j0 >= lo_last && j0 + BN - 1 <= pos0;
 #pragma unroll
         for (int a = 0; a < UW; a += SEG) {
@@ -472,6 +475,43 @@ __global__ void __launch_bounds__(Cfg<BQ>::THREADS, 1) attention_talk_mma_kernel
 #pragma unroll
                     for (int x = 0; x < SEG; ++x) mma_bf16(o[a + x][n], va, pb[x][m][0], pb[x][m][1]);
                 }
+        }
+    };
+
+    if constexpr (C::KST == 2) {
+        // Two barriers a tile: between one and the next the exchange of tile t, then softmax and values of tile t
+        // beside the scores of tile t + 1, which need nothing of one another.
+        if (n_tiles > 0) {
+            cp_async_wait_all();
+            __syncthreads();
+            if (n_tiles > 1) fetch_keys(1);
+            pass1(ks);
+        }
+        for (int t = 0; t < n_tiles; ++t) {
+            __syncthreads();
+            fetch_values(t);
+            if (t + 2 < n_tiles) look_up(t + 2);
+            pass2();
+            cp_async_wait_all();  // the values of tile t and the keys of tile t + 1
+            __syncthreads();
+            if (t + 2 < n_tiles) fetch_keys(t + 2);
+            pass3(klo + t * BN);
+            if (t + 1 < n_tiles) pass1(ks + ((t + 1) & 1) * G * BN * KS);
+        }
+    } else {
+        for (int t = 0; t < n_tiles; ++t) {
+            cp_async_wait_all();
+            __syncthreads();
+            fetch_values(t);
+            pass1(ks);
+            __syncthreads();
+            if (t + 2 < n_tiles) look_up(t + 2);
+            if (t + 1 < n_tiles) fetch_keys(t + 1);
+            pass2();
+            if (t + 1 < n_tiles) cp_async_wait_but_one();  // the values are here; the next keys need not be
+            else cp_async_wait_all();
+            __syncthreads();
+            pass3(klo + t * BN);
         }
     }
 
@@ -600,10 +640,15 @@ int launch_talk(const Params& p, int n_entries, int max_rows, cudaStream_t s) {
         if (ce != cudaSuccess) return (int)ce;
         configured = true;
     }
-    const dim3 grid((max_rows + BQ - 1) / BQ, n_entries, C::ES * p.splits);
+    const int tiles = (max_rows + BQ - 1) / BQ;
+    Params q = p;
+    q.run_tiles = p.chunk / BQ > 0 && p.chunk / BQ < tiles ? p.chunk / BQ : 0;
+    // (whole runs of tiles: those beyond the entry's last row have nothing to do)
+    const int cols = q.run_tiles ? (tiles + q.run_tiles - 1) / q.run_tiles * q.run_tiles : tiles;
+    const dim3 grid(cols, n_entries, C::ES * p.splits);
     cudaError_t le = p.splits == 1
-        ? launch_kernel(attention_talk_mma_kernel<BQ, false>, grid, dim3(C::THREADS), C::SMEM, s, p)
-        : launch_kernel(attention_talk_mma_kernel<BQ, true>, grid, dim3(C::THREADS), C::SMEM, s, p);
+        ? launch_kernel(attention_talk_mma_kernel<BQ, false>, grid, dim3(C::THREADS), C::SMEM, s, q)
+        : launch_kernel(attention_talk_mma_kernel<BQ, true>, grid, dim3(C::THREADS), C::SMEM, s, q);
     if (le != cudaSuccess) return (int)le;
     if (p.splits > 1) {
         le = launch_kernel(attention_talk_merge_kernel, dim3((unsigned)((long long)p.n_rows * H)), dim3(128), 0, s,
@@ -672,6 +717,7 @@ IB_EXPORT int ib_attention_talk_mma(const void* q, int q_stride, const void* k_p
     p.splits = splits;
     p.slice_len = slice_len;
     p.n_rows = n_rows;
+    p.run_tiles = 0;
     p.err = err;
     p.stats = (float*)scratch;
     p.part = scratch ? p.stats + (size_t)splits * n_rows * H * 2 : nullptr;

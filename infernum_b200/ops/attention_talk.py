@@ -57,9 +57,9 @@ def layout(heads: int, kv_heads: int, dim: int, vdim: int, queries: int) -> Tupl
     padded = -(-heads // 16) * 16
     block = next((e for e in range(vdim, 15, -16) if vdim % e == 0 and mine * e <= most), 16)
 
-    def smem(bn: int) -> int:
+    def smem(bn: int, stages: int = 1) -> int:
         region = -(-(3 * bn * (padded + 8) * 2 + heads * (bn + 8) * 4) // 128) * 128 + 32
-        total = units * 8 * (dim + 8) * 2 + kv_heads * bn * ((dim + 8) + (block + 8)) * 2 + queries * region \
+        total = units * 8 * (dim + 8) * 2 + kv_heads * bn * (stages * (dim + 8) + (block + 8)) * 2 + queries * region \
             + padded * (padded + 8) * 2 + 3 * bn * 4
         return max(total, warps * 8 * (block + 8) * 2)
 
@@ -68,7 +68,9 @@ def layout(heads: int, kv_heads: int, dim: int, vdim: int, queries: int) -> Tupl
         # few rows: as many keys as leave room for a second CTA on the SM, if any do
         half = SMEM_MAX // 2 - 1024
         bn = 32 if smem(32) <= half else (16 if smem(16) <= half else bn)
-    return bn, vdim // block, smem(bn), smem(bn) <= SMEM_MAX and mine * block <= most
+    stages = 2 if queries == 8 and smem(bn, 2) <= SMEM_MAX else 1
+    total = smem(bn, stages)
+    return bn, vdim // block, total, total <= SMEM_MAX and mine * block <= most
 
 
 def supported(heads: int, kv_heads: int, dim: int, vdim: int) -> bool:
