@@ -5,7 +5,9 @@
 //   pool  [pages, 1, page_size, W]   each token's latent c (KV elements) followed
 //                        by the rotated key part all heads share
 //   out   [N, H, KV]     sum_j p_j c_j;  s_j = (q . pool_j) * scale over the
-//                        visible keys max(0, p - window + 1) <= j <= p
+//                        visible keys max(0, p - window + 1) <= j <= p; with `sink` [H]
+//                        exp(sink_h) more in the denominator (no key, no value, not
+//                        scaled); with `gate` [N, H] times sigmoid(gate)
 //
 // Every head reads the same keys, and a key's value is its own first KV
 // elements.  So the rows of a step are packed with their heads on the M side
@@ -88,10 +90,14 @@ struct LatentParams {
     int n_entries, heads, page_size, num_pages, window;
     float scale;
     int splits;
+    const float* sink;               // [H], or null
+    const bf16* gate; int gate_rs;   // [N, H] with rows gate_rs apart, or null
     float* part_o; float* part_ml;   // [splits, N * H, KV] and [splits, N * H, 2]
     int n_rows_total;
     unsigned* err;
 };
+
+__device__ __forceinline__ float gate_factor(bf16 logit) { return 1.f / (1.f + __expf(-__bfloat162float(logit))); }
 
 constexpr int LDP = KT + 8;       // row stride of the P tile (bf16)
 
@@ -194,8 +200,10 @@ __global__ void __launch_bounds__(128 * RG) latent_attention_kernel(const Latent
         }
     }
     for (int i = tid; i < M; i += THREADS) {
-        m_s[i] = -INFINITY;
-        l_s[i] = 0.f;
+        // a sink is there from the start, as a key without a value would be (of the first slice's keys)
+        const bool sunk = p.sink && blockIdx.z == 0 && g0 + i <= g_last;
+        m_s[i] = sunk ? p.sink[(g0 + i) % H] : -INFINITY;
+        l_s[i] = sunk ? 1.f : 0.f;
     }
 
     for (int t = t_lo; t < t_hi; ++t) {
@@ -330,7 +338,8 @@ __global__ void __launch_bounds__(128 * RG) latent_attention_kernel(const Latent
             if (g > g_last) continue;
             const int r = g / H, h = g % H;
             if (p.splits <= 1) {
-                const float inv = l > 0.f ? 1.f / l : 0.f;
+                float inv = l > 0.f ? 1.f / l : 0.f;
+                if (p.gate) inv *= gate_factor(p.gate[(size_t)(row0 + r) * p.gate_rs + h]);
                 bf16* dst = p.out + (size_t)(row0 + r) * p.o_rs + (size_t)h * p.o_hs + warp * (KV / 4) + qd * 2;
 #pragma unroll
                 for (int nt = 0; nt < NT; ++nt)
@@ -357,7 +366,7 @@ __global__ void __launch_bounds__(128 * RG) latent_attention_kernel(const Latent
 // other.
 __global__ void latent_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                       bf16* __restrict__ out, int o_rs, int o_hs, int n_rows, int heads,
-                                      int splits) {
+                                      int splits, const bf16* __restrict__ gate, int gate_rs) {
     pdl_trigger();
     pdl_wait();
     __shared__ float w_s[64];     // splits <= 64
@@ -380,7 +389,8 @@ __global__ void latent_combine_kernel(const float* __restrict__ part_o, const fl
             w_s[s] = w;
             denom += w * l_sh[s];
         }
-        const float inv = denom > 0.f ? 1.f / denom : 0.f;
+        float inv = denom > 0.f ? 1.f / denom : 0.f;
+        if (gate) inv *= gate_factor(gate[(size_t)r * gate_rs + h]);
         for (int s = 0; s < splits; ++s) w_s[s] *= inv;
     }
     __syncthreads();
@@ -435,15 +445,16 @@ IB_EXPORT long long ib_attention_latent_scratch_bytes(int n_rows, int heads, int
 // `mt`: 1, 2: that many sixteens of packed rows for four warps; 3: 32 rows, 4: 64 rows, for eight
 // warps in two groups.
 // `splits` > 1 needs scratch of
-// ib_attention_latent_scratch_bytes.
+// ib_attention_latent_scratch_bytes.  `sink` float32 [H] or null; `gate` bf16 [N, H], rows gate_rs apart, or null.
 IB_EXPORT int ib_attention_latent(const void* q, int q_rs, int q_hs, const void* pool, void* out, int o_rs, int o_hs,
                                   const int* cu_rows, const int* q_start, const int* tables, int max_blocks,
                                   int n_entries, int n_rows, int max_rows_per_entry, int heads, int page_size,
                                   int num_pages, int window, float scale, int mt, int splits, void* scratch,
-                                  long long scratch_bytes, unsigned* err, void* stream) {
+                                  long long scratch_bytes, const float* sink, const void* gate, int gate_rs,
+                                  unsigned* err, void* stream) {
     if (n_entries <= 0 || n_rows <= 0) return IB_OK;
     if (!q || !pool || !out || !cu_rows || !q_start || !tables || !err || heads <= 0 || page_size <= 0 ||
-        num_pages <= 0 || max_blocks <= 0 || max_rows_per_entry <= 0 || splits < 1 || splits > 64)
+        num_pages <= 0 || max_blocks <= 0 || max_rows_per_entry <= 0 || splits < 1 || splits > 64 || (gate && gate_rs < heads))
         return IB_ERR_BAD_ARG;
     if ((q_rs % 8) || (q_hs % 8) || (o_rs % 2) || (o_hs % 2) || ((uintptr_t)q & 15) || ((uintptr_t)pool & 15) ||
         ((uintptr_t)out & 3))
@@ -457,6 +468,7 @@ IB_EXPORT int ib_attention_latent(const void* q, int q_rs, int q_hs, const void*
     p.cu_rows = cu_rows; p.q_start = q_start; p.tables = tables; p.max_blocks = max_blocks;
     p.n_entries = n_entries; p.heads = heads; p.page_size = page_size; p.num_pages = num_pages; p.window = window;
     p.scale = scale; p.splits = splits; p.n_rows_total = n_rows; p.err = err;
+    p.sink = sink; p.gate = (const bf16*)gate; p.gate_rs = gate_rs;
     p.part_o = nullptr; p.part_ml = nullptr;
     if (splits > 1) {
         if (!scratch || scratch_bytes < ib_attention_latent_scratch_bytes(n_rows, heads, splits)) return IB_ERR_BAD_ARG;
@@ -472,7 +484,7 @@ IB_EXPORT int ib_attention_latent(const void* q, int q_rs, int q_hs, const void*
     if (splits > 1) {
         cudaError_t le = launch_kernel(latent_combine_kernel, dim3(n_rows * heads), dim3(KV >= 256 ? 128 : 64), 0, s,
                                        (const float*)p.part_o, (const float*)p.part_ml, (bf16*)out, o_rs, o_hs,
-                                       n_rows, heads, splits);
+                                       n_rows, heads, splits, (const bf16*)gate, gate_rs);
         if (le != cudaSuccess) return (int)le;
         IB_LAUNCH_CHECK();
     }

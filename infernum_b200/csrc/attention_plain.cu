@@ -35,6 +35,7 @@ __global__ void attention_plain_kernel(const T* __restrict__ q, int q_stride,
                                        int nh, int nkv, int hd, int page_size, int num_pages,
                                        int window, float scale, int hdv, int v_width, int q_hs, int o_hs,
                                        const float* __restrict__ sink, int keep_first,
+                                       const T* __restrict__ gate, int gate_stride,
                                        unsigned* __restrict__ err) {
     const int row = blockIdx.x;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -94,7 +95,8 @@ __global__ void attention_plain_kernel(const T* __restrict__ q, int q_stride,
         for (int i = 0; i < PLAIN_MAX_REGS; ++i) acc[i] *= corr;
     }
     T* op = out + (size_t)row * out_stride + (size_t)head * o_hs;
-    const float inv = l > 0.f ? 1.f / l : 0.f;
+    float inv = l > 0.f ? 1.f / l : 0.f;
+    if (gate) inv *= 1.f / (1.f + expf(-to_f32(gate[(size_t)row * gate_stride + head])));
 #pragma unroll
     for (int i = 0; i < PLAIN_MAX_REGS; ++i) {
         const int d = lane + 32 * i;
@@ -107,13 +109,13 @@ static int launch_plain(const void* q, int q_stride, const void* k_pool, const v
                         int out_stride, const int* positions, const int* row_entry, const int* block_tables,
                         int max_blocks, int n_rows, int nh, int nkv, int hd, int page_size, int num_pages,
                         int window, float scale, int hdv, int v_width, int q_hs, int o_hs, const float* sink,
-                        int keep_first, unsigned* err, cudaStream_t s) {
+                        int keep_first, const void* gate, int gate_stride, unsigned* err, cudaStream_t s) {
     const int warps = 4;
     dim3 grid(n_rows, (nh + warps - 1) / warps);
     attention_plain_kernel<T, NREG><<<grid, warps * 32, 0, s>>>(
         (const T*)q, q_stride, (const T*)k_pool, (const T*)v_pool, (T*)out, out_stride, positions, row_entry,
         block_tables, max_blocks, nh, nkv, hd, page_size, num_pages, window, scale, hdv, v_width, q_hs, o_hs, sink,
-        keep_first, err);
+        keep_first, (const T*)gate, gate_stride, err);
     IB_LAUNCH_CHECK();
     return IB_OK;
 }
@@ -122,17 +124,20 @@ static int launch_plain(const void* q, int q_stride, const void* k_pool, const v
 // `q_hs` and output heads `o_hs` elements apart; `sink` (optional, float32 [nh])
 // adds exp(sink[head]) to each softmax denominator.
 // `keep_first`: the keys at positions below it stay visible behind a window.
-IB_EXPORT int ib_attention_plain_mask(const void* q, int q_stride, const void* k_pool, const void* v_pool,
+// `gate` (optional, of the activation dtype, [rows, nh] with rows `gate_stride` apart): a head's result is
+// multiplied by its sigmoid.
+IB_EXPORT int ib_attention_plain_gated(const void* q, int q_stride, const void* k_pool, const void* v_pool,
                                       void* out, int out_stride, int act_dtype, const int* positions,
                                       const int* row_entry, const int* block_tables, int max_blocks, int n_rows,
                                       int nh, int nkv, int hd, int page_size, int num_pages, int window,
                                       float scale, int hdv, int v_width, int q_hs, int o_hs, const float* sink,
-                                      int keep_first, unsigned* err, void* stream) {
+                                      int keep_first, const void* gate, int gate_stride, unsigned* err,
+                                      void* stream) {
     if (n_rows <= 0) return IB_OK;
     if (!q || !k_pool || !v_pool || !out || !positions || !row_entry || !block_tables || !err)
         return IB_ERR_BAD_ARG;
     if (nh <= 0 || nkv <= 0 || nh % nkv != 0 || hd <= 0 || page_size <= 0 || max_blocks <= 0 ||
-        num_pages <= 0 || hdv <= 0 || hdv > v_width || q_hs < hd || o_hs < hdv)
+        num_pages <= 0 || hdv <= 0 || hdv > v_width || q_hs < hd || o_hs < hdv || (gate && gate_stride < nh))
         return IB_ERR_BAD_ARG;
     const int wide = hd > hdv ? hd : hdv;
     if (wide > 32 * 32) return IB_ERR_TOO_LARGE;
@@ -140,7 +145,7 @@ IB_EXPORT int ib_attention_plain_mask(const void* q, int q_stride, const void* k
 #define IB_PLAIN(T, NREG)                                                                                   \
     return launch_plain<T, NREG>(q, q_stride, k_pool, v_pool, out, out_stride, positions, row_entry,        \
                                  block_tables, max_blocks, n_rows, nh, nkv, hd, page_size, num_pages, window, \
-                                 scale, hdv, v_width, q_hs, o_hs, sink, keep_first, err, s)
+                                 scale, hdv, v_width, q_hs, o_hs, sink, keep_first, gate, gate_stride, err, s)
     if (act_dtype == 0) {
         if (wide <= 256) IB_PLAIN(float, 8);
         if (wide <= 640) IB_PLAIN(float, 20);
@@ -153,6 +158,17 @@ IB_EXPORT int ib_attention_plain_mask(const void* q, int q_stride, const void* k
     }
 #undef IB_PLAIN
     return IB_ERR_UNSUPPORTED;
+}
+
+IB_EXPORT int ib_attention_plain_mask(const void* q, int q_stride, const void* k_pool, const void* v_pool,
+                                      void* out, int out_stride, int act_dtype, const int* positions,
+                                      const int* row_entry, const int* block_tables, int max_blocks, int n_rows,
+                                      int nh, int nkv, int hd, int page_size, int num_pages, int window,
+                                      float scale, int hdv, int v_width, int q_hs, int o_hs, const float* sink,
+                                      int keep_first, unsigned* err, void* stream) {
+    return ib_attention_plain_gated(q, q_stride, k_pool, v_pool, out, out_stride, act_dtype, positions, row_entry,
+                                    block_tables, max_blocks, n_rows, nh, nkv, hd, page_size, num_pages, window, scale,
+                                    hdv, v_width, q_hs, o_hs, sink, keep_first, nullptr, 0, err, stream);
 }
 
 IB_EXPORT int ib_attention_plain_ex(const void* q, int q_stride, const void* k_pool, const void* v_pool,

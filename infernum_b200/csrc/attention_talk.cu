@@ -16,6 +16,7 @@
 //                       rotated (element i with i + rd/2, angle = position * f_i); query head h is
 //                       multiplied by q_scale[h] (what scales its scores).  Queries are
 //                       written back in place, keys and values to their pages.  32-bit, one rounding.
+//                       The values may also be the keys as they were projected.
 //   attention_talk      one CTA per row, all heads: keys in tiles of 32 that start at absolute
 //                       multiples of 32; the heads' scores, their combination, the running softmax
 //                       and the weighted values each a pass over shared memory.  32-bit throughout:
@@ -30,7 +31,7 @@ __global__ void qk_row_norm_append_kernel(T* __restrict__ x, int x_stride, const
                                           const float* __restrict__ inv_freq,
                                           int rd, const int* __restrict__ positions, const int* __restrict__ row_entry,
                                           const int* __restrict__ block_tables, int max_blocks, T* __restrict__ k_pool,
-                                          T* __restrict__ v_pool, int nh, int nkv, int d, int e, int page_size,
+                                          T* __restrict__ v_pool, int nh, int nkv, int d, int e, int v_off, int page_size,
                                           int num_pages, unsigned* __restrict__ err) {
     pdl_trigger();
     pdl_wait();
@@ -61,7 +62,7 @@ __global__ void qk_row_norm_append_kernel(T* __restrict__ x, int x_stride, const
     for (int it = threadIdx.x; it < items; it += blockDim.x) {
         if (it >= (nh + nkv) * per_head) {
             const int c = it - (nh + nkv) * per_head, g = c / e;
-            if (!bad) v_pool[(at + (size_t)g * page_size) * e + c % e] = xr[qc + kc + c];
+            if (!bad) v_pool[(at + (size_t)g * page_size) * e + c % e] = xr[v_off + c];
             continue;
         }
         const int head = it / per_head, i = it % per_head;
@@ -120,7 +121,7 @@ qk_row_norm_append_vec8_kernel(bf16* __restrict__ x, int x_stride, const TW* __r
                                float eps, const float* __restrict__ q_scale, const float* __restrict__ inv_freq, int rd,
                                const int* __restrict__ positions, const int* __restrict__ row_entry,
                                const int* __restrict__ block_tables, int max_blocks, bf16* __restrict__ k_pool,
-                               bf16* __restrict__ v_pool, int nh, int nkv, int d, int e, int page_size, int num_pages,
+                               bf16* __restrict__ v_pool, int nh, int nkv, int d, int e, int v_off, int page_size, int num_pages,
                                unsigned* __restrict__ err) {
     pdl_trigger();
     __shared__ __align__(16) float sn_s[ROW_MAX_PAIRS];
@@ -165,7 +166,7 @@ qk_row_norm_append_vec8_kernel(bf16* __restrict__ x, int x_stride, const TW* __r
 #pragma unroll
     for (int n = 0; n < ROW_HOLD; ++n) {
         if (threadIdx.x + n * blockDim.x >= n_all) break;
-        ha[n] = *reinterpret_cast<const uint4*>(xr + (head_of[n] < 0 ? qc + kc : head_of[n] * d) + c_of[n]);
+        ha[n] = *reinterpret_cast<const uint4*>(xr + (head_of[n] < 0 ? v_off : head_of[n] * d) + c_of[n]);
         if (head_of[n] >= 0 && c_of[n] < half) hb[n] = *reinterpret_cast<const uint4*>(xr + head_of[n] * d + c_of[n] + half);
     }
     {
@@ -247,32 +248,33 @@ qk_row_norm_append_vec8_kernel(bf16* __restrict__ x, int x_stride, const TW* __r
     for (int it = threadIdx.x + ROW_HOLD * blockDim.x; it < n_all; it += blockDim.x) {
         int head, c;
         place(it, head, c);
-        const bf16* src = xr + (head < 0 ? qc + kc : head * d) + c;
+        const bf16* src = xr + (head < 0 ? v_off : head * d) + c;
         finish(head, c, *reinterpret_cast<const uint4*>(src),
                head >= 0 && c < half ? *reinterpret_cast<const uint4*>(src + half) : make_uint4(0, 0, 0, 0));
     }
 }
 
-// x rows: [nh * d | nkv * d | nkv * e | anything]; qw [nh * d] / kw [nkv * d] of type w_dtype (0 float32, 1 bf16), or
+// x rows: [nh * d | nkv * d | ...], the values' nkv * e from column v_off on (behind the queries, which are written
+// over; v_off = nh * d makes the keys, as they were projected, the values too); qw [nh * d] / kw [nkv * d] of type w_dtype (0 float32, 1 bf16), or
 // null: not normed; q_scale float32 [nh] or null.
 IB_EXPORT int ib_qk_row_norm_append(void* x, int x_stride, int dtype, const void* qw, const void* kw, int w_dtype, float eps,
                                     const float* q_scale, const float* inv_freq, int rd, const int* positions,
                                     const int* row_entry, const int* block_tables, int max_blocks, void* k_pool,
-                                    void* v_pool, int n_rows, int nh, int nkv, int d, int e, int page_size, int num_pages,
-                                    unsigned* err, void* stream) {
+                                    void* v_pool, int n_rows, int nh, int nkv, int d, int e, int v_off, int page_size,
+                                    int num_pages, unsigned* err, void* stream) {
     if (n_rows <= 0) return IB_OK;
     if (!x || !positions || !row_entry || !block_tables || !k_pool || !v_pool || !err) return IB_ERR_BAD_ARG;
     if (nh <= 0 || nkv <= 0 || d <= 0 || e <= 0 || page_size <= 0 || num_pages <= 0 || max_blocks <= 0 || rd < 0 ||
         (rd & 1) || rd > d || (rd > 0 && !inv_freq) || ((qw || kw) && !(eps > 0.f)) || w_dtype < 0 || w_dtype > 1)
         return IB_ERR_BAD_ARG;
-    if (x_stride < (nh + nkv) * d + nkv * e) return IB_ERR_BAD_ARG;
+    if (v_off < nh * d || x_stride < (nh + nkv) * d || x_stride < v_off + nkv * e) return IB_ERR_BAD_ARG;
     cudaStream_t s = (cudaStream_t)stream;
     cudaError_t le;
 #define IB_ROW(KERNEL, T, TW, THREADS)                                                                                   \
     le = launch_kernel(KERNEL, dim3(n_rows), dim3(THREADS), 0, s, (T*)x, x_stride, (const TW*)qw, (const TW*)kw, eps, q_scale, \
-                       inv_freq, rd, positions, row_entry, block_tables, max_blocks, (T*)k_pool, (T*)v_pool, nh, nkv, d, e, \
+                       inv_freq, rd, positions, row_entry, block_tables, max_blocks, (T*)k_pool, (T*)v_pool, nh, nkv, d, e, v_off, \
                        page_size, num_pages, err)
-    if (dtype == 1 && d % 8 == 0 && e % 8 == 0 && rd % 16 == 0 && rd / 2 <= ROW_MAX_PAIRS && x_stride % 8 == 0 &&
+    if (dtype == 1 && d % 8 == 0 && e % 8 == 0 && v_off % 8 == 0 && rd % 16 == 0 && rd / 2 <= ROW_MAX_PAIRS && x_stride % 8 == 0 &&
         !(((uintptr_t)x | (uintptr_t)k_pool | (uintptr_t)v_pool | (uintptr_t)qw | (uintptr_t)kw) & 15)) {
         const int items = (nh + nkv) * ((rd >> 4) + ((d - rd) >> 3)) + nkv * (e >> 3);
         const int threads = items <= 384 && n_rows >= 1024 ? 128 : 256;

@@ -207,6 +207,15 @@ __device__ __forceinline__ float gate_times(float g, float u, int act, float lim
     return g / (1.f + expf(-g)) * u;
 }
 
+// An activation of one value, in 32-bit: act 1 = the square of what relu leaves, max(v, 0)^2; 0 = none.
+__device__ __forceinline__ float act_alone(float v, int act) {
+    if (act == 1) {
+        v = fmaxf(v, 0.f);
+        return v * v;
+    }
+    return v;
+}
+
 }  // namespace ib
 
 // Turns programmatic dependent launch on or off for this library (default on).

@@ -624,11 +624,13 @@ IB_EXPORT int ib_rope_append(void* qkv, int act_dtype, int qkv_stride, const int
 // With `scale` [N, n_scales] every output is also multiplied by
 // scale[row, i / cols_per_scale]: the outputs are those of n_scales experts
 // side by side and the scale is the weight the row's router gave each (0 for
-// an expert it did not choose).
+// an expert it did not choose).  From output column `limit_col` on the clamped
+// activation's limit is `limit2` (another expert's; I for none).
 template <typename T>
 __global__ void gated_act_kernel(const T* __restrict__ x, T* __restrict__ out, int I, int blk,
                                  size_t total, int act, const float* __restrict__ scale,
-                                 int cols_per_scale, int n_scales, float limit, float alpha, int out_stride) {
+                                 int cols_per_scale, int n_scales, float limit, float alpha, int out_stride,
+                                 int limit_col, float limit2) {
     pdl_trigger();
     pdl_wait();
     size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -638,7 +640,7 @@ __global__ void gated_act_kernel(const T* __restrict__ x, T* __restrict__ out, i
     const size_t gi = row * 2 * I + (size_t)(i / blk) * 2 * blk + (i % blk);
     const float g = to_f32(x[gi]);
     const float u = to_f32(x[gi + blk]);
-    float y = gate_times(g, u, act + 1, limit, alpha);
+    float y = gate_times(g, u, act + 1, i < limit_col ? limit : limit2, alpha);
     if (scale) y *= scale[row * n_scales + i / cols_per_scale];
     out[row * out_stride + i] = from_f32<T>(y);
 }
@@ -647,7 +649,7 @@ __global__ void gated_act_kernel(const T* __restrict__ x, T* __restrict__ out, i
 __global__ void gated_act_vec8_kernel(const bf16* __restrict__ x, bf16* __restrict__ out, int I,
                                       int blk, size_t total_vec, int act, const float* __restrict__ scale,
                                       int cols_per_scale, int n_scales, float limit, float alpha,
-                                      int out_stride) {
+                                      int out_stride, int limit_col, float limit2) {
     pdl_trigger();
     pdl_wait();
     const size_t v = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -662,6 +664,7 @@ __global__ void gated_act_vec8_kernel(const bf16* __restrict__ x, bf16* __restri
     const __nv_bfloat162* u2 = reinterpret_cast<const __nv_bfloat162*>(&u4);
     // (cols_per_scale is a multiple of 8 here: the eight outputs share a scale)
     const float sc = scale ? scale[row * n_scales + i / cols_per_scale] : 1.f;
+    if (i >= limit_col) limit = limit2;  // (a multiple of 8 here)
     uint4 o4;
     __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(&o4);
 #pragma unroll
@@ -676,19 +679,19 @@ __global__ void gated_act_vec8_kernel(const bf16* __restrict__ x, bf16* __restri
 
 IB_EXPORT int ib_gated_act_strided(const void* x, void* out, int out_stride, int act_dtype, int n_rows, int I, int blk,
                                    int act, float limit, float alpha, const float* scale, int cols_per_scale,
-                                   void* stream) {
+                                   int limit_col, float limit2, void* stream) {
     if (n_rows <= 0) return IB_OK;
-    if (!x || !out || I <= 0 || blk <= 0 || I % blk || act < 0 || act > 2 || out_stride < I) return IB_ERR_BAD_ARG;
+    if (!x || !out || I <= 0 || blk <= 0 || I % blk || act < 0 || act > 2 || out_stride < I || limit_col < 0) return IB_ERR_BAD_ARG;
     if (scale && (cols_per_scale <= 0 || I % cols_per_scale)) return IB_ERR_BAD_ARG;
     const int n_scales = scale ? I / cols_per_scale : 0;
     cudaStream_t s = (cudaStream_t)stream;
     const size_t total = (size_t)n_rows * I;
-    if (act_dtype == 1 && I % 8 == 0 && blk % 8 == 0 && out_stride % 8 == 0 && (!scale || cols_per_scale % 8 == 0) &&
+    if (act_dtype == 1 && I % 8 == 0 && blk % 8 == 0 && out_stride % 8 == 0 && (!scale || cols_per_scale % 8 == 0) && limit_col % 8 == 0 &&
         !(((uintptr_t)x | (uintptr_t)out) & 15)) {
         const size_t total_vec = total / 8;
         cudaError_t le = launch_kernel(gated_act_vec8_kernel, dim3((unsigned)((total_vec + 255) / 256)),
                                        dim3(256), 0, s, (const bf16*)x, (bf16*)out, I, blk, total_vec, act, scale,
-                                       cols_per_scale, n_scales, limit, alpha, out_stride);
+                                       cols_per_scale, n_scales, limit, alpha, out_stride, limit_col, limit2);
         if (le != cudaSuccess) return (int)le;
         IB_LAUNCH_CHECK();
         return IB_OK;
@@ -697,12 +700,12 @@ IB_EXPORT int ib_gated_act_strided(const void* x, void* out, int out_stride, int
     if (act_dtype == 0) {
         cudaError_t le = launch_kernel(gated_act_kernel<float>, dim3(blocks), dim3(256), 0, s,
                                        (const float*)x, (float*)out, I, blk, total, act, scale, cols_per_scale,
-                                       n_scales, limit, alpha, out_stride);
+                                       n_scales, limit, alpha, out_stride, limit_col, limit2);
         if (le != cudaSuccess) return (int)le;
     } else if (act_dtype == 1) {
         cudaError_t le = launch_kernel(gated_act_kernel<bf16>, dim3(blocks), dim3(256), 0, s,
                                        (const bf16*)x, (bf16*)out, I, blk, total, act, scale, cols_per_scale,
-                                       n_scales, limit, alpha, out_stride);
+                                       n_scales, limit, alpha, out_stride, limit_col, limit2);
         if (le != cudaSuccess) return (int)le;
     } else {
         return IB_ERR_UNSUPPORTED;
@@ -714,7 +717,7 @@ IB_EXPORT int ib_gated_act_strided(const void* x, void* out, int out_stride, int
 IB_EXPORT int ib_gated_act(const void* x, void* out, int act_dtype, int n_rows, int I, int blk, int act,
                            const float* scale, int cols_per_scale, void* stream) {
     if (act > 1) return IB_ERR_BAD_ARG;  // (the clamped activation comes with its limit)
-    return ib_gated_act_strided(x, out, I, act_dtype, n_rows, I, blk, act, 0.f, 0.f, scale, cols_per_scale, stream);
+    return ib_gated_act_strided(x, out, I, act_dtype, n_rows, I, blk, act, 0.f, 0.f, scale, cols_per_scale, I, 0.f, stream);
 }
 
 IB_EXPORT int ib_silu_mul(const void* x, void* out, int act_dtype, int n_rows, int I, int blk,

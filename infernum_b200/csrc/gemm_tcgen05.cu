@@ -188,6 +188,7 @@ struct GemmParams {
     int out_f32;
     float act_limit, act_alpha;  // of the clamped activation
     int swiglu;           // gate_times' code: W rows are 64 gates then their 64 ups per tile; out is [T, N/2]
+    int alone;            // act_alone's code, for products without a gate
 };
 
 template <int BN>
@@ -363,7 +364,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w,
                     for (int j = 0; j < 16; ++j) {
                         const int t = t0 + c + j;
                         if (t < p.T && n < p.N) {
-                            const float f = __uint_as_float(v[j]);
+                            const float f = act_alone(__uint_as_float(v[j]), p.alone);
                             if (p.out_f32) ((float*)p.out)[(size_t)t * p.ldo + n] = f;
                             else ((bf16*)p.out)[(size_t)t * p.ldo + n] = __float2bfloat16_rn(f);
                         }
@@ -435,6 +436,9 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w,
                             acc.z += part[u][sidx].z;
                             acc.w += part[u][sidx].w;
                         }
+                        if (p.alone)
+                            acc = make_float4(act_alone(acc.x, p.alone), act_alone(acc.y, p.alone),
+                                              act_alone(acc.z, p.alone), act_alone(acc.w, p.alone));
                         if (p.out_f32) {
                             *reinterpret_cast<float4*>((float*)p.out + (size_t)t * p.ldo + n4) = acc;
                         } else {
@@ -459,6 +463,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w,
                 float acc = 0.f;
 #pragma unroll
                 for (int sidx = 0; sidx < 8; ++sidx) acc += part[sidx];
+                acc = act_alone(acc, p.alone);
                 if (n < p.N) {
                     if (p.out_f32) ((float*)p.out)[(size_t)t * p.ldo + n] = acc;
                     else ((bf16*)p.out)[(size_t)t * p.ldo + n] = __float2bfloat16_rn(acc);
@@ -559,9 +564,13 @@ IB_EXPORT int ib_gemm_tc_token_tile(int T) {
 // CTAs of a cluster.  swiglu > 0 (gate_times' code; act_limit and act_alpha are those of code 3): W holds, per
 // 128 rows, 64 gate rows followed by their 64 up rows; out is [T, N / 2] bf16 with
 // out[t, 64 b + r] = gate_times(x . W[128 b + r], x . W[128 b + 64 + r]); K is not split.
+// swiglu < 0: no gates; -swiglu is act_alone's code, applied to every value of the product.
 IB_EXPORT int ib_gemm_tc(const void* x, int ldx, const void* w, int ldw, void* out, int ldo,
                          int out_f32, int T, int N, int K, int splits, int swiglu, unsigned* err,
                          void* stream, float act_limit, float act_alpha) {
+    const int alone = swiglu < 0 ? -swiglu : 0;
+    if (alone) swiglu = 0;
+    if (alone > 1) return IB_ERR_BAD_ARG;
     if (T <= 0 || N <= 0) return IB_OK;
     if (!x || !w || !out || !err || K <= 0) return IB_ERR_BAD_ARG;
     // TMA: 16-byte aligned bases and row strides
@@ -587,6 +596,7 @@ IB_EXPORT int ib_gemm_tc(const void* x, int ldx, const void* w, int ldw, void* o
     p.splits = (kblocks + p.kblocks_per_split - 1) / p.kblocks_per_split;  // no empty slice
     p.out_f32 = out_f32;
     p.swiglu = swiglu;
+    p.alone = alone;
     p.act_limit = act_limit;
     p.act_alpha = act_alpha;
     CUtensorMap mw, mx;

@@ -163,8 +163,10 @@ struct Params {
     bf16* out;
     unsigned* err;
     int T, N, K, ldo;
-    int act;  // with the gated epilogue: gate_times' code
+    int act;  // with the gated epilogue: gate_times' code, without: act_alone's
     float act_limit, act_alpha;
+    int limit_col;        // from this output column on the limit is act_limit2 (16 | limit_col)
+    float act_limit2;
     const float* scale;   // with the gated epilogue, optional [T, n_scales]: out[t, c] *= scale[t, c / cols_per_scale]
     int n_scales, cols_per_scale;   // (experts side by side and the weight a token's router gave each; 16 | cols_per_scale)
     int t_tiles;   // token tiles of 256
@@ -337,9 +339,10 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constan
                         // (sixteen columns share a scale; those past the row's end are not stored)
                         const float sc = p.scale && live && col < limit
                                              ? p.scale[(size_t)gt * p.n_scales + col / p.cols_per_scale] : 1.f;
+                        const float limit_here = col < p.limit_col ? p.act_limit : p.act_limit2;
 #pragma unroll
                         for (int q = 0; q < 16; ++q)
-                            v[q] = gate_times(__uint_as_float(g[q]), __uint_as_float(u[q]), p.act, p.act_limit, p.act_alpha) * sc;
+                            v[q] = gate_times(__uint_as_float(g[q]), __uint_as_float(u[q]), p.act, limit_here, p.act_alpha) * sc;
                         if (live) store16(row, col, limit, v);
                     }
                 }
@@ -355,11 +358,11 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constan
                     tmem_ld_wait();
                     float v[16];
 #pragma unroll
-                    for (int q = 0; q < 16; ++q) v[q] = __uint_as_float(a[q]);
+                    for (int q = 0; q < 16; ++q) v[q] = act_alone(__uint_as_float(a[q]), p.act);
                     if (live) store16(row, n0 + c, limit, v);
                     if (two) {
 #pragma unroll
-                        for (int q = 0; q < 16; ++q) v[q] = __uint_as_float(b[q]);
+                        for (int q = 0; q < 16; ++q) v[q] = act_alone(__uint_as_float(b[q]), p.act);
                         if (live) store16(row, n0 + c + 16, limit, v);
                     }
                 }
@@ -450,10 +453,15 @@ int launch_pair(const CUtensorMap& mx, const CUtensorMap& mw, const CUtensorMap&
 // `swiglu` names the activation (gate_times' codes; act_limit and act_alpha are those of code 3).
 // `scale` (with `swiglu` only; float32 [T, (N/2) / cols_per_scale], or null): every output is also
 // multiplied by scale[t, column / cols_per_scale] (cols_per_scale a multiple of 16 that divides N/2).
+// From output column `limit_col` on (a multiple of 16; N for none) the clamped activation's limit is act_limit2.
+// swiglu < 0: no gates; -swiglu is act_alone's code, applied to every value of the product.
 IB_EXPORT int ib_gemm_pair_scaled(const void* x, int ldx, const void* w, int ldw, void* out, int ldo, int T, int N,
                                   int K, int swiglu, int bn_a, int cols_a, int bn_b, int t_group, int sm_count,
                                   const float* scale, int cols_per_scale, unsigned* err, void* stream, float act_limit,
-                                  float act_alpha) {
+                                  float act_alpha, int limit_col, float act_limit2) {
+    const int alone = swiglu < 0 ? -swiglu : 0;
+    if (alone) swiglu = 0;
+    if (alone > 1 || limit_col < 0 || limit_col % 16) return IB_ERR_BAD_ARG;
     if (T <= 0 || N <= 0) return IB_OK;
     if (scale && (!swiglu || cols_per_scale <= 0 || cols_per_scale % 16 || (N / 2) % cols_per_scale))
         return IB_ERR_BAD_ARG;
@@ -471,7 +479,9 @@ IB_EXPORT int ib_gemm_pair_scaled(const void* x, int ldx, const void* w, int ldw
     p.N = N;
     p.K = K;
     p.ldo = ldo;
-    p.act = swiglu;
+    p.act = alone ? alone : swiglu;
+    p.limit_col = limit_col;
+    p.act_limit2 = act_limit2;
     p.act_limit = act_limit;
     p.act_alpha = act_alpha;
     p.scale = scale;
@@ -505,5 +515,5 @@ IB_EXPORT int ib_gemm_pair(const void* x, int ldx, const void* w, int ldw, void*
                            int K, int swiglu, int bn_a, int cols_a, int bn_b, int t_group, int sm_count,
                            unsigned* err, void* stream) {
     return ib_gemm_pair_scaled(x, ldx, w, ldw, out, ldo, T, N, K, swiglu, bn_a, cols_a, bn_b, t_group, sm_count,
-                               nullptr, 0, err, stream, 0.f, 0.f);
+                               nullptr, 0, err, stream, 0.f, 0.f, 0, 0.f);
 }

@@ -120,6 +120,47 @@ IB_EXPORT int ib_moe_route(const float* logits, int ld, const float* bias, int E
     return IB_OK;
 }
 
+// Strikes out (-inf) the values z[E] of all but the `keep` best of `n_groups` equal groups of neighbours; a group's
+// score, kept in gs[n_groups], is the sum of its `group_top` largest values, the lower index first among equals.
+// By one warp; `group_top` > 1 needs groups of at most 64.
+__device__ __forceinline__ void close_groups(float* z, float* gs, int E, int n_groups, int keep, int group_top,
+                                             int lane) {
+    const int per = E / n_groups;
+    for (int g = lane; g < n_groups; g += 32) {
+        float sum = 0.f;
+        unsigned long long taken = 0ull;
+        for (int k = 0; k < group_top && k < per; ++k) {
+            float best = -INFINITY;
+            int at = -1;
+            for (int i = 0; i < per; ++i) {
+                if (group_top > 1 && ((taken >> i) & 1ull)) continue;
+                const float v = z[g * per + i];
+                if (v > best) { best = v; at = i; }
+            }
+            if (at < 0) break;
+            if (group_top > 1) taken |= 1ull << at;
+            sum += best;
+        }
+        gs[g] = sum;
+    }
+    __syncwarp();
+    // lane 0 picks the best groups; a chosen one is marked by -inf
+    if (lane == 0) {
+        for (int k = 0; k < keep; ++k) {
+            float best = -INFINITY;
+            int at = -1;
+            for (int g = 0; g < n_groups; ++g)
+                if (gs[g] > best) { best = gs[g]; at = g; }
+            if (at < 0) break;
+            gs[at] = -INFINITY;
+        }
+    }
+    __syncwarp();
+    for (int e = lane; e < E; e += 32)
+        if (gs[e / per] != -INFINITY) z[e] = -INFINITY;
+    __syncwarp();
+}
+
 __global__ void moe_route_scored_kernel(const float* __restrict__ logits, int ld, const float* __restrict__ bias,
                                         int E, int top, int n_groups, int keep, int group_top, int renorm,
                                         int* __restrict__ ids, float* __restrict__ weights,
@@ -135,43 +176,7 @@ __global__ void moe_route_scored_kernel(const float* __restrict__ logits, int ld
         if (gate) gate[(size_t)row * E + e] = 0.f;
     }
     __syncwarp();
-    if (n_groups > 1) {
-        const int per = E / n_groups;
-        // a lane a group: the sum of its group_top largest scores (lowest index among equals)
-        for (int g = lane; g < n_groups; g += 32) {
-            float sum = 0.f;
-            unsigned long long taken = 0ull;  // (groups of more than 64 experts: see the host check)
-            for (int k = 0; k < group_top && k < per; ++k) {
-                float best = -INFINITY;
-                int at = -1;
-                for (int i = 0; i < per; ++i) {
-                    if ((taken >> i) & 1ull) continue;
-                    const float v = z[g * per + i];
-                    if (v > best) { best = v; at = i; }
-                }
-                if (at < 0) break;
-                taken |= 1ull << at;
-                sum += best;
-            }
-            gs[g] = sum;
-        }
-        __syncwarp();
-        // lane 0 picks the best groups and strikes out the experts of the others
-        if (lane == 0) {
-            for (int k = 0; k < keep; ++k) {
-                float best = -INFINITY;
-                int at = -1;
-                for (int g = 0; g < n_groups; ++g)
-                    if (gs[g] > best) { best = gs[g]; at = g; }
-                if (at < 0) break;
-                gs[at] = -INFINITY;  // chosen: marked by -inf, told apart from the rest below
-            }
-        }
-        __syncwarp();
-        for (int e = lane; e < E; e += 32)
-            if (gs[e / per] != -INFINITY) z[e] = -INFINITY;
-        __syncwarp();
-    }
+    if (n_groups > 1) close_groups(z, gs, E, n_groups, keep, group_top, lane);
     float denom = 0.f;
     for (int k = 0; k < top; ++k) {
         float best = -INFINITY;
@@ -215,7 +220,7 @@ IB_EXPORT int ib_moe_route_scored(const float* logits, int ld, const float* bias
     if (n_groups > 1 && (E % n_groups || keep <= 0 || keep > n_groups || group_top <= 0 ||
                          (long long)keep * (E / n_groups) < top))
         return IB_ERR_BAD_ARG;
-    if (n_groups > 1 && E / n_groups > 64) return IB_ERR_TOO_LARGE;
+    if (n_groups > 1 && group_top > 1 && E / n_groups > 64) return IB_ERR_TOO_LARGE;
     const size_t smem = (size_t)(E + (n_groups > 1 ? n_groups : 0)) * sizeof(float);
     if (smem > 48 * 1024) return IB_ERR_TOO_LARGE;
     cudaError_t le = launch_kernel(moe_route_scored_kernel, dim3(n_rows), dim3(32), smem, (cudaStream_t)stream, logits,
@@ -227,7 +232,9 @@ IB_EXPORT int ib_moe_route_scored(const float* logits, int ld, const float* bias
 
 // A third way of scoring (ib_moe_route_softmax_all): s = softmax(z) over all E_all router
 // outputs; the choice is made by s_e + correction_e (the lower index among equals), the
-// weights are the chosen s_e (without the correction) over their sum + 1e-20.  The last
+// weights are the chosen s_e (without the correction) over their sum + 1e-20, or - `renorm` 0 -
+// as they are.  With n_groups > 1 only the experts of the `keep` best groups can be chosen,
+// groups scored by the sum of their `group_top` largest choice values.  The last
 // E_all - E outputs have no expert behind them: choosing one hands the token's input on
 // with that weight.  Written: ids / weights [N, top]; the dense row gate[N, E] for the
 // experts that exist; extra[N, 2] = (the sum of the weights that fell on the outputs
@@ -238,7 +245,8 @@ IB_EXPORT int ib_moe_route_scored(const float* logits, int ld, const float* bias
 __global__ void moe_route_softmax_all_kernel(const float* __restrict__ logits, int ld,
                                              const float* __restrict__ correction, int E_all, int E, int top,
                                              int with_gate, int* __restrict__ ids, float* __restrict__ weights,
-                                             float* __restrict__ gate, float* __restrict__ extra, int gate_cols) {
+                                             float* __restrict__ gate, float* __restrict__ extra, int gate_cols,
+                                             int n_groups, int keep, int group_top, int renorm) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ float sm[];
@@ -264,6 +272,7 @@ __global__ void moe_route_softmax_all_kernel(const float* __restrict__ logits, i
         if (gate && e < E) gate[(size_t)row * gate_cols + e] = 0.f;
     }
     __syncwarp();
+    if (n_groups > 1) close_groups(c, c + E_all, E_all, n_groups, keep, group_top, lane);
     float sum = 0.f;
     for (int k = 0; k < top; ++k) {
         float best = -INFINITY;
@@ -287,7 +296,7 @@ __global__ void moe_route_softmax_all_kernel(const float* __restrict__ logits, i
         __syncwarp();
     }
     if (lane == 0) {
-        const float inv = 1.f / (sum + 1e-20f);
+        const float inv = renorm ? 1.f / (sum + 1e-20f) : 1.f;
         float passed = 0.f;
         for (int k = 0; k < top; ++k) {
             const int at = ids[(size_t)row * top + k];
@@ -311,15 +320,21 @@ __global__ void moe_route_softmax_all_kernel(const float* __restrict__ logits, i
 
 IB_EXPORT int ib_moe_route_softmax_all(const float* logits, int ld, const float* correction, int E_all, int E, int top,
                                        int with_gate, int* ids, float* weights, float* gate, float* extra,
-                                       int gate_cols, int n_rows, void* stream) {
+                                       int gate_cols, int n_groups, int keep, int group_top, int renorm, int n_rows,
+                                       void* stream) {
     if (n_rows <= 0) return IB_OK;
     if (!logits || !ids || !weights || E_all <= 0 || E < 0 || E > E_all || top <= 0 || top > E_all ||
         ld < E_all + (with_gate ? 1 : 0) || (gate && gate_cols < E))
         return IB_ERR_BAD_ARG;
-    const size_t smem = (size_t)E_all * 2 * sizeof(float);
+    if (n_groups > 1 && (E_all % n_groups || keep <= 0 || keep > n_groups || group_top <= 0 ||
+                         (long long)keep * (E_all / n_groups) < top))
+        return IB_ERR_BAD_ARG;
+    if (n_groups > 1 && group_top > 1 && E_all / n_groups > 64) return IB_ERR_TOO_LARGE;
+    const size_t smem = (size_t)(E_all * 2 + (n_groups > 1 ? n_groups : 0)) * sizeof(float);
     if (smem > 48 * 1024) return IB_ERR_TOO_LARGE;
     cudaError_t le = launch_kernel(moe_route_softmax_all_kernel, dim3(n_rows), dim3(32), smem, (cudaStream_t)stream,
-                                   logits, ld, correction, E_all, E, top, with_gate, ids, weights, gate, extra, gate_cols);
+                                   logits, ld, correction, E_all, E, top, with_gate, ids, weights, gate, extra, gate_cols,
+                                   n_groups, keep, group_top, renorm);
     if (le != cudaSuccess) return (int)le;
     IB_LAUNCH_CHECK();
     return IB_OK;

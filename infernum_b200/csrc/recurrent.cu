@@ -246,6 +246,94 @@ IB_EXPORT int ib_wkv_prepare(const void* r, const void* k, const void* v, int ld
     return IB_OK;
 }
 
+// gla_prepare: per key channel (q * q_scale, k, a, 0) with the decay a = sigmoid(z)^(1/tau) =
+// exp(-softplus(-z) / tau), and v in 32-bit, by head: [heads][rows][K] and [heads][rows][P].  A row of `x`
+// holds q | k (heads * K each) and v (heads * P) at three column offsets.  z [rows][heads * K] comes made
+// (`z` float32), or is made here from a low-rank pair: z = W2 lo + bias, `lo` [rank] at another offset of
+// the row, W2 [heads * K, rank].  In the second form a CTA has 128 channels and GLA_ROWS rows: a channel's
+// W2 row is read once for all of them, sixteen of its values at a time.
+constexpr int GLA_ROWS = 8, GLA_PIECE = 16;
+
+template <typename T>
+__global__ void __launch_bounds__(128)
+gla_prepare_kernel(const T* __restrict__ x, int ld, int q_off, int k_off, int v_off, int lo_off, int rank,
+                   const T* __restrict__ w2, const float* __restrict__ bias, const float* __restrict__ z,
+                   float q_scale, float inv_tau, float4* __restrict__ f, float* __restrict__ vo, int heads, int K,
+                   int P, int n_rows) {
+    pdl_trigger();
+    __shared__ float lo_s[GLA_ROWS][GLA_PIECE];
+    const int c = blockIdx.x * blockDim.x + threadIdx.x, r0 = blockIdx.y * GLA_ROWS;
+    const int nr = min(GLA_ROWS, n_rows - r0);
+    const int hk = heads * K, hp = heads * P;
+    float acc[GLA_ROWS];
+    const float b = c < hk && bias ? bias[c] : 0.f;
+#pragma unroll
+    for (int r = 0; r < GLA_ROWS; ++r) acc[r] = b;
+    pdl_wait();
+    if (z) {
+        if (c < hk)
+            for (int r = 0; r < nr; ++r) acc[r] += z[(size_t)(r0 + r) * hk + c];
+    } else {
+        for (int k0 = 0; k0 < rank; k0 += GLA_PIECE) {
+            const int n = min(GLA_PIECE, rank - k0);
+            __syncthreads();
+            const int lr = threadIdx.x / GLA_PIECE, lc = threadIdx.x % GLA_PIECE;  // 128 threads: all of the piece
+            lo_s[lr][lc] = lr < nr && lc < n ? to_f32(x[(size_t)(r0 + lr) * ld + lo_off + k0 + lc]) : 0.f;
+            float w[GLA_PIECE];
+#pragma unroll
+            for (int i = 0; i < GLA_PIECE; ++i) w[i] = c < hk && i < n ? to_f32(w2[(size_t)c * rank + k0 + i]) : 0.f;
+            __syncthreads();
+#pragma unroll
+            for (int r = 0; r < GLA_ROWS; ++r)
+#pragma unroll
+                for (int i = 0; i < GLA_PIECE; ++i) acc[r] = fmaf(w[i], lo_s[r][i], acc[r]);
+        }
+    }
+    if (c < hk) {
+        const int head = c / K;
+#pragma unroll
+        for (int r = 0; r < GLA_ROWS; ++r) {
+            if (r >= nr) break;
+            const T* xr = x + (size_t)(r0 + r) * ld;
+            const float log_a = fminf(acc[r], 0.f) - log1pf(expf(-fabsf(acc[r])));  // log sigmoid(z), never above 0
+            f[((size_t)head * n_rows + r0 + r) * K + (c - head * K)] =
+                make_float4(to_f32(xr[q_off + c]) * q_scale, to_f32(xr[k_off + c]), expf(log_a * inv_tau), 0.f);
+        }
+    }
+    if (c < hp) {
+        const int head = c / P;
+        for (int r = 0; r < nr; ++r)
+            vo[((size_t)head * n_rows + r0 + r) * P + (c - head * P)] = to_f32(x[(size_t)(r0 + r) * ld + v_off + c]);
+    }
+}
+
+// x rows `ld` apart; bias float32 [heads * K] or null; z float32 or null (then w2 of x's type and rank > 0).
+IB_EXPORT int ib_gla_prepare(const void* x, int ld, int act_dtype, int q_off, int k_off, int v_off, int lo_off, int rank,
+                             const void* w2, const float* bias, const float* z, float q_scale, float inv_tau, void* f,
+                             float* vo, int n_rows, int heads, int K, int P, void* stream) {
+    if (n_rows <= 0) return IB_OK;
+    if (!x || !f || !vo || heads <= 0 || K <= 0 || P <= 0 || q_off < 0 || k_off < 0 || v_off < 0 || !(inv_tau > 0.f) ||
+        ((uintptr_t)f & 15) || q_off + heads * K > ld || k_off + heads * K > ld || v_off + heads * P > ld)
+        return IB_ERR_BAD_ARG;
+    if (!z && (!w2 || rank <= 0 || lo_off < 0 || lo_off + rank > ld)) return IB_ERR_BAD_ARG;
+    cudaStream_t s = (cudaStream_t)stream;
+    const int cols = heads * (K > P ? K : P);
+    const dim3 grid((cols + 127) / 128, (n_rows + GLA_ROWS - 1) / GLA_ROWS);
+    if (grid.y > 65535) return IB_ERR_TOO_LARGE;
+    cudaError_t le;
+    if (act_dtype == 0)
+        le = launch_kernel(gla_prepare_kernel<float>, grid, dim3(128), 0, s, (const float*)x, ld, q_off, k_off, v_off,
+                           lo_off, rank, (const float*)w2, bias, z, q_scale, inv_tau, (float4*)f, vo, heads, K, P, n_rows);
+    else if (act_dtype == 1)
+        le = launch_kernel(gla_prepare_kernel<bf16>, grid, dim3(128), 0, s, (const bf16*)x, ld, q_off, k_off, v_off,
+                           lo_off, rank, (const bf16*)w2, bias, z, q_scale, inv_tau, (float4*)f, vo, heads, K, P, n_rows);
+    else
+        return IB_ERR_UNSUPPORTED;
+    if (le != cudaSuccess) return (int)le;
+    IB_LAUNCH_CHECK();
+    return IB_OK;
+}
+
 // ---------------------------------------------------------------------------
 // One warp per (row, head): out = o / sqrt(mean_head(o^2) + eps) * w * silu(g).
 template <typename T>
@@ -421,7 +509,7 @@ IB_EXPORT int ib_qk_norm_append(void* x, int x_stride, int act_dtype, const floa
 // ---------------------------------------------------------------------------
 // Elementwise: op 0: a <- a * sigmoid(b)   (an output gate)
 //              op 1: a <- ca * a + cb * b  (two mixers side by side)
-//              op 2: a <- tanh(a)
+//              op 2: a <- tanh(a);  op 3: a <- max(a, 0)^2
 // a is [rows, cols] contiguous, b has rows `b_stride` apart.
 template <typename T>
 __global__ void pointwise_kernel(T* __restrict__ a, const T* __restrict__ b, int b_stride, int cols, size_t total,
@@ -436,14 +524,15 @@ __global__ void pointwise_kernel(T* __restrict__ a, const T* __restrict__ b, int
     float r;
     if (op == 0) r = av / (1.f + expf(-bv));
     else if (op == 1) r = ca * av + cb * bv;
-    else r = tanhf(av);
+    else if (op == 2) r = tanhf(av);
+    else r = act_alone(av, 1);
     a[idx] = from_f32<T>(r);
 }
 
 IB_EXPORT int ib_pointwise(void* a, const void* b, int b_stride, int act_dtype, int rows, int cols, int op, float ca,
                            float cb, void* stream) {
     if (rows <= 0 || cols <= 0) return IB_OK;
-    if (!a || (op != 2 && !b) || op < 0 || op > 2) return IB_ERR_BAD_ARG;
+    if (!a || (op < 2 && !b) || op < 0 || op > 3) return IB_ERR_BAD_ARG;
     cudaStream_t s = (cudaStream_t)stream;
     const size_t total = (size_t)rows * cols;
     const unsigned grid = (unsigned)((total + 255) / 256);

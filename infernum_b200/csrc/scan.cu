@@ -6,13 +6,15 @@
 //
 //   wkv:  o_t[j] = sum_i r_t[i] (S[i][j] + u[i] k_t[i] v_t[j])        (u only for the current token)
 //         S[i][j] <- w_t[i] S[i][j] + k_t[i] v_t[j]
+//   gla:  S[i][j] <- a_t[i] S[i][j] + k_t[i] v_t[j],   o_t[j] = sum_i q_t[i] S[i][j]   (the state after its update)
 //   ssd:  S[n][p] <- a_t S[n][p] + B_t[n] (dt_t x_t[p]),   y_t[p] = sum_n C_t[n] S[n][p] + D x_t[p]
 //   delta: S <- g_t S;  u = beta_t (v_t - S^T k_t);  S <- S + k_t u^T;  o_t = S^T q_t
 //         (a gated delta rule; o_t is taken from the state after its update)
 //
-// Everything a token brings - (r, k, w, u k) per key channel and v for wkv; (B, C)
+// Everything a token brings - (r, k, w, u k) per key channel and v for wkv; (q, k, a) per
+// key channel and v for gla; (B, C)
 // per state row, x, and (dt, a) per head for ssd - has been made in 32-bit by a
-// parallel pass before (recurrent.cu: wkv_prepare, ssd_prepare), so the scan only
+// parallel pass before (recurrent.cu: wkv_prepare, gla_prepare, ssd_prepare), so the scan only
 // copies: CHUNK tokens at a time go to shared memory by cp.async, two stages deep,
 // while the tokens of the chunk before are walked.
 //
@@ -92,7 +94,7 @@ template <int N>
 __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;\n" ::"n"(N) : "memory"); }
 
 struct WkvParams {
-    const float4* f;    // [heads][rows][ROWS]: r, k, w, u * k
+    const float4* f;    // [heads][rows][ROWS]: r, k, w, u * k (gla: q, k, a, unused)
     const float* v;     // [heads][rows][P]
     int n_rows;         // rows of the whole step
     float* state;       // request slot s, head h: state + s * state_stride + h * P * ROWS, [P][ROWS]
@@ -103,6 +105,9 @@ struct WkvParams {
     int heads, P, cols; // cols: columns of one CTA
 };
 
+// GLA: the result is read from the state after the token's update, without it (wkv) from the one before,
+// the current token's own share weighted by u.
+template <bool GLA>
 __global__ void __launch_bounds__(512) wkv_scan_kernel(const WkvParams p) {
     pdl_wait();
     extern __shared__ float4 smem4[];
@@ -156,8 +161,13 @@ __global__ void __launch_bounds__(512) wkv_scan_kernel(const WkvParams p) {
 #pragma unroll
             for (int ii = 0; ii < RPT; ++ii) {
                 const float4 q = f[ii * SPLIT];
-                acc = fmaf(q.x, fmaf(q.w, vj, S[ii]), acc);
-                S[ii] = fmaf(q.z, S[ii], q.y * vj);
+                if (GLA) {
+                    S[ii] = fmaf(q.z, S[ii], q.y * vj);
+                    acc = fmaf(q.x, S[ii], acc);
+                } else {
+                    acc = fmaf(q.x, fmaf(q.w, vj, S[ii]), acc);
+                    S[ii] = fmaf(q.z, S[ii], q.y * vj);
+                }
             }
             acc = split_sum(acc);
             if (active && part == 0) p.out[(size_t)(c0 + t) * ldo + hp + j0 + col] = acc;
@@ -381,9 +391,10 @@ static int scan_geometry(int P, int col_slices, int* cols, int* threads) {
 
 // f: float4 [heads][rows][ROWS]; v: float32 [heads][rows][P]; out: float32 [rows][heads * P].
 // `col_slices` CTAs share the columns of a head (it must divide P).
-IB_EXPORT int ib_wkv_scan(const void* f, const float* v, int n_rows, float* state, long long state_stride,
-                          const int* cu_rows, const int* slot_ids, float* out, int n_entries, int heads, int P,
-                          int col_slices, void* stream) {
+template <bool GLA>
+static int launch_wkv(const void* f, const float* v, int n_rows, float* state, long long state_stride,
+                      const int* cu_rows, const int* slot_ids, float* out, int n_entries, int heads, int P,
+                      int col_slices, void* stream) {
     if (n_entries <= 0) return IB_OK;
     if (!f || !v || !state || !cu_rows || !slot_ids || !out || heads <= 0 || ((uintptr_t)f & 15)) return IB_ERR_BAD_ARG;
     int cols, threads;
@@ -392,11 +403,25 @@ IB_EXPORT int ib_wkv_scan(const void* f, const float* v, int n_rows, float* stat
     WkvParams p{(const float4*)f, v, n_rows, state, state_stride, cu_rows, slot_ids, out, heads, P, cols};
     const size_t smem = 2 * ((size_t)CHUNK_WKV * ROWS * sizeof(float4) + (size_t)CHUNK_WKV * cols * sizeof(float));
     if (smem > 48 * 1024) return IB_ERR_TOO_LARGE;
-    cudaError_t le = launch_kernel_in_order(wkv_scan_kernel, dim3(n_entries, heads, col_slices), dim3(threads), smem,
+    cudaError_t le = launch_kernel_in_order(wkv_scan_kernel<GLA>, dim3(n_entries, heads, col_slices), dim3(threads), smem,
                                    (cudaStream_t)stream, p);
     if (le != cudaSuccess) return (int)le;
     IB_LAUNCH_CHECK();
     return IB_OK;
+}
+
+IB_EXPORT int ib_wkv_scan(const void* f, const float* v, int n_rows, float* state, long long state_stride,
+                          const int* cu_rows, const int* slot_ids, float* out, int n_entries, int heads, int P,
+                          int col_slices, void* stream) {
+    return launch_wkv<false>(f, v, n_rows, state, state_stride, cu_rows, slot_ids, out, n_entries, heads, P, col_slices,
+                             stream);
+}
+
+IB_EXPORT int ib_gla_scan(const void* f, const float* v, int n_rows, float* state, long long state_stride,
+                          const int* cu_rows, const int* slot_ids, float* out, int n_entries, int heads, int P,
+                          int col_slices, void* stream) {
+    return launch_wkv<true>(f, v, n_rows, state, state_stride, cu_rows, slot_ids, out, n_entries, heads, P, col_slices,
+                            stream);
 }
 
 // x: float32 [heads][rows][P]; bc: float2 [groups][rows][ROWS]; dd: float2 [heads][rows];

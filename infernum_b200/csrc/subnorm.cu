@@ -14,11 +14,11 @@
 
 using namespace ib;
 
-// Token embedding into the 32-bit stream and, when asked, its copy in the
+// Token embedding, times `scale`, into the 32-bit stream and, when asked, its copy in the
 // activation dtype (sub-layers of this arrangement read the stream itself).
 template <typename TW, typename TA>
 __global__ void embed_dual_kernel(const int* __restrict__ ids, const TW* __restrict__ table,
-                                  float* __restrict__ out, TA* __restrict__ act, int H, int V,
+                                  float* __restrict__ out, TA* __restrict__ act, int H, int V, float scale,
                                   unsigned* __restrict__ err) {
     pdl_trigger();
     pdl_wait();
@@ -30,14 +30,14 @@ __global__ void embed_dual_kernel(const int* __restrict__ ids, const TW* __restr
     if (bad && threadIdx.x == 0) atomicOr(err, IB_FLAG_BAD_TOKEN);
     const TW* src = table + (size_t)(bad ? 0 : id) * H;
     for (int i = threadIdx.x; i < H; i += blockDim.x) {
-        const float v = bad ? 0.f : to_f32(src[i]);
+        const float v = bad ? 0.f : to_f32(src[i]) * scale;
         o[i] = v;
         if (a) a[i] = from_f32<TA>(v);
     }
 }
 
 IB_EXPORT int ib_embed_dual(const int* ids, const void* table, int table_dtype, float* out, void* act, int act_dtype,
-                            int n_rows, int H, int V, unsigned* err, void* stream) {
+                            int n_rows, int H, int V, float scale, unsigned* err, void* stream) {
     if (n_rows <= 0) return IB_OK;
     if (!ids || !table || !out || !err || H <= 0 || V <= 0) return IB_ERR_BAD_ARG;
     cudaStream_t s = (cudaStream_t)stream;
@@ -45,13 +45,13 @@ IB_EXPORT int ib_embed_dual(const int* ids, const void* table, int table_dtype, 
     cudaError_t le;
     if (table_dtype == 0 && (!act || act_dtype == 0))
         le = launch_kernel(embed_dual_kernel<float, float>, dim3(n_rows), dim3(threads), 0, s, ids, (const float*)table,
-                           out, (float*)act, H, V, err);
+                           out, (float*)act, H, V, scale, err);
     else if (table_dtype == 1 && (!act || act_dtype == 1))
         le = launch_kernel(embed_dual_kernel<bf16, bf16>, dim3(n_rows), dim3(threads), 0, s, ids, (const bf16*)table,
-                           out, (bf16*)act, H, V, err);
+                           out, (bf16*)act, H, V, scale, err);
     else if (table_dtype == 0 && act_dtype == 1)
         le = launch_kernel(embed_dual_kernel<float, bf16>, dim3(n_rows), dim3(threads), 0, s, ids, (const float*)table,
-                           out, (bf16*)act, H, V, err);
+                           out, (bf16*)act, H, V, scale, err);
     else
         return IB_ERR_UNSUPPORTED;
     if (le != cudaSuccess) return (int)le;

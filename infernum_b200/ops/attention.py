@@ -37,21 +37,23 @@ def paged_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
 
 
 def latent_attention(q_abs: torch.Tensor, pool: torch.Tensor, out: torch.Tensor, kv_rank: int, ctx,
-                     tables: torch.Tensor, scale: float, window: int, rt) -> None:
+                     tables: torch.Tensor, scale: float, window: int, rt, sink=None, gate=None) -> None:
     """Attention of every head of every row over its request's cached latents.
 
     ``q_abs`` [N, heads, kv_rank + rot_dim] holds each head's query in latent
     space followed by its rotated part; the pool [pages, 1, page_size,
     kv_rank + rot_dim] each token's latent followed by the shared rotated key;
     ``out`` [N, heads, kv_rank] receives the weighted sums of latents.  Rows and
-    heads may lie in any order in memory (strides).  bfloat16 engines take the
+    heads may lie in any order in memory (strides).  ``sink`` (float32 [heads]): a logit
+    per head whose exponential is added to the softmax's denominator; ``gate`` ([N, heads]):
+    a head's result is multiplied by its sigmoid.  bfloat16 engines take the
     tensor-core kernel when the sizes have a variant, everything else the plain
     32-bit kernel; ``rt.options["attention"] = "plain"`` forces the latter."""
     impl = rt.options.get("attention", "auto")
     if q_abs.dtype == torch.bfloat16 and impl != "plain":
         from . import attention_latent
 
-        if attention_latent.run(q_abs, pool, out, kv_rank, ctx, tables, scale, window, rt):
+        if attention_latent.run(q_abs, pool, out, kv_rank, ctx, tables, scale, window, rt, sink=sink, gate=gate):
             return
     core.attention_latent_plain(q_abs, pool, out, kv_rank, ctx.positions, ctx.row_entry, tables, scale,
-                                window, rt.err)
+                                window, rt.err, sink=sink, gate=gate)

@@ -41,7 +41,7 @@ def lib_for(kv_rank: int, width: int) -> ctypes.CDLL:
         lib.ib_attention_latent.argtypes = [
             _c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int,
             _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_void_p, _c_ll,
-            _c_void_p, _c_void_p]
+            _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p]
         lib.ib_attention_latent.restype = _c_int
         lib.ib_attention_latent_scratch_bytes.argtypes = [_c_int, _c_int, _c_int]
         lib.ib_attention_latent_scratch_bytes.restype = _c_ll
@@ -70,7 +70,7 @@ def choose_plan(rows_per_entry, heads: int, max_kv_len: int, window: int, kv_ran
 
 
 def run(q_abs: torch.Tensor, pool: torch.Tensor, out: torch.Tensor, kv_rank: int, ctx, tables: torch.Tensor,
-        scale: float, window: int, rt) -> bool:
+        scale: float, window: int, rt, sink=None, gate=None) -> bool:
     num_pages, one, page_size, width = pool.shape
     N, heads, _ = q_abs.shape
     if not supported(kv_rank, width) or q_abs.dtype != torch.bfloat16:
@@ -78,7 +78,8 @@ def run(q_abs: torch.Tensor, pool: torch.Tensor, out: torch.Tensor, kv_rank: int
     if q_abs.stride(0) % 8 or q_abs.stride(1) % 8 or out.stride(0) % 2 or out.stride(1) % 2 \
             or q_abs.data_ptr() % 16 or pool.data_ptr() % 16 or out.data_ptr() % 4:
         return False
-    core.require_cuda(q_abs, pool, out, tables)
+    core.require_cuda(q_abs, pool, out, tables, sink, gate)
+    core.check_sink_and_gate(sink, gate, q_abs, "attention_latent")
     key = ("latent_plan", heads, kv_rank, width, int(window))
     plan = ctx.scratch.get(key)
     if plan is None:
@@ -102,6 +103,8 @@ def run(q_abs: torch.Tensor, pool: torch.Tensor, out: torch.Tensor, kv_rank: int
         q_abs.data_ptr(), q_abs.stride(0), q_abs.stride(1), pool.data_ptr(), out.data_ptr(), out.stride(0),
         out.stride(1), ctx.cu_rows.data_ptr(), ctx.q_start.data_ptr(), tables.data_ptr(), tables.shape[1],
         ctx.n_entries, N, ctx.max_rows_per_entry, heads, page_size, num_pages, int(window), float(scale), mt, splits,
-        scratch_ptr, scratch_bytes, rt.err.data_ptr(), core.stream_ptr(q_abs))
+        scratch_ptr, scratch_bytes, sink.data_ptr() if sink is not None else None,
+        gate.data_ptr() if gate is not None else None, gate.stride(0) if gate is not None else 0, rt.err.data_ptr(),
+        core.stream_ptr(q_abs))
     core.check(code, "attention_latent_mma")
     return True

@@ -87,7 +87,7 @@ def core_lib() -> ctypes.CDLL:
         lib.ib_attention_plain_mask.argtypes = lib.ib_attention_plain.argtypes[:19] + [
             _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_void_p, _c_void_p]
         lib.ib_embed_dual.argtypes = [_c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int,
-                                      _c_void_p, _c_void_p]
+                                      _c_float, _c_void_p, _c_void_p]
         lib.ib_sub_norm_add.argtypes = [_c_void_p, _c_void_p, _c_int, _c_void_p, _c_float, _c_void_p, _c_int, _c_void_p,
                                         _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_void_p]
         lib.ib_part_rmsnorm.argtypes = [_c_void_p, _c_void_p, _c_void_p, _c_float, _c_void_p, _c_int, _c_int, _c_int,
@@ -100,7 +100,12 @@ def core_lib() -> ctypes.CDLL:
                                             _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p]
         lib.ib_moe_route_scored.argtypes = [_c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
                                             _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p]
-        for fn in ("ib_attention_plain_mask", "ib_embed_dual", "ib_sub_norm_add", "ib_part_rmsnorm", "ib_delta_prepare",
+        lib.ib_attention_plain_gated.argtypes = lib.ib_attention_plain.argtypes[:19] + [
+            _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_void_p]
+        lib.ib_gla_prepare.argtypes = [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p,
+                                       _c_void_p, _c_void_p, _c_float, _c_float, _c_void_p, _c_void_p, _c_int, _c_int,
+                                       _c_int, _c_int, _c_void_p]
+        for fn in ("ib_attention_plain_gated", "ib_gla_prepare", "ib_attention_plain_mask", "ib_embed_dual", "ib_sub_norm_add", "ib_part_rmsnorm", "ib_delta_prepare",
                    "ib_rope_norm_append", "ib_moe_route_scored"):
             getattr(lib, fn).restype = _c_int
         lib.ib_gemm_plain_batched.argtypes = [_c_void_p, _c_int, _c_int, _c_ll, _c_void_p, _c_int, _c_int, _c_ll,
@@ -157,7 +162,8 @@ def core_lib() -> ctypes.CDLL:
         lib.ib_latent_prepare_ex.argtypes = lib.ib_latent_prepare.argtypes[:22] + [_c_int, _c_float, _c_void_p, _c_void_p]
         lib.ib_latent_q_rotate_ex.argtypes = lib.ib_latent_q_rotate.argtypes[:14] + [_c_int, _c_float, _c_void_p]
         lib.ib_moe_route_softmax_all.argtypes = [_c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p,
-                                                 _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_void_p]
+                                                 _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int,
+                                                 _c_int, _c_void_p]
         lib.ib_moe_combine.argtypes = [_c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int,
                                        _c_int, _c_void_p]
         lib.ib_gated_norm_add.argtypes = [_c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_float,
@@ -182,14 +188,14 @@ def core_lib() -> ctypes.CDLL:
         lib.ib_embed_scaled.argtypes = [_c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_float,
                                         _c_void_p, _c_void_p]
         lib.ib_gated_act_strided.argtypes = [_c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
-                                             _c_float, _c_float, _c_void_p, _c_int, _c_void_p]
+                                             _c_float, _c_float, _c_void_p, _c_int, _c_int, _c_float, _c_void_p]
         lib.ib_add_rmsnorm_pair.argtypes = [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p,
                                             _c_void_p, _c_int, _c_int, _c_int, _c_float, _c_void_p]
         lib.ib_reenter_add.argtypes = [_c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int,
                                        _c_void_p]
         lib.ib_qk_row_norm_append.argtypes = [_c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_int, _c_float, _c_void_p,
                                               _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_int,
-                                              _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p]
+                                              _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p]
         lib.ib_attention_talk.argtypes = [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_void_p,
                                           _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int,
                                           _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
@@ -676,12 +682,12 @@ def softcap(logits: torch.Tensor, cap: float) -> None:
 
 def gated_act(gate_up: torch.Tensor, out: torch.Tensor, activation: str = "silu", block: Optional[int] = None,
               scale: Optional[torch.Tensor] = None, cols_per_scale: int = 0, limit: float = float("inf"),
-              alpha: float = 1.0) -> None:
+              alpha: float = 1.0, limit_col: Optional[int] = None, limit2: float = float("inf")) -> None:
     """out = act(gate) * up for rows [N, 2I] (``block`` as in ``silu_mul``); with
     ``scale`` [N, I / cols_per_scale] (float32) each run of ``cols_per_scale``
     outputs is multiplied by its scale.  ``clamped_swish`` is ``g' sigmoid(alpha g') (u' + 1)``
-    with ``g' = min(g, limit)`` and ``u'`` the up held to [-limit, limit].  The rows of
-    ``out`` may lie in wider ones."""
+    with ``g' = min(g, limit)`` and ``u'`` the up held to [-limit, limit]; from output
+    column ``limit_col`` on the limit is ``limit2``.  The rows of ``out`` may lie in wider ones."""
     require_cuda(gate_up, out, scale)
     N, two_i = gate_up.shape
     if two_i % 2 or out.shape != (N, two_i // 2) or out.dtype != gate_up.dtype \
@@ -698,7 +704,8 @@ def gated_act(gate_up: torch.Tensor, out: torch.Tensor, activation: str = "silu"
         raise KernelError("gated_act: scale must be contiguous float32 [N, I / cols_per_scale]")
     check(core_lib().ib_gated_act_strided(gate_up.data_ptr(), out.data_ptr(), out.stride(0), dtype_code(out.dtype), N, I,
                                           blk, ACTIVATIONS[activation], float(limit), float(alpha), _ptr(scale),
-                                          int(cols_per_scale), stream_ptr(out)), "gated_act")
+                                          int(cols_per_scale), I if limit_col is None else int(limit_col), float(limit2),
+                                          stream_ptr(out)), "gated_act")
 
 
 def embed_hashed(ctx, prev_state: torch.Tensor, table: torch.Tensor, bigram: torch.Tensor, buckets: int,
@@ -791,13 +798,17 @@ def latent_q_rotate(q: torch.Tensor, heads: int, dim: int, rot_dim: int, rotary_
 
 def attention_latent_plain(q_abs: torch.Tensor, pool: torch.Tensor, out: torch.Tensor, kv_rank: int,
                            positions: torch.Tensor, row_entry: torch.Tensor, block_tables: torch.Tensor,
-                           scale: float, window: int, err: torch.Tensor) -> None:
+                           scale: float, window: int, err: torch.Tensor, sink: Optional[torch.Tensor] = None,
+                           gate: Optional[torch.Tensor] = None) -> None:
     """Attention of all heads over one latent cache, in 32-bit: ``q_abs``
     [N, heads, width] holds each head's query in latent space followed by its
     rotated part, the pool [pages, 1, page_size, width] each token's latent
     followed by the shared rotated key; a token's value is its latent.  ``out``
-    [N, heads, kv_rank]."""
-    require_cuda(q_abs, pool, out, positions, row_entry, block_tables, err)
+    [N, heads, kv_rank].  ``sink`` (float32 [heads]): a logit per head more in the softmax's
+    denominator; ``gate`` ([N, heads], a view of wider rows is fine): a head's result is
+    multiplied by its sigmoid."""
+    require_cuda(q_abs, pool, out, positions, row_entry, block_tables, err, sink, gate)
+    check_sink_and_gate(sink, gate, q_abs, "attention_latent_plain")
     _int32(positions, "positions")
     _int32(row_entry, "row_entry")
     _int32(block_tables, "block_tables")
@@ -807,13 +818,24 @@ def attention_latent_plain(q_abs: torch.Tensor, pool: torch.Tensor, out: torch.T
             or not (q_abs.dtype == pool.dtype == out.dtype) or not pool.is_contiguous():
         raise KernelError("attention_latent_plain: q_abs [N, heads, width], pool [pages, 1, page, width] and "
                           "out [N, heads, kv_rank] do not fit")
-    check(core_lib().ib_attention_plain_ex(q_abs.data_ptr(), q_abs.stride(0), pool.data_ptr(), pool.data_ptr(),
-                                           out.data_ptr(), out.stride(0), dtype_code(q_abs.dtype),
-                                           positions.data_ptr(), row_entry.data_ptr(), block_tables.data_ptr(),
-                                           block_tables.shape[1], N, heads, 1, width, page_size, num_pages,
-                                           int(window), float(scale), int(kv_rank), width, q_abs.stride(1),
-                                           out.stride(1), None, err.data_ptr(), stream_ptr(q_abs)),
+    check(core_lib().ib_attention_plain_gated(q_abs.data_ptr(), q_abs.stride(0), pool.data_ptr(), pool.data_ptr(),
+                                              out.data_ptr(), out.stride(0), dtype_code(q_abs.dtype),
+                                              positions.data_ptr(), row_entry.data_ptr(), block_tables.data_ptr(),
+                                              block_tables.shape[1], N, heads, 1, width, page_size, num_pages,
+                                              int(window), float(scale), int(kv_rank), width, q_abs.stride(1),
+                                              out.stride(1), _ptr(sink), 0, _ptr(gate),
+                                              gate.stride(0) if gate is not None else 0, err.data_ptr(),
+                                              stream_ptr(q_abs)),
           "attention_latent_plain")
+
+
+def check_sink_and_gate(sink: Optional[torch.Tensor], gate: Optional[torch.Tensor], q: torch.Tensor, what: str) -> None:
+    """``q`` [N, heads, width]: ``sink`` must be float32 [heads], ``gate`` [N, heads] of its dtype."""
+    N, heads = q.shape[0], q.shape[1]
+    if sink is not None and (sink.dtype != torch.float32 or sink.shape != (heads,) or not sink.is_contiguous()):
+        raise KernelError(f"{what}: sink must be contiguous float32 [{heads}]")
+    if gate is not None and (gate.shape != (N, heads) or gate.stride(1) != 1 or gate.dtype != q.dtype):
+        raise KernelError(f"{what}: gate must be [{N}, {heads}] of the queries' dtype with unit inner stride")
 
 
 def gemm_plain_batched(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
@@ -1021,12 +1043,12 @@ def qk_norm_append(x: torch.Tensor, q_weight: Optional[torch.Tensor], k_weight: 
                                        err.data_ptr(), stream_ptr(x)), "qk_norm_append")
 
 
-_POINTWISE = {"sigmoid_gate": 0, "axpby": 1, "tanh": 2}
+_POINTWISE = {"sigmoid_gate": 0, "axpby": 1, "tanh": 2, "relu2": 3}
 
 
 def pointwise(a: torch.Tensor, b: Optional[torch.Tensor], op: str, ca: float = 1.0, cb: float = 1.0) -> None:
     """In place on ``a`` [N, C] (contiguous): ``sigmoid_gate`` a * sigmoid(b);
-    ``axpby`` ca * a + cb * b; ``tanh`` tanh(a).  ``b`` may be a view of wider rows."""
+    ``axpby`` ca * a + cb * b; ``tanh`` tanh(a); ``relu2`` max(a, 0)^2.  ``b`` may be a view of wider rows."""
     require_cuda(a, b)
     if a.dim() != 2 or not a.is_contiguous() or op not in _POINTWISE:
         raise KernelError("pointwise: a must be contiguous [N, C]; ops: " + ", ".join(sorted(_POINTWISE)))
@@ -1044,8 +1066,8 @@ def pointwise(a: torch.Tensor, b: Optional[torch.Tensor], op: str, ca: float = 1
 # routing by sigmoid scores inside the best groups of experts.
 # ---------------------------------------------------------------------------
 def embed_dual(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor, act: Optional[torch.Tensor],
-               err: torch.Tensor) -> None:
-    """out[t, :] = table[ids[t], :] into a float32 stream and, when given, into
+               err: torch.Tensor, scale: float = 1.0) -> None:
+    """out[t, :] = table[ids[t], :] * scale into a float32 stream and, when given, into
     ``act`` in the activation dtype."""
     require_cuda(ids, table, out, act, err)
     _int32(ids, "ids")
@@ -1057,7 +1079,7 @@ def embed_dual(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor, act: O
         raise KernelError(f"embed_dual: act must be contiguous [{n}, {H}]")
     check(core_lib().ib_embed_dual(ids.data_ptr(), table.data_ptr(), dtype_code(table.dtype), out.data_ptr(),
                                    _ptr(act), dtype_code(act.dtype) if act is not None else 0, n, H, V,
-                                   err.data_ptr(), stream_ptr(out)), "embed_dual")
+                                   float(scale), err.data_ptr(), stream_ptr(out)), "embed_dual")
 
 
 def sub_norm_add(x_in: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, parts: int, eps: float,
@@ -1317,9 +1339,12 @@ def attention_diff(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, 
 
 def moe_route_softmax_all(logits: torch.Tensor, correction: Optional[torch.Tensor], outputs: int, experts: int, top: int,
                           ids: torch.Tensor, weights: torch.Tensor, gate: Optional[torch.Tensor],
-                          extra: Optional[torch.Tensor]) -> None:
+                          extra: Optional[torch.Tensor], groups: int = 1, keep: int = 1, group_top: int = 1,
+                          renorm: bool = True) -> None:
     """Routing by ``s = softmax(logits[:, :outputs])``: the ``top`` largest ``s + correction`` are chosen
-    (lowest index among equals), their weights are ``s`` over the chosen ones' sum (+ 1e-20).  Outputs
+    (lowest index among equals), their weights are ``s`` over the chosen ones' sum (+ 1e-20), or - ``renorm``
+    False - ``s`` as it is.  ``groups`` > 1: only outputs of the ``keep`` best of that many equal groups of
+    neighbours can be chosen, a group scored by the sum of its ``group_top`` largest ``s + correction``.  Outputs
     from ``experts`` on have no expert: their weight is summed into ``extra[:, 0]``.  ``gate`` [N, experts]
     gets the dense weights of the experts that exist.  When ``logits`` has one more column, ``extra[:, 1]``
     is its sigmoid, else 1; a ``gate`` wider than ``experts`` gets that number in its further columns."""
@@ -1339,7 +1364,8 @@ def moe_route_softmax_all(logits: torch.Tensor, correction: Optional[torch.Tenso
     check(core_lib().ib_moe_route_softmax_all(logits.data_ptr(), logits.stride(0), _ptr(correction), int(outputs),
                                               int(experts), int(top), 1 if cols == outputs + 1 else 0, ids.data_ptr(),
                                               weights.data_ptr(), _ptr(gate), _ptr(extra),
-                                              gate.shape[1] if gate is not None else int(experts), N, stream_ptr(logits)),
+                                              gate.shape[1] if gate is not None else int(experts), int(groups), int(keep),
+                                              int(group_top), 1 if renorm else 0, N, stream_ptr(logits)),
           "moe_route_softmax_all")
 
 
@@ -1401,12 +1427,14 @@ def reenter_add(x: torch.Tensor, delta: Optional[torch.Tensor], origin: Optional
 def qk_row_norm_append(x: torch.Tensor, q_weight: Optional[torch.Tensor], k_weight: Optional[torch.Tensor], eps: float,
                        q_scale: Optional[torch.Tensor], inv_freq: Optional[torch.Tensor], rotary_dim: int, n_heads: int, n_kv_heads: int, dim: int,
                        vdim: int, positions: torch.Tensor, row_entry: torch.Tensor, block_tables: torch.Tensor,
-                       k_pool: torch.Tensor, v_pool: torch.Tensor, err: torch.Tensor) -> None:
+                       k_pool: torch.Tensor, v_pool: torch.Tensor, err: torch.Tensor,
+                       value_from_key: bool = False) -> None:
     """Rows of ``x``: ``n_heads`` queries and ``n_kv_heads`` keys of ``dim``, ``n_kv_heads`` values of ``vdim``.
     All of a row's queries are divided by their one root mean square and multiplied by ``q_weight``
     ([n_heads * dim], float32 or bfloat16; None: neither), its keys likewise; the first ``rotary_dim``
     dimensions of every head are rotated (halves paired); query head h is multiplied by ``q_scale[h]``
-    (float32; None: 1).  All of it in 32-bit with one rounding at the end.  Queries are written back, keys and values to their pages."""
+    (float32; None: 1).  All of it in 32-bit with one rounding at the end.  Queries are written back, keys and values to their pages.
+    ``value_from_key``: a token's values are its keys as projected (``vdim`` = ``dim``; the row holds none)."""
     require_cuda(x, q_weight, k_weight, q_scale, inv_freq, positions, row_entry, block_tables, k_pool, v_pool, err)
     _int32(positions, "positions")
     _int32(row_entry, "row_entry")
@@ -1418,7 +1446,10 @@ def qk_row_norm_append(x: torch.Tensor, q_weight: Optional[torch.Tensor], k_weig
         raise KernelError("qk_row_norm_append: both norms' weights must have one dtype")
     _f32_vec(q_scale, n_heads, "qk_row_norm_append: q_scale")
     num_pages, nkv_pool, page_size, d_pool = k_pool.shape
-    if x.dim() != 2 or x.stride(1) != 1 or x.shape[1] < (n_heads + n_kv_heads) * dim + n_kv_heads * vdim:
+    v_off = (n_heads if value_from_key else n_heads + n_kv_heads) * dim
+    if value_from_key and vdim != dim:
+        raise KernelError("qk_row_norm_append: values taken from keys have the keys' size")
+    if x.dim() != 2 or x.stride(1) != 1 or x.shape[1] < v_off + n_kv_heads * vdim:
         raise KernelError("qk_row_norm_append: x rows must hold queries, keys and values with unit inner stride")
     if nkv_pool != n_kv_heads or d_pool != dim or v_pool.shape != (num_pages, n_kv_heads, page_size, vdim) \
             or k_pool.dtype != x.dtype or v_pool.dtype != x.dtype or not k_pool.is_contiguous() \
@@ -1433,7 +1464,7 @@ def qk_row_norm_append(x: torch.Tensor, q_weight: Optional[torch.Tensor], k_weig
                                            float(eps), _ptr(q_scale), _ptr(inv_freq), int(rotary_dim),
                                            positions.data_ptr(), row_entry.data_ptr(), block_tables.data_ptr(), block_tables.shape[1],
                                            k_pool.data_ptr(), v_pool.data_ptr(), x.shape[0], n_heads, n_kv_heads, dim,
-                                           vdim, page_size, num_pages, err.data_ptr(), stream_ptr(x)),
+                                           vdim, v_off, page_size, num_pages, err.data_ptr(), stream_ptr(x)),
           "qk_row_norm_append")
 
 

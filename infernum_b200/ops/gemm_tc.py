@@ -32,6 +32,8 @@ BM, BK = 128, 64
 # the gate's activation in a fused epilogue, as the kernels number them (0: no gated epilogue;
 # ``swiglu=True`` in the calls below is SiLU)
 GATE_CODES = {"silu": 1, "gelu_tanh": 2, "clamped_swish": 3}
+# activations of a product without a gate, as its epilogue takes them
+ALONE_CODES = {"relu2": -1}
 # What a tile of gemm_pair costs beside its width, in weight rows: its token half is
 # fetched and its prologue and epilogue run whatever the width.
 PAIR_TILE_OVERHEAD = 66
@@ -82,7 +84,7 @@ def pair_lib() -> ctypes.CDLL:
         l.ib_gemm_pair.restype = _c_int
         l.ib_gemm_pair_scaled.argtypes = [_c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_int,
                                           _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p,
-                                          _c_int, _c_void_p, _c_void_p, _c_float, _c_float]
+                                          _c_int, _c_void_p, _c_void_p, _c_float, _c_float, _c_int, _c_float]
         l.ib_gemm_pair_scaled.restype = _c_int
         lib()  # the SM count
         _pair_lib = l
@@ -131,7 +133,8 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, splits: Optiona
     """Runs the tcgen05 kernel; raises KernelError if the operands do not fit it.
     ``swiglu``: ``w`` holds, per 128 rows, 64 gate rows then their 64 up rows, and
     ``out`` [T, N/2] receives silu(gate) * up (at most 64 tokens); a code of ``GATE_CODES`` names another
-    activation (``act_limit`` and ``act_alpha`` are the clamped one's)."""
+    activation (``act_limit`` and ``act_alpha`` are the clamped one's), a (negative) code of ``ALONE_CODES`` one
+    that is applied to every value of a product without a gate."""
     core.require_cuda(x, w, out)
     T, K = x.shape
     N = w.shape[0]
@@ -196,13 +199,14 @@ def gemm_pair(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor,
               err: Optional[torch.Tensor] = None, swiglu: bool = False,
               tiling: Optional[Tuple[int, int, int]] = None, token_group: Optional[int] = None,
               scale: Optional[torch.Tensor] = None, cols_per_scale: int = 0, act_limit: float = 0.0,
-              act_alpha: float = 0.0) -> None:
+              act_alpha: float = 0.0, limit_col: Optional[int] = None, act_limit2: float = 0.0) -> None:
     """The product for many tokens: tiles of 256 tokens x up to 256 weight rows,
     each computed by two SMs as one (tcgen05 ``cta_group::2``); bf16 out.
     ``swiglu`` as in ``gemm_tc``, for any number of tokens.  ``scale`` (with
     ``swiglu``; float32 [T, I / cols_per_scale], contiguous): every output is also
     multiplied by ``scale[t, column // cols_per_scale]``, as the outputs of experts
-    side by side are by the weights a token's router gave them."""
+    side by side are by the weights a token's router gave them.  From output column ``limit_col``
+    on (a multiple of 16) the clamped activation's limit is ``act_limit2``."""
     core.require_cuda(x, w, out)
     T, K = x.shape
     N = w.shape[0]
@@ -213,13 +217,14 @@ def gemm_pair(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor,
                 or tuple(scale.shape) != (T, (N // 2) // cols_per_scale):
             raise KernelError(f"gemm_pair: scale must be contiguous float32 [{T}, {(N // 2) // cols_per_scale}]")
         core.require_cuda(scale)
-    bn_a, cols_a, bn_b = tiling or choose_pair_tiling(T, N, POLICY["sm_count"], swiglu)
+    bn_a, cols_a, bn_b = tiling or choose_pair_tiling(T, N, POLICY["sm_count"], int(swiglu) > 0)
     code = pair_lib().ib_gemm_pair_scaled(x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(),
                                           out.stride(0), T, N, K, int(swiglu), bn_a, cols_a, bn_b,
                                           token_group or choose_token_group(T, K), POLICY["sm_count"],
                                           scale.data_ptr() if scale is not None else None, int(cols_per_scale),
                                           (err if err is not None else _error_word(x.device)).data_ptr(),
-                                          core.stream_ptr(x), float(act_limit), float(act_alpha))
+                                          core.stream_ptr(x), float(act_limit), float(act_alpha),
+                                          -(-N // 16) * 16 if limit_col is None else int(limit_col), float(act_limit2))
     core.check(code, "gemm_pair")
 
 
@@ -247,12 +252,12 @@ def route(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, err: Optional[tor
 def swiglu_route(x: torch.Tensor, w_interleaved: torch.Tensor, out: torch.Tensor,
                  err: Optional[torch.Tensor] = None, activation: str = "silu",
                  scale: Optional[torch.Tensor] = None, cols_per_scale: int = 0, act_limit: float = 0.0,
-                 act_alpha: float = 0.0) -> bool:
+                 act_alpha: float = 0.0, limit_col: Optional[int] = None, act_limit2: float = 0.0) -> bool:
     """The gate/up product with SiLU(gate) * up applied in its epilogue, when
     the policy and the operands allow; ``out`` is [T, I].  Up to 64 tokens go to
     the kernel that streams the weights once (decode), prompts to the kernel on
     pairs of SMs when their length suits its tiles (``pair_suits``).  With
-    ``scale`` (see ``gemm_pair``) only the latter is offered."""
+    ``scale`` or a second limit (see ``gemm_pair``) only the latter is offered."""
     mode = POLICY["mode"]
     if mode in ("none", "cublas", "library") or activation not in GATE_CODES:
         return False
@@ -264,16 +269,36 @@ def swiglu_route(x: torch.Tensor, w_interleaved: torch.Tensor, out: torch.Tensor
     T = x.shape[0]
     if scale is not None and (cols_per_scale <= 0 or cols_per_scale % 16):
         return False
+    if limit_col is not None and limit_col % 16:
+        return False
     if T <= min(POLICY["max_tokens"], 64):
-        if scale is not None:
+        if scale is not None or limit_col is not None:
             return False
         gemm_tc(x, w_interleaved, out, splits=1, swiglu=code, err=err, act_limit=act_limit, act_alpha=act_alpha)
         return True
     if pair_suits(T, fused_activation=True):
         gemm_pair(x, w_interleaved, out, swiglu=code, err=err, scale=scale, cols_per_scale=cols_per_scale,
-                  act_limit=act_limit, act_alpha=act_alpha)
+                  act_limit=act_limit, act_alpha=act_alpha, limit_col=limit_col, act_limit2=act_limit2)
         return True
     return False
+
+
+def act_route(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, activation: str,
+              err: Optional[torch.Tensor] = None) -> bool:
+    """``route`` with an activation of ``ALONE_CODES`` in the product's epilogue; what ``route`` would leave
+    to the library is left to the caller."""
+    mode = POLICY["mode"]
+    if mode in ("none", "cublas", "library") or activation not in ALONE_CODES or not eligible(x, w, out):
+        return False
+    T, code = x.shape[0], ALONE_CODES[activation]
+    if T > POLICY["max_tokens"]:
+        if pair_suits(T) and out.dtype == torch.bfloat16 and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0:
+            gemm_pair(x, w, out, err=err, swiglu=code)
+            return True
+        if mode != "all":
+            return False
+    gemm_tc(x, w, out, err=err, swiglu=code)
+    return True
 
 
 def error_flags(device) -> int:

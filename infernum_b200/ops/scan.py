@@ -1,7 +1,7 @@
 """The scans of recurrent mixers (``scan.cu``): one compiled module per number
 of rows of the per-head state matrix, built when a model first needs it.
 
-``wkv_scan``, ``ssd_scan`` and ``delta_scan`` walk every entry's rows in order from the state in
+``wkv_scan``, ``gla_scan``, ``ssd_scan`` and ``delta_scan`` walk every entry's rows in order from the state in
 the request's slot and leave the new state there; what they need to know about
 the step (entries, slots) they read from the step's device tensors, so a
 recorded step replays them for other requests.
@@ -36,7 +36,8 @@ def lib_for(rows: int) -> ctypes.CDLL:
                                     _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p]
         lib.ib_delta_scan.argtypes = [_c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_ll, _c_void_p, _c_void_p,
                                       _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p]
-        for fn in ("ib_wkv_scan", "ib_ssd_scan", "ib_delta_scan", "ib_scan_rows", "ib_scan_split"):
+        lib.ib_gla_scan.argtypes = lib.ib_wkv_scan.argtypes
+        for fn in ("ib_wkv_scan", "ib_gla_scan", "ib_ssd_scan", "ib_delta_scan", "ib_scan_rows", "ib_scan_split"):
             getattr(lib, fn).restype = _c_int
         if lib.ib_scan_rows() != rows:
             raise KernelError(f"scan module for {rows} state rows was built for another size")
@@ -105,6 +106,54 @@ def wkv_scan(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: torch.Tensor,
     core.check(lib.ib_wkv_scan(factors.data_ptr(), v32.data_ptr(), N, ptr, stride, ctx.cu_rows.data_ptr(),
                                ctx.slot_ids.data_ptr(), out.data_ptr(), ctx.n_entries, heads, K, slices,
                                core.stream_ptr(r)), "wkv_scan")
+
+
+# Up to this rank the pass before ``gla_scan`` makes the decays' low-rank product itself.
+GLA_FUSED_RANK = 64
+
+
+def gla_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, lo_off: int, w2: torch.Tensor,
+             bias: Optional[torch.Tensor], tau: float, state: torch.Tensor, state_offset: int, ctx, out: torch.Tensor,
+             heads: int, dim: int, vdim: int, rt) -> None:
+    """Gated linear attention.  Per head, with S [dim, vdim] from ``state[slot, offset:]`` (stored column by
+    column): ``S <- diag(a_t) S + k_t v_t^T``, ``o_t = S^T q_t dim^-1/2``, with a decay per key channel
+    ``a = sigmoid(w2 lo + bias)^(1 / tau)``.  A row of ``proj`` holds q, k (heads x dim each), v (heads x vdim)
+    and ``lo`` ([w2's rank]) at four columns; ``w2`` [heads * dim, rank] in ``proj``'s dtype, ``bias`` float32.
+    ``out`` float32 [N, heads * vdim].  Two kernels as for the other scans: the parallel pass (with the
+    product by ``w2`` when its rank is at most ``GLA_FUSED_RANK``) and the scan."""
+    core.require_cuda(proj, w2, bias, state, out)
+    N, rank = proj.shape[0], w2.shape[1]
+    hk, hp = heads * dim, heads * vdim
+    if proj.dim() != 2 or proj.stride(1) != 1 or min(q_off, k_off, v_off, lo_off) < 0 \
+            or max(q_off + hk, k_off + hk, v_off + hp, lo_off + rank) > proj.shape[1]:
+        raise KernelError("gla_scan: the projected rows do not hold q, k, v and the decay's low-rank values")
+    if w2.shape[0] != hk or w2.dtype != proj.dtype or not w2.is_contiguous():
+        raise KernelError(f"gla_scan: w2 must be contiguous [{hk}, rank] of the rows' dtype")
+    if bias is not None and (bias.dtype != torch.float32 or bias.shape != (hk,) or not bias.is_contiguous()):
+        raise KernelError(f"gla_scan: bias must be contiguous float32 [{hk}]")
+    if out.shape != (N, hp) or out.dtype != torch.float32 or not out.is_contiguous():
+        raise KernelError("gla_scan: out must be contiguous float32 [N, heads * vdim]")
+    if not tau > 0:
+        raise KernelError(f"gla_scan: tau {tau} must be positive")
+    lib = lib_for(dim)
+    z = None
+    if rank > GLA_FUSED_RANK:
+        from ..parts.linear import matmul_nt
+
+        z = matmul_nt(proj[:, lo_off: lo_off + rank], w2, torch.float32, err=rt.err)
+    factors = torch.empty((heads, N, dim, 4), dtype=torch.float32, device=proj.device)
+    v32 = torch.empty((heads, N, vdim), dtype=torch.float32, device=proj.device)
+    core.check(core.core_lib().ib_gla_prepare(
+        proj.data_ptr(), proj.stride(0), core.dtype_code(proj.dtype), int(q_off), int(k_off), int(v_off), int(lo_off),
+        rank, w2.data_ptr(), bias.data_ptr() if bias is not None else None, z.data_ptr() if z is not None else None,
+        dim ** -0.5, 1.0 / float(tau), factors.data_ptr(), v32.data_ptr(), N, heads, dim, vdim, core.stream_ptr(proj)),
+        "gla_prepare")
+    ptr, stride = _state_ptr(state, state_offset)
+    sm = rt.options.get("sm_count") or SM_COUNT_FALLBACK
+    slices = choose_col_slices(ctx.n_entries, heads, vdim, lib.ib_scan_split(), sm)
+    core.check(lib.ib_gla_scan(factors.data_ptr(), v32.data_ptr(), N, ptr, stride, ctx.cu_rows.data_ptr(),
+                               ctx.slot_ids.data_ptr(), out.data_ptr(), ctx.n_entries, heads, vdim, slices,
+                               core.stream_ptr(proj)), "gla_scan")
 
 
 def ssd_scan(xbc: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor, d_skip: torch.Tensor,

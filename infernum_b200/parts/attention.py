@@ -20,13 +20,17 @@ another run named by the schedule).
 
 Options beyond the Llama layer, all off by default:
 ``names`` (the tensors' names behind the prefix: ``q``, ``k``, ``v``, ``o``);
-``qk_norm`` ({"q": name, "k": name, "eps": e}): queries and keys are divided by
-their root mean square per head and multiplied by a weight of ``head_dim``
-values that all heads share, before the scores;
+``qk_norm`` ({"q": name, "k": name, "eps": e, "over": "head" | "projection"}): "head"
+(default): queries and keys are divided by their root mean square per head and
+multiplied by a weight of ``head_dim`` values that all heads share, before the
+scores; "projection": all of a token's queries are divided by their one root mean
+square and multiplied by a weight of their size, its keys likewise, before a
+rotary ``position``, which only this form combines with;
 ``value_from_key`` (True: there is no value projection; a token's value is its
 key as projected, before any norm);
 ``sink`` (a tensor name: one learned logit per head whose exponential is added
-to the softmax's denominator; it has no key and no value and is not scaled);
+to the softmax's denominator; it has no key and no value and is not scaled), or
+``sink_logit`` (the same with one constant for every head: 0 adds a one);
 ``gate`` (a tensor name: the concatenated heads are multiplied by
 ``sigmoid(W_gate x)`` before the output projection);
 ``v_head_dim`` (the size of a value head when it differs from a key's);
@@ -80,6 +84,10 @@ class Attention(Mixer):
         if qk_norm:
             self.qk_norm = {"q": self.prefix + qk_norm["q"], "k": self.prefix + qk_norm["k"],
                             "eps": float(qk_norm["eps"])}
+        over = qk_norm.get("over", "head") if qk_norm else "head"
+        if over not in ("head", "projection"):
+            raise ConfigError(f"attention: queries and keys cannot be normed over {over!r} (head, projection)")
+        self.row_norm = over == "projection"
         self.value_from_key = bool(params.get("value_from_key", False))
         self.v_head_dim = int(params.get("v_head_dim") or self.head_dim)
         self.keep_first = int(params.get("keep_first") or 0) if self.window > 0 else 0
@@ -90,10 +98,15 @@ class Attention(Mixer):
         self.fused_prep = bool(self.bias_names or self.unit_norm or self.v_head_dim != self.head_dim)
         self.bias = None
         self.sink_name = self.prefix + params["sink"] if params.get("sink") else None
+        self.sink_logit = params.get("sink_logit")
+        if self.sink_name and self.sink_logit is not None:
+            raise ConfigError("attention: a sink is either a tensor or a constant")
         self.gate_name = self.prefix + params["gate"] if params.get("gate") else None
-        if (self.qk_norm or self.value_from_key) and self.position is not None:
-            raise ConfigError("attention: normed queries and keys, or values taken from keys, "
+        if (self.qk_norm or self.value_from_key) and self.position is not None and not self.row_norm:
+            raise ConfigError("attention: queries and keys normed per head, or values taken from keys, "
                               "are not combined with a position encoding")
+        if self.row_norm and self.position is not None and not isinstance(self.position, RotaryEmbedding):
+            raise ConfigError("attention: norms over the whole projection go with a rotary position encoding or none")
         if self.fused_prep and (self.qk_norm or self.value_from_key or self.kv_shared or self.gate_name):
             raise ConfigError("attention: biases, weightless norms after the rotation or values of another size "
                               "are not combined with weighted norms, values taken from keys, a gate or a shared cache")
@@ -127,8 +140,8 @@ class Attention(Mixer):
             for k, n in ((("q"), qd), ("k", kvd), ("v", vd)):
                 specs[self.bias_names[k]] = WeightSpec((n,), init="normal", std=0.1)
         if self.qk_norm:
-            specs[self.qk_norm["q"]] = WeightSpec((self.head_dim,), init="norm")
-            specs[self.qk_norm["k"]] = WeightSpec((self.head_dim,), init="norm")
+            specs[self.qk_norm["q"]] = WeightSpec((qd if self.row_norm else self.head_dim,), init="norm")
+            specs[self.qk_norm["k"]] = WeightSpec((kvd if self.row_norm else self.head_dim,), init="norm")
         if self.sink_name:
             specs[self.sink_name] = WeightSpec((self.num_heads,), init="normal", std=1.0)
         if self.gate_name:
@@ -145,8 +158,13 @@ class Attention(Mixer):
         self.qkv = Linear(torch.cat(mats, dim=0) if len(mats) > 1 else mats[0], self.rt)
         self.o = Linear(weights[self.names["o"]], self.rt)
         if self.qk_norm:
-            self.q_norm_w = weights[self.qk_norm["q"]].to(torch.float32).contiguous()
-            self.k_norm_w = weights[self.qk_norm["k"]].to(torch.float32).contiguous()
+            self.q_norm_w, self.k_norm_w = (weights[self.qk_norm[k]].contiguous() for k in ("q", "k"))
+            # (norms over the whole projection keep their weights as stored: a row reads all of them)
+            if not self.row_norm or self.q_norm_w.dtype != self.k_norm_w.dtype:
+                self.q_norm_w, self.k_norm_w = self.q_norm_w.to(torch.float32), self.k_norm_w.to(torch.float32)
+        if self.sink_logit is not None:
+            self.sink = torch.full((self.num_heads,), float(self.sink_logit), dtype=torch.float32,
+                                   device=self.qkv.weight.device)
         if self.sink_name:
             self.sink = weights[self.sink_name].to(torch.float32).contiguous()
         if self.bias_names:
@@ -180,6 +198,15 @@ class Attention(Mixer):
                                   bool(self.unit_norm and self.unit_norm["value"]),
                                   self.unit_norm["eps"] if self.unit_norm else 1e-6, nh, nkv, hd, ctx.positions,
                                   ctx.row_entry, tables, cache.k_pool, cache.v_pool, self.rt.err)
+            return self._attend(qkv, ctx, cache, tables)
+        if self.row_norm:
+            if not cache.owner:
+                raise ConfigError("attention with normed keys must own its cache")
+            rotary = self.position
+            core.qk_row_norm_append(qkv, self.q_norm_w, self.k_norm_w, self.qk_norm["eps"], None,
+                                    rotary.inv_freq if rotary else None, rotary.rotary_dim if rotary else 0, nh, nkv, hd,
+                                    hd, ctx.positions, ctx.row_entry, tables, cache.k_pool, cache.v_pool, self.rt.err,
+                                    value_from_key=self.value_from_key)
             return self._attend(qkv, ctx, cache, tables)
         if self.qk_norm or self.value_from_key:
             if not cache.owner:

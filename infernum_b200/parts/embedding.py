@@ -33,7 +33,7 @@ class TokenEmbedding(Embedding):
     "params"} with ``apply_f32``: the looked-up rows are normed, in 32-bit, before
     they become the stream); ``keep_origin`` (True: the stream keeps the embedding's
     output, as this part leaves it, in ``stream.origin``); ``scale`` (the rows are
-    multiplied by it as they are looked up; not together with ``act`` or ``result_slots``)."""
+    multiplied by it as they are looked up)."""
 
     def __init__(self, params, rt: Runtime):
         super().__init__(params, rt)
@@ -44,8 +44,6 @@ class TokenEmbedding(Embedding):
         self.result_slots = int(params.get("result_slots") or 0)
         self.keep_origin = bool(params.get("keep_origin", False))
         self.scale = float(params.get("scale", 1.0))
-        if self.scale != 1.0 and (self.with_act or self.result_slots):
-            raise ConfigError("token embedding: a scaled embedding keeps no activation copy or results")
         self.norm = None
         if params.get("norm"):
             from .base import NORMS
@@ -78,7 +76,7 @@ class TokenEmbedding(Embedding):
         act = None
         if self.with_act and not self.rt.is_fp32:
             act = torch.empty((n, self.hidden_size), dtype=self.rt.dtype, device=dev)
-        core.embed_dual(ctx.token_ids, self.weight, out, act, self.rt.err)
+        core.embed_dual(ctx.token_ids, self.weight, out, act, self.rt.err, self.scale)
         stream = ResidualStream(out, (out if act is None else act) if self.with_act else None)
         stream.results = results
         return stream

@@ -36,6 +36,13 @@ Without a query latent (``q_rank`` 0 or None) the queries are a projection of
 ``rotary_scaling`` rescales the frequencies (``rope.rotary_inv_freq``) and, for
 "ramp" scaling, multiplies cosine and sine by its magnitude.
 
+``sink`` (a tensor name behind the prefix: one learned logit per head, whose
+exponential is one term more in the softmax's denominator; no key, no value, not
+scaled) and ``gate`` (a tensor name: head h's result is multiplied by
+``sigmoid(W_gate h)_h``; its rows ride in the down product) are off by default.  The
+gate is one number per head, so the attention kernels apply it to the sum of
+latents, before ``W_uv``.
+
 Parameters: ``hidden_size``, ``num_heads``, ``dim``, ``rot_dim``, ``vdim``,
 ``q_rank``, ``kv_rank``, ``scale``, ``window`` (0 = all keys), ``cache_window``
 (default: window), ``eps``, ``rotary_dim`` (default rot_dim), ``theta``,
@@ -82,6 +89,8 @@ class LatentAttention(Mixer):
         self.prefix = params.get("prefix", "")
         names = {**_DEFAULT_NAMES, **(params.get("names") or {})}
         self.names = {k: self.prefix + v for k, v in names.items()}
+        self.sink_name, self.gate_name = (self.prefix + params[k] if params.get(k) else None for k in ("sink", "gate"))
+        self.sink: Optional[torch.Tensor] = None
         scaling = params.get("rotary_scaling")
         self.adjacent = params.get("rotary_pairing", "half") == "adjacent"
         self.magnitude = rotary_magnitude(scaling)
@@ -112,17 +121,27 @@ class LatentAttention(Mixer):
         if not self.kv_shared:
             specs[n["dkv"]] = WeightSpec((self.kv_rank + self.rot_dim, self.hidden_size))
             specs[n["dkv_norm"]] = WeightSpec((self.kv_rank,), init="norm")
+        if self.sink_name:
+            specs[self.sink_name] = WeightSpec((H,), init="normal", std=1.0)
+        if self.gate_name:
+            specs[self.gate_name] = WeightSpec((H, self.hidden_size))
         return specs
 
     def bind(self, weights) -> None:
         H, n = self.num_heads, self.names
-        mats = [weights[n["dq"] if self.q_rank else n["q"]]] + ([] if self.kv_shared else [weights[n["dkv"]]])
+        mats = [weights[n["dq"] if self.q_rank else n["q"]]] + ([] if self.kv_shared else [weights[n["dkv"]]]) \
+            + ([weights[self.gate_name]] if self.gate_name else [])
         if len({m.dtype for m in mats}) != 1:
             raise ConfigError(f"{self.prefix}: the down projections are stored in different dtypes")
-        # both down projections read the same input: one product [dq | c | r]
+        # both down projections and the gate read the same input: one product [dq | c | r | gate]
+        self.gate_off = sum(m.shape[0] for m in mats) - H
+        rows = sum(m.shape[0] for m in mats)
+        if self.gate_name and rows % 8:  # rows of the product 16 bytes apart
+            mats.append(torch.zeros((8 - rows % 8, self.hidden_size), dtype=mats[0].dtype, device=mats[0].device))
         self.down = Linear(torch.cat(mats, dim=0) if len(mats) > 1 else mats[0], self.rt)
         self.uq = Linear(weights[n["uq"]], self.rt) if self.q_rank else None
         self.o = Linear(weights[n["o"]], self.rt)
+        self.sink = weights[self.sink_name].to(torch.float32).contiguous() if self.sink_name else None
         act = self.rt.dtype
         self.q_norm = weights[n["dq_norm"]].to(act).contiguous() if self.q_rank else None
         self.kv_norm = None if self.kv_shared else weights[n["dkv_norm"]].to(act).contiguous()
@@ -144,6 +163,7 @@ class LatentAttention(Mixer):
         tables = ctx.block_tables[cache.group]
         pool = cache.k_pool
         lat = self.down(x)
+        gate = lat[:, self.gate_off: self.gate_off + H] if self.gate_name else None
         if self.q_rank:
             cq = torch.empty((N, self.q_rank), dtype=x.dtype, device=x.device)
             core.latent_prepare(lat, self.q_rank, self.kv_rank, self.rot_dim, self.rotary_dim, self.q_norm,
@@ -168,7 +188,7 @@ class LatentAttention(Mixer):
         batched_matmul_nt(q3[:, :, : self.dim].transpose(0, 1), self.uk_t, q_abs[:, :, : self.kv_rank])
         o_lat = torch.empty((H, N, self.kv_rank), dtype=x.dtype, device=x.device)
         attn_ops.latent_attention(q_abs.transpose(0, 1), pool, o_lat.transpose(0, 1), self.kv_rank, ctx, tables,
-                                  self.scale, self.window, self.rt)
+                                  self.scale, self.window, self.rt, sink=self.sink, gate=gate)
         o = torch.empty((N, H, self.vdim), dtype=x.dtype, device=x.device)
         batched_matmul_nt(o_lat, self.uv, o.transpose(0, 1))
         return self.o(o.view(N, H * self.vdim))

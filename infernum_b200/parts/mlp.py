@@ -1,4 +1,10 @@
-"""SwiGLU feed-forward: ``d = (silu(x Wg^T) * (x Wu^T)) Wd^T`` with
+"""Feed-forwards.
+
+``mlp``: without a gate, ``y = act(W_up x) W_down^T``.  Parameters: ``hidden_size``,
+``intermediate_size``, ``prefix``, ``names`` (of the two tensors behind the prefix: ``up``,
+``down``), ``activation``: "relu2", the square of what relu leaves.
+
+``swiglu``: SwiGLU feed-forward: ``d = (silu(x Wg^T) * (x Wu^T)) Wd^T`` with
 ``silu(g) = g / (1 + exp(-g))`` evaluated in 32-bit
 (infernum-llama/src/graph_builder.rs:498-501; infernum-cuda/kernels/silu.cu:105-116).
 Gate and up are one product.  When the intermediate size is a multiple of 64
@@ -26,7 +32,48 @@ import torch
 from ..errors import ConfigError
 from ..ops import core
 from .base import FEED_FORWARDS, FeedForward, Runtime, WeightSpec
-from .linear import Linear
+from .linear import Linear, matmul_nt
+
+
+@FEED_FORWARDS.register("mlp")
+class Mlp(FeedForward):
+    def __init__(self, params, rt: Runtime):
+        super().__init__(params, rt)
+        self.hidden_size = int(params["hidden_size"])
+        self.intermediate_size = int(params["intermediate_size"])
+        prefix, names = params.get("prefix", ""), params.get("names") or {}
+        self.names = {k: prefix + names.get(k, k) for k in ("up", "down")}
+        self.activation = params.get("activation", "relu2")
+        if self.activation != "relu2":
+            raise ConfigError(f"feed-forward: unknown activation {self.activation!r}; known: relu2")
+        self.up: Optional[Linear] = None
+        self.down: Optional[Linear] = None
+
+    def weight_specs(self) -> Dict[str, WeightSpec]:
+        h, i = self.hidden_size, self.intermediate_size
+        return {self.names["up"]: WeightSpec((i, h)), self.names["down"]: WeightSpec((h, i))}
+
+    def bind(self, weights) -> None:
+        self.up, self.down = (Linear(weights[self.names[k]], self.rt) for k in ("up", "down"))
+
+    def weight_bytes(self) -> int:
+        return self.up.nbytes + self.down.nbytes
+
+    @property
+    def out_proj(self) -> Linear:
+        return self.down
+
+    def forward(self, x: torch.Tensor, ctx=None) -> torch.Tensor:
+        act = torch.empty((x.shape[0], self.intermediate_size), dtype=x.dtype, device=x.device)
+        if x.dtype == torch.bfloat16 and self.up.weight.dtype == torch.bfloat16:
+            from ..ops import gemm_tc
+
+            # the activation in the product's epilogue, where the product is the package's own
+            if gemm_tc.act_route(x, self.up.weight, act, self.activation, err=self.up.err):
+                return self.down(act)
+        matmul_nt(x, self.up.weight, out=act, err=self.up.err)
+        core.pointwise(act, None, self.activation)
+        return self.down(act)
 
 
 @FEED_FORWARDS.register("swiglu")

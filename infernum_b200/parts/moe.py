@@ -16,7 +16,7 @@ with the concatenated vector.  Every expert is computed for every token; what
 a token did not choose is multiplied by an exact 0.
 
 Parameters: ``hidden_size``, ``expert_size`` (ff), ``experts``, ``top``,
-``activation`` ("silu" | "gelu_tanh"), ``prefix``, ``expert_names`` (format of
+``activation`` ("silu" | "gelu_tanh" | "clamped_swish" with ``limit`` and ``alpha``), ``prefix``, ``expert_names`` (format of
 an expert's tensors behind the prefix, default "e{e}.{w}" with w in gate, up,
 down), ``router`` and ``router_bias`` (names behind the prefix; bias None for
 none); ``scoring``: "softmax_top" (default, as above) or "sigmoid": the scores
@@ -28,10 +28,12 @@ the ``keep`` best-scored groups are struck out before the choice;
 "softmax_all": the router has ``experts + identity`` outputs, the scores are the
 softmax over all of them, the ``top`` largest ``score + correction`` (a tensor,
 name in ``correction``, or None) are chosen, and their weights are the scores
-without the correction over the chosen ones' sum (+ 1e-20); the last
+without the correction over the chosen ones' sum (+ 1e-20; ``renormalize`` False:
+as they are); ``groups`` as above, scored by the sum of the ``top`` largest choice
+values (1: the best expert's); the last
 ``identity`` outputs have no expert and no tensors: choosing one adds the
 weight times the token's input.  ``shared`` ({"size", "prefix", "gate"}): one more
-gated feed-forward that every token uses, added times ``sigmoid(w_gate . x)``
+gated feed-forward that every token uses, with a ``limit`` of its own, added times ``sigmoid(w_gate . x)``
 (one number per token; ``gate`` names the [1, hidden] tensor behind the shared
 expert's prefix, None: no gate).  When its width is a multiple of an expert's, it
 runs as further columns of the experts' two products, its gate in the dense row
@@ -64,6 +66,8 @@ class MixtureOfExperts(FeedForward):
         self.activation = params.get("activation", "silu")
         if self.activation not in core.ACTIVATIONS:
             raise ConfigError(f"mixture of experts: unknown activation {self.activation!r}")
+        unbounded = lambda v: float("inf") if v is None else float(v)  # noqa: E731
+        self.limit, self.alpha = unbounded(params.get("limit")), float(params.get("alpha", 1.0))
         self.prefix = params.get("prefix", "")
         self.expert_names = params.get("expert_names", "e{e}.{w}")
         self.router_name = self.prefix + params.get("router", "router")
@@ -80,23 +84,25 @@ class MixtureOfExperts(FeedForward):
         self.shared = None
         if shared:
             self.shared = {"size": int(shared["size"]), "prefix": self.prefix + shared.get("prefix", "shared."),
-                           "gate": shared.get("gate")}
+                           "gate": shared.get("gate"), "limit": unbounded(shared.get("limit"))}
         if (self.identity or self.correction_name or self.shared) and self.scoring != "softmax_all":
             raise ConfigError("mixture of experts: outputs without an expert, a correction of the choice and an "
                               "expert for every token go with softmax_all scoring")
-        self.renormalize = bool(params.get("renormalize", False))
+        # (softmax_all renormalizes unless told otherwise, sigmoid scores do not)
+        self.renormalize = bool(params.get("renormalize", self.scoring == "softmax_all"))
         groups = params.get("groups") or {}
         self.group_count = int(groups.get("count", 1))
         self.group_keep = int(groups.get("keep", self.group_count))
         self.group_top = int(groups.get("top", 2))
         if self.group_count > 1:
-            if self.scoring != "sigmoid":
-                raise ConfigError("mixture of experts: groups of experts go with sigmoid scoring")
+            if self.scoring not in ("sigmoid", "softmax_all") or self.identity:
+                raise ConfigError("mixture of experts: groups of experts go with sigmoid or softmax_all scoring, "
+                                  "every router output having an expert")
             if self.experts % self.group_count or not 0 < self.group_keep <= self.group_count \
                     or self.group_keep * (self.experts // self.group_count) < self.top:
                 raise ConfigError(f"mixture of experts: {self.experts} experts in {self.group_count} groups of which "
                                   f"{self.group_keep} stay open cannot give {self.top} choices")
-            if self.experts // self.group_count > 64:
+            if self.group_top > 1 and self.experts // self.group_count > 64:
                 raise ConfigError("mixture of experts: a group of more than 64 experts is beyond the routing kernel")
         self.gate_up: Optional[Linear] = None
         self.down: Optional[Linear] = None
@@ -165,7 +171,8 @@ class MixtureOfExperts(FeedForward):
             if not self.shared_runs:
                 self.shared_ffn = SwiGLU({"hidden_size": h, "intermediate_size": self.shared["size"], "prefix": sp,
                                           "names": {"gate": "gate", "up": "up", "down": "down"},
-                                          "activation": self.activation}, self.rt)
+                                          "activation": self.activation, "limit": self.shared["limit"],
+                                          "alpha": self.alpha}, self.rt)
                 self.shared_ffn.bind(weights)
             if self.shared["gate"]:
                 # the gate's logit is one more row of the router's product
@@ -187,7 +194,8 @@ class MixtureOfExperts(FeedForward):
         if self.scoring == "softmax_all":
             self._extra = torch.empty((n, 2), dtype=torch.float32, device=dev)
             core.moe_route_softmax_all(logits, self.correction, self.experts + self.identity, self.experts, self.top,
-                                       ids, wts, gate, self._extra)
+                                       ids, wts, gate, self._extra, groups=self.group_count, keep=self.group_keep,
+                                       group_top=self.group_top, renorm=self.renormalize)
         elif self.scoring == "sigmoid":
             core.moe_route_scored(logits, self.router_bias, self.top, ids, wts, gate, groups=self.group_count,
                                   keep=self.group_keep, group_top=self.group_top, renorm=self.renormalize)
@@ -199,15 +207,20 @@ class MixtureOfExperts(FeedForward):
         _ids, _wts, gate = self.route(x)
         act = torch.empty((x.shape[0], gate.shape[1] * self.expert_size), dtype=x.dtype, device=x.device)
         fused = False
+        # the columns of an expert that every token uses may have a limit of their own
+        limit_col = self.experts * self.expert_size if self.shared_runs and self.shared["limit"] != self.limit else None
+        limit2 = self.shared["limit"] if limit_col is not None else 0.0
         if self.block == 64 and x.dtype == torch.bfloat16 and self.gate_up.weight.dtype == torch.bfloat16:
             from ..ops import gemm_tc
 
             # prompts: activation and the router's weights in the product's epilogue
             fused = gemm_tc.swiglu_route(x, self.gate_up.weight, act, self.gate_up.err, activation=self.activation,
-                                         scale=gate, cols_per_scale=self.expert_size)
+                                         scale=gate, cols_per_scale=self.expert_size, act_limit=self.limit,
+                                         act_alpha=self.alpha, limit_col=limit_col, act_limit2=limit2)
         if not fused:
             core.gated_act(self.gate_up(x), act, self.activation, block=self.block, scale=gate,
-                           cols_per_scale=self.expert_size)
+                           cols_per_scale=self.expert_size, limit=self.limit, alpha=self.alpha, limit_col=limit_col,
+                           limit2=limit2)
         routed = self.down(act)
         if self.scoring != "softmax_all" or not (self.identity or self.shared_ffn is not None):
             return routed  # (an expert for every token that ran as columns of the products is in there)

@@ -172,7 +172,8 @@ class PartRMSNorm(Norm):
 
     ``add_gated(stream, y, gate, bias, mult)``: ``x + mult * norm(y * sigmoid(gate + bias))``.
 
-    Parameters: ``hidden_size``, ``eps``, ``parts`` (default 1), ``weight``.
+    Parameters: ``hidden_size``, ``eps``, ``parts`` (default 1), ``weight``, ``optional`` (the
+    checkpoint may leave the weight out; the norm is then not used).
     """
 
     def __init__(self, params, rt: Runtime):
@@ -181,14 +182,17 @@ class PartRMSNorm(Norm):
         self.eps = float(params["eps"])
         self.parts = int(params.get("parts", 1))
         self.weight_name = params["weight"]
+        self.optional = bool(params.get("optional", False))
         self.weight: Optional[torch.Tensor] = None
         self._stored_bytes = 0
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
-        return {self.weight_name: WeightSpec((self.hidden_size,), init="norm")}
+        return {self.weight_name: WeightSpec((self.hidden_size,), init="norm", optional=self.optional)}
 
     def bind(self, weights) -> None:
-        w = weights[self.weight_name]
+        w = weights.get(self.weight_name) if self.optional else weights[self.weight_name]
+        if w is None:
+            return
         self._stored_bytes = w.numel() * w.element_size()
         self.weight = w.to(torch.float32).contiguous()
 

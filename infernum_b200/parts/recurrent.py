@@ -15,6 +15,16 @@ Tensors behind the prefix: ``mu.{r,k,v,g,w}`` [hidden], ``r, k, v, g`` [heads*di
 hidden], ``w1`` [rank, hidden], ``w2`` [heads*dim, rank], ``w0`` [heads*dim], ``u``
 [heads, dim], ``norm`` [heads*dim], ``o`` [hidden, heads*dim].
 
+``gla``: gated linear attention.  ``q = W_q h dim^-1/2``, ``k = W_k h`` (heads x dim), ``v = W_v h``
+(heads x vdim), a decay per key channel ``a = sigmoid(W_a2 (W_a1 h) + b)^(1/tau)``.  Per head
+``S <- diag(a_t) S + k_t v_t^T``, ``o_t = S^T q_t`` (``S`` is dim x vdim); ``o`` is divided by its root
+mean square per head, multiplied by ``norm`` (vdim values shared by the heads) and by
+``silu(W_g h)``, and projected by ``W_o``.
+Parameters: ``hidden_size``, ``num_heads``, ``head_dim``, ``vdim``, ``tau``, ``eps``, ``prefix``,
+``decay_rank`` (None: taken from the checkpoint's ``a1``).
+Tensors: ``q, k`` [heads*dim, hidden], ``v, g`` [heads*vdim, hidden], ``a1`` [rank, hidden], ``a2``
+[heads*dim, rank], ``a2.b`` [heads*dim], ``norm`` [vdim], ``o`` [hidden, heads*vdim].
+
 ``ssd``: a selective state space layer with a scalar decay per head.  ``W_in h``
 is laid out ``[z: inner | x: inner | B: groups*state | C: groups*state | dt: heads]``
 (inner = heads * vdim); x, B and C pass a causal convolution per channel and SiLU;
@@ -129,6 +139,76 @@ class WkvMixer(Mixer):
         y = torch.empty((N, self.hk), dtype=x.dtype, device=x.device)
         core.head_norm_gate(o, g, self.norm, self.heads, self.eps, y)
         return self.proj["o"](y)
+
+
+@MIXERS.register("gla")
+class GlaMixer(Mixer):
+    def __init__(self, params, rt: Runtime):
+        super().__init__(params, rt)
+        self.hidden_size = int(params["hidden_size"])
+        self.heads = int(params["num_heads"])
+        self.dim = int(params["head_dim"])
+        self.vdim = int(params.get("vdim") or self.dim)
+        self.tau = float(params.get("tau", 1.0))
+        self.eps = float(params["eps"])
+        self.prefix = params.get("prefix", "")
+        rank = params.get("decay_rank")
+        self.decay_rank = int(rank) if rank else None
+        if self.dim > scan_ops.MAX_ROWS:
+            raise ConfigError(f"gla: a key of {self.dim} channels is beyond {scan_ops.MAX_ROWS}")
+        if not self.tau > 0:
+            raise ConfigError(f"gla: tau {self.tau} must be positive")
+        self.qk, self.inner = self.heads * self.dim, self.heads * self.vdim
+        # rows of the one input product: q | k | v | gate | a1
+        self.off_v = 2 * self.qk
+        self.off_gate = self.off_v + self.inner
+        self.off_a = self.off_gate + self.inner
+
+    def state_spec(self) -> Optional[StateSpec]:
+        return StateSpec((self.heads * self.dim * self.vdim,), torch.float32)
+
+    def weight_specs(self) -> Dict[str, WeightSpec]:
+        p, D = self.prefix, self.hidden_size
+        rank = self.decay_rank if self.decay_rank else -1
+        draw = self.decay_rank or 16
+        return {
+            p + "q": WeightSpec((self.qk, D)), p + "k": WeightSpec((self.qk, D)), p + "v": WeightSpec((self.inner, D)),
+            p + "g": WeightSpec((self.inner, D)),
+            p + "a1": WeightSpec((rank, D), draw_shape=(draw, D)),
+            p + "a2": WeightSpec((self.qk, rank), draw_shape=(self.qk, draw)),
+            p + "a2.b": WeightSpec((self.qk,), init="normal", std=0.5),
+            p + "norm": WeightSpec((self.vdim,), init="norm"),
+            p + "o": WeightSpec((D, self.inner)),
+        }
+
+    def bind(self, weights) -> None:
+        p = self.prefix
+        mats = [weights[p + n] for n in ("q", "k", "v", "g", "a1")]
+        if len({m.dtype for m in mats}) != 1:
+            raise ConfigError(f"{p}: the input projections are stored in different dtypes")
+        if weights[p + "a1"].shape[0] != weights[p + "a2"].shape[1]:
+            raise ConfigError(f"{p}: the decay's two matrices do not share a rank")
+        rows = sum(m.shape[0] for m in mats)
+        if rows % 8:  # rows of the product 16 bytes apart
+            mats.append(torch.zeros((8 - rows % 8, self.hidden_size), dtype=mats[0].dtype, device=mats[0].device))
+        self.w_in = Linear(torch.cat(mats, dim=0), self.rt)
+        self.w_o = Linear(weights[p + "o"], self.rt)
+        self.a2 = weights[p + "a2"].to(self.rt.dtype).contiguous()
+        self.a2_bias = _f32(weights[p + "a2.b"])
+        self.norm = _f32(weights[p + "norm"]).repeat(self.heads)  # the heads share one weight
+
+    def weight_bytes(self) -> int:
+        return self.w_in.nbytes + self.w_o.nbytes + self.a2.numel() * self.a2.element_size()
+
+    def forward(self, x: torch.Tensor, ctx, cache) -> torch.Tensor:
+        N = x.shape[0]
+        proj = self.w_in(x)
+        o = torch.empty((N, self.inner), dtype=torch.float32, device=x.device)
+        scan_ops.gla_scan(proj, 0, self.qk, self.off_v, self.off_a, self.a2, self.a2_bias, self.tau, cache.state, 0, ctx, o,
+                          self.heads, self.dim, self.vdim, self.rt)
+        y = torch.empty((N, self.inner), dtype=x.dtype, device=x.device)
+        core.head_norm_gate(o, proj[:, self.off_gate: self.off_gate + self.inner], self.norm, self.heads, self.eps, y)
+        return self.w_o(y)
 
 
 @MIXERS.register("ssd")

@@ -74,3 +74,5 @@ def _ensure_builtin() -> None:
         from .models import vodatar  # noqa: F401
     if "Menitar" not in _ARCHITECTURES:
         from .models import menitar  # noqa: F401
+    if "Nutatar" not in _ARCHITECTURES:
+        from .models import nutatar  # noqa: F401
