@@ -161,7 +161,7 @@ def gla(h: torch.Tensor, m: Dict, w: Dict[str, torch.Tensor], p: str, eps: float
     e = m.get("vdim") or d
     q = (h @ w[p + "q"].T * d ** -0.5).reshape(T, H, d)
     k, v = (h @ w[p + "k"].T).reshape(T, H, d), (h @ w[p + "v"].T).reshape(T, H, e)
-    a = decays(h, m["tau"], w, p).reshape(T, H, d)
+    a = decays(h, m.get("tau", 1.0), w, p).reshape(T, H, d)
     heads = [rms_norm(decayed_state(q[:, n], k[:, n], v[:, n], a[:, n]), w[p + "norm"], eps) for n in range(H)]
     g = h @ w[p + "g"].T
     return (torch.cat(heads, dim=1) * g * torch.sigmoid(g)) @ w[p + "o"].T
