@@ -523,6 +523,60 @@ def menitar_prefill_flops(cfg: dict, T: int) -> float:
     return total + 2.0 * D * cfg["vocab"]
 
 
+def nutatar_config(width, layers, heads, kv_heads, ff, vocab, q_rank, window=4096, experts=16, top=4):
+    """Layers in fours: attention through a latent (heads of 128 + 64 rotated, values of 128, a latent of 512,
+    frequencies on a ramp, sinks and head gates), the same over the latents that layer cached, window
+    attention whose values are its keys (heads of 128, half of each rotated), and gated linear attention
+    (heads of 64 keys and 128 values).  Feed-forwards alternate: a squared-relu layer of the weights of a
+    gated one (3 ff / 2 columns), and a mixture of experts that does half a dense layer's work in its chosen
+    experts (ff / (2 top) columns each; four groups of which two stay open) and half in a shared one."""
+    lat = {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "q_rank": q_rank, "kv_rank": 512, "scale": 192 ** -0.5,
+           "rot": {"dims": 64, "base": 10000.0,
+                   "scaling": {"factor": 4.0, "original": 2048, "fast": 32.0, "slow": 1.0}}}
+    att = {"heads": heads, "kv_heads": kv_heads, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": window},
+           "rot": {"dims": 64, "base": 500000.0}}
+    gla = {"heads": width // 128, "dim": 64, "vdim": 128, "tau": 16.0}
+    dense = {"kind": "dense", "ff": ff * 3 // 2}
+    moe = {"kind": "moe", "expert": {"ff": ff // (2 * top), "limit": 7.0}, "shared": {"ff": ff // 2, "limit": 5.0},
+           "router": {"experts": experts, "top": top, "groups": {"count": 4, "keep": 2}}}
+    out = []
+    for i in range(layers):
+        kind, mixer = (("latent_attention", lat), ("latent_attention", {**lat, "kv_from": i - i % 4}), ("attention", att),
+                       ("gla", gla))[i % 4]
+        out.append({"type": kind, "mixer": mixer, "mlp": dense if i % 2 == 0 else moe})
+    return {"architecture": "Nutatar", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": 16.0},
+            "layers": out, "max_position": 8192}
+
+
+def nutatar_prefill_flops(cfg: dict, T: int) -> float:
+    """Multiply-adds x 2 of one prompt step: the products (a token's chosen experts and the shared one only),
+    attention in latent space as the engine computes it, the window attention over the keys a query sees, and
+    the recurrence's update and read-out of its state."""
+    D, total = cfg["width"], 0.0
+    for layer in cfg["layers"]:
+        m = layer["mixer"]
+        H = m["heads"]
+        if layer["type"] == "latent_attention":
+            d, r, v, kr, qr = m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"], m["q_rank"]
+            down = qr + H + (0 if "kv_from" in m else kr + r)
+            total += 2.0 * T * (D * down + qr * H * (d + r) + H * d * kr + H * kr * v + H * v * D)
+            total += 2.0 * H * (2 * kr + r) * T * (T + 1) / 2.0
+        elif layer["type"] == "attention":
+            G, d, w = m["kv_heads"], m["dim"], (m.get("mask") or {}).get("size", 0)
+            keys = sum(min(t + 1, w) if w else t + 1 for t in range(T))
+            total += 2.0 * T * D * (2 * H * d + G * d) + 4.0 * H * d * keys
+        else:
+            d, v = m["dim"], m["vdim"]
+            total += 2.0 * T * D * (2 * H * d + 3 * H * v + 16) + 2.0 * T * 16 * H * d + 2.0 * T * H * d * v * 2.5
+        mlp = layer.get("mlp")
+        if mlp and mlp["kind"] == "dense":
+            total += 4.0 * T * D * mlp["ff"]
+        elif mlp:
+            total += 6.0 * T * D * (mlp["expert"]["ff"] * mlp["router"]["top"] + (mlp.get("shared") or {}).get("ff", 0)) \
+                + 2.0 * T * D * mlp["router"]["experts"]
+    return total + 2.0 * D * cfg["vocab"]
+
+
 DESIGN_SIZES = {
     # name: (width, layers, heads, feed-forward, vocabulary, q_rank, llama kv heads)
     "2b-shape": (2048, 8, 16, 8192, 32000, 768, 4),
@@ -533,7 +587,7 @@ DESIGN_SIZES = {
 def design_compare(args, peaks) -> dict:
     """Prefill and decode of the chosen design at a few sizes, and of the decoder it is set beside
     (the Llama decoder; for Bolovik the Nadozen decoder, whose layers also alternate window
-    attention and a recurrent state; for Vodatar the Rugesun decoder, which also has attention
+    attention and a recurrent state; for Vodatar and Nutatar the Rugesun decoder, which also has attention
     through a latent and mixtures of experts) at the same width, depth, heads, feed-forward width and
     vocabulary."""
     import gc
@@ -565,6 +619,11 @@ def design_compare(args, peaks) -> dict:
         elif args.design == "vodatar":
             other = vodatar_config(width, layers, heads, kv_heads, ff, vocab)
             other_flops = vodatar_prefill_flops
+            beside, beside_cfg, beside_flops = "rugesun", rugesun_config(width, layers, heads, ff, vocab, q_rank), \
+                rugesun_prefill_flops
+        elif args.design == "nutatar":
+            other = nutatar_config(width, layers, heads, kv_heads, ff, vocab, q_rank)
+            other_flops = nutatar_prefill_flops
             beside, beside_cfg, beside_flops = "rugesun", rugesun_config(width, layers, heads, ff, vocab, q_rank), \
                 rugesun_prefill_flops
         elif args.design == "menitar":
@@ -689,9 +748,9 @@ def main() -> int:
     ap.add_argument("--only", choices=["decode", "prefill"], default=None,
                     help="run one part only and print its numbers (for profiling)")
     ap.add_argument("--no-cuda-graph", action="store_true", help="launch decode steps kernel by kernel")
-    ap.add_argument("--design", choices=["rugesun", "nadozen", "bolovik", "vodatar", "menitar"], default=None,
+    ap.add_argument("--design", choices=["rugesun", "nadozen", "bolovik", "vodatar", "menitar", "nutatar"], default=None,
                     help="instead of the default workload: prefill and decode of this design at a few sizes,\n"
-                         "beside the Llama decoder (bolovik: the Nadozen decoder; vodatar: the Rugesun decoder) at equal sizes; prints one JSON line {\"design\": ...}")
+                         "beside the Llama decoder (bolovik: the Nadozen decoder; vodatar, nutatar: the Rugesun decoder) at equal sizes; prints one JSON line {\"design\": ...}")
     ap.add_argument("--size", default=None, help="with --design: one of its sizes only")
     ap.add_argument("--only-model", default=None, help="with --design: the design's name, or the name of the one beside it, only")
     args = ap.parse_args()

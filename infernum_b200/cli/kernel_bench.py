@@ -8,6 +8,8 @@ counters (without that flag ncu locks the clocks of a GPU that others share).
     python -m infernum_b200.cli.kernel_bench attention-prefill --tokens 512 --prefix 3584
     python -m infernum_b200.cli.kernel_bench talk-prefill --tokens 2048 --chunk 1024
     python -m infernum_b200.cli.kernel_bench talk-decode --batch 8 --kv-len 1100
+    python -m infernum_b200.cli.kernel_bench gla-scan --tokens 2048 --heads 16 --head-dim 64 --vdim 128
+    python -m infernum_b200.cli.kernel_bench wkv-scan --batch 64 --tokens 1 --heads 32 --head-dim 64
     python -m infernum_b200.cli.kernel_bench qk-row-norm --tokens 2048 --rotary 64
     python -m infernum_b200.cli.kernel_bench norm-pair --tokens 2048 --hidden 4096
     python -m infernum_b200.cli.kernel_bench gemm --tokens 8 --n 4096 --k 4096
@@ -94,7 +96,7 @@ def _attention_case(batch, rows, kv_len, nh, nkv, hd, page_size, device):
 
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawTextHelpFormatter)
-    ap.add_argument("kernel", choices=["attention-decode", "attention-prefill", "talk-decode", "talk-prefill", "gemm", "norm",
+    ap.add_argument("kernel", choices=["attention-decode", "attention-prefill", "talk-decode", "talk-prefill", "gla-scan", "wkv-scan", "gemm", "norm",
                                        "norm-pair", "qk-row-norm", "rope", "silu"])
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--tokens", type=int, default=2048)
@@ -103,6 +105,7 @@ def main(argv=None) -> int:
     ap.add_argument("--heads", type=int, default=32)
     ap.add_argument("--kv-heads", type=int, default=8)
     ap.add_argument("--head-dim", type=int, default=128)
+    ap.add_argument("--vdim", type=int, default=0, help="gla-scan: the size of a value (default: head-dim)")
     ap.add_argument("--chunk", type=int, default=0, help="talk-*: positions in a run that see one another")
     ap.add_argument("--rotary", type=int, default=64, help="qk-row-norm: rotated dimensions of a head")
     ap.add_argument("--hidden", type=int, default=4096)
@@ -187,6 +190,35 @@ def main(argv=None) -> int:
         nbytes, flops = batch * keys * nkv * hd * 2 * 2, batch * 2.0 * nh * (2 * hd + nh) * keys
         out.update(gbs=nbytes / us / 1e3, frac_of_hbm=nbytes / us / 1e3 / peaks["hbm_gbs"]) if decode else \
             out.update(tflops=flops / us / 1e6, frac_of_bf16=flops / us / 1e6 / peaks["bf16_tflops"])
+    elif args.kernel in ("gla-scan", "wkv-scan"):
+        # --batch entries of --tokens tokens each, the pass before the scan and the scan itself
+        from ..ops import scan
+
+        gla, B, T = args.kernel == "gla-scan", args.batch, args.tokens
+        N, v, rank = B * T, (args.vdim or hd) if args.kernel == "gla-scan" else hd, 16
+        n = max(2, int(300e6 / (B * nh * hd * v * 4)) + 1) if B * nh * hd * v * 4 < 300e6 else 2
+        states = [torch.zeros(B + 1, nh * hd * v, device=dev) for _ in range(n)]
+        i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)  # noqa: E731
+        ctx = SimpleNamespace(n_entries=B, n_rows=N, cu_rows=i32([i * T for i in range(B + 1)]), slot_ids=i32(list(range(B))))
+        o = torch.empty(N, nh * v, device=dev)
+        if gla:
+            proj = torch.randn(N, nh * (2 * hd + v) + rank, device=dev).to(torch.bfloat16)
+            w2 = torch.randn(nh * hd, rank, device=dev).to(torch.bfloat16)
+            b = torch.randn(nh * hd, device=dev)
+            fns = [lambda s=s: scan.gla_scan(proj, 0, nh * hd, 2 * nh * hd, nh * (2 * hd + v), w2, b, 16.0, s, 0, ctx, o, nh,
+                                             hd, v, rt) for s in states]
+            made = 4 * nh * hd + nh * v
+            nbytes = N * (proj.shape[1] * 2 + made * 8 + nh * v * 4) + 2 * B * nh * hd * v * 4
+        else:
+            r, k, vv = (torch.randn(N, nh * hd, device=dev).to(torch.bfloat16) for _ in range(3))
+            z = torch.randn(N, nh * hd, device=dev)
+            w0, u = torch.randn(nh * hd, device=dev), torch.randn(nh * hd, device=dev)
+            fns = [lambda s=s: scan.wkv_scan(r, k, vv, z, w0, u, s, 0, ctx, o, nh, rt) for s in states]
+            nbytes = N * nh * hd * (3 * 2 + 4 + 5 * 8 + 4) + 2 * B * nh * hd * hd * 4
+        us = _time(fns, args.reps, args.warmup, not args.no_graph)
+        flops = 2.0 * N * nh * hd * v * (2.5 if gla else 3.0)
+        out.update(batch=B, tokens=T, heads=nh, dim=hd, vdim=v, us=us, gbs=nbytes / us / 1e3,
+                   frac_of_hbm=nbytes / us / 1e3 / peaks["hbm_gbs"], gflops=flops / us / 1e3)
     elif args.kernel == "gemm":
         T, N, K = args.tokens, args.n, args.k
         copies = max(2, int(300e6 / (N * K * 2)) + 1)
