@@ -250,41 +250,48 @@ IB_EXPORT int ib_wkv_prepare(const void* r, const void* k, const void* v, int ld
 // exp(-softplus(-z) / tau), and v in 32-bit, by head: [heads][rows][K] and [heads][rows][P].  A row of `x`
 // holds q | k (heads * K each) and v (heads * P) at three column offsets.  z [rows][heads * K] comes made
 // (`z` float32), or is made here from a low-rank pair: z = W2 lo + bias, `lo` [rank] at another offset of
-// the row, W2 [heads * K, rank].  In the second form a CTA has 128 channels and GLA_ROWS rows: a channel's
-// W2 row is read once for all of them, sixteen of its values at a time.
-constexpr int GLA_ROWS = 8, GLA_PIECE = 16;
+// the row, W2 [heads * K, rank].  A CTA has 128 channels and ROWS rows: a channel's W2 row is read once for
+// all of them, sixteen of its values at a time, the first sixteen before the rows' producer is done.
+constexpr int GLA_PIECE = 16;
 
-template <typename T>
+template <typename T, int ROWS>
 __global__ void __launch_bounds__(128)
 gla_prepare_kernel(const T* __restrict__ x, int ld, int q_off, int k_off, int v_off, int lo_off, int rank,
                    const T* __restrict__ w2, const float* __restrict__ bias, const float* __restrict__ z,
                    float q_scale, float inv_tau, float4* __restrict__ f, float* __restrict__ vo, int heads, int K,
                    int P, int n_rows) {
     pdl_trigger();
-    __shared__ float lo_s[GLA_ROWS][GLA_PIECE];
-    const int c = blockIdx.x * blockDim.x + threadIdx.x, r0 = blockIdx.y * GLA_ROWS;
-    const int nr = min(GLA_ROWS, n_rows - r0);
+    static_assert(ROWS * GLA_PIECE <= 128, "a piece of all rows is one value a thread");
+    __shared__ float lo_s[ROWS][GLA_PIECE];
+    const int c = blockIdx.x * blockDim.x + threadIdx.x, r0 = blockIdx.y * ROWS;
+    const int nr = min(ROWS, n_rows - r0);
     const int hk = heads * K, hp = heads * P;
-    float acc[GLA_ROWS];
+    float acc[ROWS], w[GLA_PIECE];
     const float b = c < hk && bias ? bias[c] : 0.f;
 #pragma unroll
-    for (int r = 0; r < GLA_ROWS; ++r) acc[r] = b;
+    for (int r = 0; r < ROWS; ++r) acc[r] = b;
+    auto fetch_w = [&](int k0) {
+#pragma unroll
+        for (int i = 0; i < GLA_PIECE; ++i) w[i] = c < hk && k0 + i < rank ? to_f32(w2[(size_t)c * rank + k0 + i]) : 0.f;
+    };
+    if (!z) fetch_w(0);
     pdl_wait();
     if (z) {
-        if (c < hk)
-            for (int r = 0; r < nr; ++r) acc[r] += z[(size_t)(r0 + r) * hk + c];
+#pragma unroll
+        for (int r = 0; r < ROWS; ++r)
+            if (c < hk && r < nr) acc[r] += z[(size_t)(r0 + r) * hk + c];
     } else {
         for (int k0 = 0; k0 < rank; k0 += GLA_PIECE) {
             const int n = min(GLA_PIECE, rank - k0);
+            if (k0) {
+                fetch_w(k0);
+                __syncthreads();
+            }
+            const int lr = threadIdx.x / GLA_PIECE, lc = threadIdx.x % GLA_PIECE;
+            if (lr < ROWS) lo_s[lr][lc] = lr < nr && lc < n ? to_f32(x[(size_t)(r0 + lr) * ld + lo_off + k0 + lc]) : 0.f;
             __syncthreads();
-            const int lr = threadIdx.x / GLA_PIECE, lc = threadIdx.x % GLA_PIECE;  // 128 threads: all of the piece
-            lo_s[lr][lc] = lr < nr && lc < n ? to_f32(x[(size_t)(r0 + lr) * ld + lo_off + k0 + lc]) : 0.f;
-            float w[GLA_PIECE];
 #pragma unroll
-            for (int i = 0; i < GLA_PIECE; ++i) w[i] = c < hk && i < n ? to_f32(w2[(size_t)c * rank + k0 + i]) : 0.f;
-            __syncthreads();
-#pragma unroll
-            for (int r = 0; r < GLA_ROWS; ++r)
+            for (int r = 0; r < ROWS; ++r)
 #pragma unroll
                 for (int i = 0; i < GLA_PIECE; ++i) acc[r] = fmaf(w[i], lo_s[r][i], acc[r]);
         }
@@ -292,7 +299,7 @@ gla_prepare_kernel(const T* __restrict__ x, int ld, int q_off, int k_off, int v_
     if (c < hk) {
         const int head = c / K;
 #pragma unroll
-        for (int r = 0; r < GLA_ROWS; ++r) {
+        for (int r = 0; r < ROWS; ++r) {
             if (r >= nr) break;
             const T* xr = x + (size_t)(r0 + r) * ld;
             const float log_a = fminf(acc[r], 0.f) - log1pf(expf(-fabsf(acc[r])));  // log sigmoid(z), never above 0
@@ -302,8 +309,9 @@ gla_prepare_kernel(const T* __restrict__ x, int ld, int q_off, int k_off, int v_
     }
     if (c < hp) {
         const int head = c / P;
-        for (int r = 0; r < nr; ++r)
-            vo[((size_t)head * n_rows + r0 + r) * P + (c - head * P)] = to_f32(x[(size_t)(r0 + r) * ld + v_off + c]);
+#pragma unroll
+        for (int r = 0; r < ROWS; ++r)
+            if (r < nr) vo[((size_t)head * n_rows + r0 + r) * P + (c - head * P)] = to_f32(x[(size_t)(r0 + r) * ld + v_off + c]);
     }
 }
 
@@ -318,17 +326,19 @@ IB_EXPORT int ib_gla_prepare(const void* x, int ld, int act_dtype, int q_off, in
     if (!z && (!w2 || rank <= 0 || lo_off < 0 || lo_off + rank > ld)) return IB_ERR_BAD_ARG;
     cudaStream_t s = (cudaStream_t)stream;
     const int cols = heads * (K > P ? K : P);
-    const dim3 grid((cols + 127) / 128, (n_rows + GLA_ROWS - 1) / GLA_ROWS);
+    const int rows = n_rows <= 64 ? 1 : 8;  // (few rows: a CTA each, the weights come from L2)
+    const dim3 grid((cols + 127) / 128, (n_rows + rows - 1) / rows);
     if (grid.y > 65535) return IB_ERR_TOO_LARGE;
     cudaError_t le;
-    if (act_dtype == 0)
-        le = launch_kernel(gla_prepare_kernel<float>, grid, dim3(128), 0, s, (const float*)x, ld, q_off, k_off, v_off,
-                           lo_off, rank, (const float*)w2, bias, z, q_scale, inv_tau, (float4*)f, vo, heads, K, P, n_rows);
-    else if (act_dtype == 1)
-        le = launch_kernel(gla_prepare_kernel<bf16>, grid, dim3(128), 0, s, (const bf16*)x, ld, q_off, k_off, v_off,
-                           lo_off, rank, (const bf16*)w2, bias, z, q_scale, inv_tau, (float4*)f, vo, heads, K, P, n_rows);
-    else
-        return IB_ERR_UNSUPPORTED;
+#define IB_GLA(T, ROWS)                                                                                               \
+    le = launch_kernel(gla_prepare_kernel<T, ROWS>, grid, dim3(128), 0, s, (const T*)x, ld, q_off, k_off, v_off, lo_off, \
+                       rank, (const T*)w2, bias, z, q_scale, inv_tau, (float4*)f, vo, heads, K, P, n_rows)
+    if (act_dtype == 0 && rows == 1) IB_GLA(float, 1);
+    else if (act_dtype == 0) IB_GLA(float, 8);
+    else if (act_dtype == 1 && rows == 1) IB_GLA(bf16, 1);
+    else if (act_dtype == 1) IB_GLA(bf16, 8);
+    else return IB_ERR_UNSUPPORTED;
+#undef IB_GLA
     if (le != cudaSuccess) return (int)le;
     IB_LAUNCH_CHECK();
     return IB_OK;
