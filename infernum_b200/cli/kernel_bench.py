@@ -199,7 +199,7 @@ def main(argv=None) -> int:
         n = max(2, int(300e6 / (B * nh * hd * v * 4)) + 1) if B * nh * hd * v * 4 < 300e6 else 2
         states = [torch.zeros(B + 1, nh * hd * v, device=dev) for _ in range(n)]
         i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)  # noqa: E731
-        ctx = SimpleNamespace(n_entries=B, n_rows=N, cu_rows=i32([i * T for i in range(B + 1)]), slot_ids=i32(list(range(B))))
+        ctx = SimpleNamespace(n_entries=B, n_rows=N, max_rows_per_entry=T, cu_rows=i32([i * T for i in range(B + 1)]), slot_ids=i32(list(range(B))))
         o = torch.empty(N, nh * v, device=dev)
         if gla:
             proj = torch.randn(N, nh * (2 * hd + v) + rank, device=dev).to(torch.bfloat16)

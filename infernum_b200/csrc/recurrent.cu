@@ -251,7 +251,7 @@ IB_EXPORT int ib_wkv_prepare(const void* r, const void* k, const void* v, int ld
 // holds q | k (heads * K each) and v (heads * P) at three column offsets.  z [rows][heads * K] comes made
 // (`z` float32), or is made here from a low-rank pair: z = W2 lo + bias, `lo` [rank] at another offset of
 // the row, W2 [heads * K, rank].  A CTA has 128 channels and ROWS rows: a channel's W2 row is read once for
-// all of them, sixteen of its values at a time, the first sixteen before the rows' producer is done.
+// all of them, sixteen of its values at a time (with a row a CTA, the first sixteen before the rows' producer is done).
 constexpr int GLA_PIECE = 16;
 
 template <typename T, int ROWS>
@@ -274,7 +274,7 @@ gla_prepare_kernel(const T* __restrict__ x, int ld, int q_off, int k_off, int v_
 #pragma unroll
         for (int i = 0; i < GLA_PIECE; ++i) w[i] = c < hk && k0 + i < rank ? to_f32(w2[(size_t)c * rank + k0 + i]) : 0.f;
     };
-    if (!z) fetch_w(0);
+    if (ROWS == 1 && !z) fetch_w(0);
     pdl_wait();
     if (z) {
 #pragma unroll
@@ -283,12 +283,11 @@ gla_prepare_kernel(const T* __restrict__ x, int ld, int q_off, int k_off, int v_
     } else {
         for (int k0 = 0; k0 < rank; k0 += GLA_PIECE) {
             const int n = min(GLA_PIECE, rank - k0);
-            if (k0) {
-                fetch_w(k0);
-                __syncthreads();
-            }
             const int lr = threadIdx.x / GLA_PIECE, lc = threadIdx.x % GLA_PIECE;
-            if (lr < ROWS) lo_s[lr][lc] = lr < nr && lc < n ? to_f32(x[(size_t)(r0 + lr) * ld + lo_off + k0 + lc]) : 0.f;
+            const float lo = lr < nr && lc < n ? to_f32(x[(size_t)(r0 + lr) * ld + lo_off + k0 + lc]) : 0.f;
+            if (ROWS > 1 || k0) fetch_w(k0);
+            if (k0) __syncthreads();
+            if (lr < ROWS) lo_s[lr][lc] = lo;
             __syncthreads();
 #pragma unroll
             for (int r = 0; r < ROWS; ++r)

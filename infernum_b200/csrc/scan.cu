@@ -84,6 +84,41 @@ __device__ __forceinline__ float split_sum(float v) {
     return v;
 }
 
+// Tokens whose partial sums a wkv or gla scan collects before they meet over the SPLIT lanes of a column.
+#ifdef IB_SCAN_GROUP  // (tuning: -DIB_SCAN_GROUP=n, a power of two up to SPLIT and to a stage's tokens)
+constexpr int GROUP = IB_SCAN_GROUP;
+#else
+constexpr int min3(int a, int b, int c) { return a < b ? (a < c ? a : c) : (b < c ? b : c); }
+constexpr int GROUP = min3(SPLIT, CHUNK_WKV, 16);
+#endif
+static_assert(GROUP <= SPLIT && GROUP <= CHUNK_WKV && (GROUP & (GROUP - 1)) == 0, "a group of tokens is too long");
+
+// v[k] is this lane's share of token k's sum: the lanes of a column hand each other halves of what they
+// hold, so GROUP sums take about as many shuffles as one lane's values instead of log2(SPLIT) each.  A sum is
+// added up in the same order as by split_sum.  Returns the sum of token group_token(part).
+__device__ __forceinline__ float group_sum(float (&v)[GROUP], int part) {
+    int o = 1;
+#pragma unroll
+    for (int n = GROUP / 2; n >= 1; n >>= 1, o <<= 1) {
+        const bool upper = part & o;
+#pragma unroll
+        for (int i = 0; i < n; ++i) {
+            const float give = upper ? v[i] : v[i + n], keep = upper ? v[i + n] : v[i];
+            v[i] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+        }
+    }
+    float s = v[0];
+#pragma unroll
+    for (int p = GROUP; p < SPLIT; p <<= 1) s += __shfl_xor_sync(0xffffffffu, s, p);
+    return s;
+}
+__device__ __forceinline__ int group_token(int part) {
+    int t = 0, o = 1;
+#pragma unroll
+    for (int n = GROUP / 2; n >= 1; n >>= 1, o <<= 1) t += part & o ? n : 0;
+    return t;
+}
+
 template <int BYTES>
 __device__ __forceinline__ void cp_async(void* smem, const void* gmem) {
     const unsigned s = (unsigned)__cvta_generic_to_shared(smem);
@@ -106,8 +141,9 @@ struct WkvParams {
 };
 
 // GLA: the result is read from the state after the token's update, without it (wkv) from the one before,
-// the current token's own share weighted by u.
-template <bool GLA>
+// the current token's own share weighted by u.  GROUPED: tokens in groups while an entry has them (the sums and
+// the state are the same bits without); without it the kernel takes fewer registers, for steps of few tokens an entry.
+template <bool GLA, bool GROUPED>
 __global__ void __launch_bounds__(512) wkv_scan_kernel(const WkvParams p) {
     pdl_wait();
     extern __shared__ float4 smem4[];
@@ -153,8 +189,7 @@ __global__ void __launch_bounds__(512) wkv_scan_kernel(const WkvParams p) {
         __syncthreads();
         const float4* cf = s_f + buf * CHUNK_WKV * ROWS + part;
         const float* cv = s_v + buf * CHUNK_WKV * p.cols + col;
-#pragma unroll UNROLL
-        for (int t = 0; t < nt; ++t) {
+        auto step = [&](int t) {  // one token: this lane's share of the result, and its rows of the state
             const float vj = cv[t * p.cols];
             const float4* f = cf + t * ROWS;
             float acc = 0.f;
@@ -169,7 +204,21 @@ __global__ void __launch_bounds__(512) wkv_scan_kernel(const WkvParams p) {
                     S[ii] = fmaf(q.z, S[ii], q.y * vj);
                 }
             }
-            acc = split_sum(acc);
+            return acc;
+        };
+        int t = 0;
+        if (GROUPED) {
+            for (; t + GROUP <= nt; t += GROUP) {
+                float part_of[GROUP];
+#pragma unroll
+                for (int k = 0; k < GROUP; ++k) part_of[k] = step(t + k);
+                const float acc = group_sum(part_of, part);
+                if (active && part < GROUP) p.out[(size_t)(c0 + t + group_token(part)) * ldo + hp + j0 + col] = acc;
+            }
+        }
+#pragma unroll UNROLL
+        for (; t < nt; ++t) {
+            const float acc = split_sum(step(t));
             if (active && part == 0) p.out[(size_t)(c0 + t) * ldo + hp + j0 + col] = acc;
         }
         __syncthreads();  // this stage is refilled by the fetch after next
@@ -390,11 +439,12 @@ static int scan_geometry(int P, int col_slices, int* cols, int* threads) {
 }
 
 // f: float4 [heads][rows][ROWS]; v: float32 [heads][rows][P]; out: float32 [rows][heads * P].
-// `col_slices` CTAs share the columns of a head (it must divide P).
+// `col_slices` CTAs share the columns of a head (it must divide P).  max_rows: the most rows of an entry, as far as
+// the host knows; it chooses between two forms of one result.
 template <bool GLA>
 static int launch_wkv(const void* f, const float* v, int n_rows, float* state, long long state_stride,
                       const int* cu_rows, const int* slot_ids, float* out, int n_entries, int heads, int P,
-                      int col_slices, void* stream) {
+                      int col_slices, int max_rows, void* stream) {
     if (n_entries <= 0) return IB_OK;
     if (!f || !v || !state || !cu_rows || !slot_ids || !out || heads <= 0 || ((uintptr_t)f & 15)) return IB_ERR_BAD_ARG;
     int cols, threads;
@@ -403,8 +453,10 @@ static int launch_wkv(const void* f, const float* v, int n_rows, float* state, l
     WkvParams p{(const float4*)f, v, n_rows, state, state_stride, cu_rows, slot_ids, out, heads, P, cols};
     const size_t smem = 2 * ((size_t)CHUNK_WKV * ROWS * sizeof(float4) + (size_t)CHUNK_WKV * cols * sizeof(float));
     if (smem > 48 * 1024) return IB_ERR_TOO_LARGE;
-    cudaError_t le = launch_kernel_in_order(wkv_scan_kernel<GLA>, dim3(n_entries, heads, col_slices), dim3(threads), smem,
-                                   (cudaStream_t)stream, p);
+    cudaError_t le = launch_kernel_in_order(GROUP > 1 && max_rows >= GROUP ? wkv_scan_kernel<GLA, (GROUP > 1)>
+                                                                           : wkv_scan_kernel<GLA, false>,
+                                            dim3(n_entries, heads, col_slices), dim3(threads), smem,
+                                            (cudaStream_t)stream, p);
     if (le != cudaSuccess) return (int)le;
     IB_LAUNCH_CHECK();
     return IB_OK;
@@ -412,16 +464,16 @@ static int launch_wkv(const void* f, const float* v, int n_rows, float* state, l
 
 IB_EXPORT int ib_wkv_scan(const void* f, const float* v, int n_rows, float* state, long long state_stride,
                           const int* cu_rows, const int* slot_ids, float* out, int n_entries, int heads, int P,
-                          int col_slices, void* stream) {
+                          int col_slices, int max_rows, void* stream) {
     return launch_wkv<false>(f, v, n_rows, state, state_stride, cu_rows, slot_ids, out, n_entries, heads, P, col_slices,
-                             stream);
+                             max_rows, stream);
 }
 
 IB_EXPORT int ib_gla_scan(const void* f, const float* v, int n_rows, float* state, long long state_stride,
                           const int* cu_rows, const int* slot_ids, float* out, int n_entries, int heads, int P,
-                          int col_slices, void* stream) {
+                          int col_slices, int max_rows, void* stream) {
     return launch_wkv<true>(f, v, n_rows, state, state_stride, cu_rows, slot_ids, out, n_entries, heads, P, col_slices,
-                            stream);
+                            max_rows, stream);
 }
 
 // x: float32 [heads][rows][P]; bc: float2 [groups][rows][ROWS]; dd: float2 [heads][rows];

@@ -31,7 +31,7 @@ def lib_for(rows: int) -> ctypes.CDLL:
             raise KernelError(f"recurrent scan: a state of {rows} rows per head is outside 1..{MAX_ROWS}")
         lib = load_module(f"scan_r{rows}", ["scan.cu"], [f"-DIB_ROWS={rows}"])
         lib.ib_wkv_scan.argtypes = [_c_void_p, _c_void_p, _c_int, _c_void_p, _c_ll, _c_void_p, _c_void_p, _c_void_p,
-                                    _c_int, _c_int, _c_int, _c_int, _c_void_p]
+                                    _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p]
         lib.ib_ssd_scan.argtypes = [_c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_ll, _c_void_p,
                                     _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p]
         lib.ib_delta_scan.argtypes = [_c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_ll, _c_void_p, _c_void_p,
@@ -105,7 +105,7 @@ def wkv_scan(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: torch.Tensor,
     slices = choose_col_slices(ctx.n_entries, heads, K, lib.ib_scan_split(), sm)
     core.check(lib.ib_wkv_scan(factors.data_ptr(), v32.data_ptr(), N, ptr, stride, ctx.cu_rows.data_ptr(),
                                ctx.slot_ids.data_ptr(), out.data_ptr(), ctx.n_entries, heads, K, slices,
-                               core.stream_ptr(r)), "wkv_scan")
+                               getattr(ctx, "max_rows_per_entry", N), core.stream_ptr(r)), "wkv_scan")
 
 
 # Up to this rank the pass before ``gla_scan`` makes the decays' low-rank product itself.
@@ -153,7 +153,7 @@ def gla_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, lo_off: int
     slices = choose_col_slices(ctx.n_entries, heads, vdim, lib.ib_scan_split(), sm)
     core.check(lib.ib_gla_scan(factors.data_ptr(), v32.data_ptr(), N, ptr, stride, ctx.cu_rows.data_ptr(),
                                ctx.slot_ids.data_ptr(), out.data_ptr(), ctx.n_entries, heads, vdim, slices,
-                               core.stream_ptr(proj)), "gla_scan")
+                               getattr(ctx, "max_rows_per_entry", N), core.stream_ptr(proj)), "gla_scan")
 
 
 def ssd_scan(xbc: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor, d_skip: torch.Tensor,
