@@ -276,6 +276,17 @@ gla_prepare_kernel(const T* __restrict__ x, int ld, int q_off, int k_off, int v_
     };
     if (ROWS == 1 && !z) fetch_w(0);
     pdl_wait();
+    // everything the rows hold for this channel is asked for before the low-rank sum
+    T qv[ROWS], kv[ROWS], vv[ROWS];
+#pragma unroll
+    for (int r = 0; r < ROWS; ++r) {
+        const T* xr = x + (size_t)(r0 + min(r, nr - 1)) * ld;
+        if (c < hk) {
+            qv[r] = xr[q_off + c];
+            kv[r] = xr[k_off + c];
+        }
+        if (c < hp) vv[r] = xr[v_off + c];
+    }
     if (z) {
 #pragma unroll
         for (int r = 0; r < ROWS; ++r)
@@ -300,17 +311,16 @@ gla_prepare_kernel(const T* __restrict__ x, int ld, int q_off, int k_off, int v_
 #pragma unroll
         for (int r = 0; r < ROWS; ++r) {
             if (r >= nr) break;
-            const T* xr = x + (size_t)(r0 + r) * ld;
             const float log_a = fminf(acc[r], 0.f) - log1pf(expf(-fabsf(acc[r])));  // log sigmoid(z), never above 0
             f[((size_t)head * n_rows + r0 + r) * K + (c - head * K)] =
-                make_float4(to_f32(xr[q_off + c]) * q_scale, to_f32(xr[k_off + c]), expf(log_a * inv_tau), 0.f);
+                make_float4(to_f32(qv[r]) * q_scale, to_f32(kv[r]), expf(log_a * inv_tau), 0.f);
         }
     }
     if (c < hp) {
         const int head = c / P;
 #pragma unroll
         for (int r = 0; r < ROWS; ++r)
-            if (r < nr) vo[((size_t)head * n_rows + r0 + r) * P + (c - head * P)] = to_f32(x[(size_t)(r0 + r) * ld + v_off + c]);
+            if (r < nr) vo[((size_t)head * n_rows + r0 + r) * P + (c - head * P)] = to_f32(vv[r]);
     }
 }
 
