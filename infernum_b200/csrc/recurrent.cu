@@ -256,10 +256,11 @@ constexpr int GLA_PIECE = 16;
 
 template <typename T, int ROWS>
 __global__ void __launch_bounds__(128)
-gla_prepare_kernel(const T* __restrict__ x, int ld, int q_off, int k_off, int v_off, int lo_off, int rank,
-                   const T* __restrict__ w2, const float* __restrict__ bias, const float* __restrict__ z,
-                   float q_scale, float inv_tau, float4* __restrict__ f, float* __restrict__ vo, int heads, int K,
-                   int P, int n_rows) {
+gla_prepare_kernel(const T* x, int ld, int q_off, int k_off, int v_off, int lo_off, int rank,
+                   const T* __restrict__ w2, const float* __restrict__ bias, const float* z, float q_scale,
+                   float inv_tau, float4* f, float* vo, int heads, int K, int P, int n_rows) {
+    // (x and z come from the kernel before and are not __restrict__: what a const __restrict__ pointer names may be
+    // taken as never written and fetched ahead of pdl_wait, as the weights are here on purpose)
     pdl_trigger();
     static_assert(ROWS * GLA_PIECE <= 128, "a piece of all rows is one value a thread");
     __shared__ float lo_s[ROWS][GLA_PIECE];

@@ -135,7 +135,7 @@ def random_case(seed: int) -> dict:
                               rng.choice([1.0, 4.0, 16.0]), mlp()))
         else:
             heads, dim, vdim = rng.choice([1, 2, 4, 8, 12]), rng.choice([16, 24, 32, 64]), rng.choice([16, 24, 32, 48])
-            q_rank, scale = rng.choice([24, 40, 64, 80]), rng.choice([0.1, 0.2, 0.3])
+            q_rank, scale = rng.choice([24, 40, 64, 72]), rng.choice([0.1, 0.2, 0.3])
             if owners and rng.random() < 0.6:
                 at = rng.choice(owners)
                 m = layers[at]["mixer"]
